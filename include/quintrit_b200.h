@@ -202,6 +202,8 @@ typedef struct quintrit_b200_decoder quintrit_b200_decoder_t;
 #define QUINTRIT_B200_ARCH_BITNET 1 /* BitNet b1.58: NEOX RoPE pairs, squared ReLU, attention and FFN sub-norms (config.rs:419-422) */
 #define QUINTRIT_B200_ARCH_QWEN 2   /* Qwen2 / Qwen3: NEOX RoPE pairs (config.rs:464-467), SwiGLU; Qwen3 adds query/key-norm (desc.qk_norms) */
 
+#define QUINTRIT_B200_ARCH_LAYERED 3 /* a model folder whose layers differ from one another (quintrit_b200_decoder_open_gguf below); not a value of decoder_desc.arch */
+
 /*
  * Description of a model whose ternary projections are already on the device. It plays the part of GpuModel::load
  * (quintrit-runtime/src/gpu.rs:183-260) after the GGUF has been read: dense tables are given as host pointers and copied.
@@ -289,6 +291,12 @@ typedef struct quintrit_gpu_options {
  * QUINTRIT_ERR_FORMAT, a missing or mis-shaped tensor QUINTRIT_ERR_MODEL, and mixture-of-experts, hybrid and
  * query/key-norm models QUINTRIT_ERR_UNSUPPORTED (a file whose projections are all Q2_0 runs through the block-scaled kernels). On failure *out_decoder is NULL. The decoder owns the weights.
  */
+/* `path` may also be a model folder (config.json + model.safetensors): config.json's "architecture" names the design, and its sizes, constants
+ * and layers describe the model (Lasosun: mamba2, hgrn2 and windowed attention layers). Such a model serves in bfloat16, or in 32-bit
+ * arithmetic throughout with the flag QUINTRIT_B200_OPEN_FLOAT32 in options.flags (also of quintrit_model_open_gpu). Its layers keep recurrent
+ * states and windows instead of a cache of every token, so a sequence continues from its end or starts again from position 0
+ * (QUINTRIT_ERR_UNSUPPORTED for a position between), and its context may have any length up to the model's number of positions. */
+#define QUINTRIT_B200_OPEN_FLOAT32 0x100u
 int quintrit_b200_decoder_open_gguf(const char* path, const quintrit_gpu_options_t* options, quintrit_b200_decoder_t** out_decoder);
 
 /* Shape of a decoder (the part of quintrit_model_info, quintrit.h:410-420, that concerns the device). */
@@ -454,6 +462,10 @@ struct quintrit_session;
  * quintrit_session_logits. QUINTRIT_ERR_CONTEXT_OVERFLOW if the tokens do not fit, QUINTRIT_ERR_BUSY if another thread
  * uses the session. */
 int quintrit_session_feed_tokens(struct quintrit_session* session, const uint32_t* tokens, size_t count, uint32_t flags);
+/* The same, and the logits at several places: `want` lists ascending indices into `tokens`, out receives [want_count][vocab] floats (capacity
+ * counts floats). A layered model computes them in the pass that ingests the tokens. */
+int quintrit_b200_session_feed_at(struct quintrit_session* session, const uint32_t* tokens, size_t count, uint32_t flags, const uint32_t* want, size_t want_count,
+                                  float* out, size_t capacity);
 /* Copies the logits of the last position fed (vocab_size floats); QUINTRIT_ERR_INVALID_ARGUMENT if there are none. */
 int quintrit_session_logits(struct quintrit_session* session, float* out, size_t capacity);
 /* Greedy decoding from position 0 without leaving the device between tokens (quintrit_b200_decoder_generate on the

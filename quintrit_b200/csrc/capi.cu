@@ -2,6 +2,8 @@
 // matrices into the stream layout, the exact GEMV with host or device buffers, and the persistent multi-GEMV plan.
 // Host code is C++ over the CUDA runtime API; the reference's host side for the same seam is
 // rust/crates/quintrit-cuda/src/{device.rs,gemv.rs,pack.rs} and rust/crates/quintrit-c/src/cuda.rs.
+#include <sys/stat.h>
+
 #include <algorithm>
 #include <cmath>
 #include <cstdlib>
@@ -13,6 +15,7 @@
 #include "gemv_lut.cuh"
 #include "transcode.cuh"
 #include "gemm_tc.cuh"
+#include "tensor_map.cuh"
 #include "block_scaled.cuh"
 
 using namespace qtb;
@@ -214,6 +217,7 @@ struct DeviceGuard {
 }  // namespace
 
 #include "decoder.cuh"
+#include "layered.cuh"
 #include "moe.cuh"
 #include "gguf.hpp"
 
@@ -1440,6 +1444,7 @@ struct GgufModel {
     const uint16_t* head = nullptr;
     const float* out_norm = nullptr;
     uint32_t table_type = kGgmlF16;
+    std::shared_ptr<LayeredModel> layered;  // a model folder: everything but the shape above is unused
     GgufModel() = default;
     GgufModel(const GgufModel&) = delete;
     GgufModel& operator=(const GgufModel&) = delete;
@@ -1448,12 +1453,45 @@ struct GgufModel {
     }
     // Largest context a decoder of this model may have: the model's maximum, at most `limit` (0: 4096) and 7936, rounded down to
     // a multiple of 256 when it reaches 256 (gpu.rs:141-146).
+    // A layered model keeps windows and states instead of a cache of the whole context: any length up to its position table.
     uint32_t context_for(uint32_t limit) const {
+        if (layered) return static_cast<uint32_t>(std::min<uint64_t>(shape.ctx_train, limit != 0 ? limit : shape.ctx_train));
         uint64_t want = std::min<uint64_t>(shape.ctx_train, limit != 0 ? limit : 4096);
         want = std::min<uint64_t>(want, 7936);
         return static_cast<uint32_t>(want >= 256 ? want / 256 * 256 : want);
     }
 };
+
+// A model folder (config.json + model.safetensors; the design is chosen by config.json).
+int load_model_folder(const char* path, uint32_t device, bool f32, GgufModel* out) {
+    cudaDeviceProp prop;
+    int rc = require_b200(static_cast<int>(device), &prop);
+    if (rc != QUINTRIT_OK) return rc;
+    DeviceGuard g(static_cast<int>(device));
+    out->device = device;
+    if ((rc = load_layered_model(path, static_cast<int>(device), f32, &out->layered)) != QUINTRIT_OK) return rc;
+    const LayeredSpec& s = out->layered->spec;
+    GgufModelShape& m = out->shape;
+    m.arch = s.design, m.arch_id = QUINTRIT_B200_ARCH_LAYERED;
+    for (char& c : m.arch) c = static_cast<char>(std::tolower(static_cast<unsigned char>(c)));
+    m.vocab = s.vocab, m.hidden = s.width, m.layers = s.layers.size(), m.ctx_train = s.max_positions, m.eps = s.eps, m.tied = s.head == s.embed;
+    for (const LayerSpec& l : s.layers) {
+        m.inter = std::max<uint64_t>(m.inter, l.ff);
+        if (l.kind == MixerKind::kAttention && m.heads == 0) m.heads = l.heads, m.kv_heads = l.kv_heads, m.head_dim = l.dim;
+    }
+    return QUINTRIT_OK;
+}
+
+int load_gguf_model(const char* path, uint32_t device, GgufModel* out);
+
+// A model by its path: a folder, or a GGUF file.
+int load_model(const char* path, uint32_t device, uint32_t flags, GgufModel* out) {
+    const bool f32 = (flags & QUINTRIT_B200_OPEN_FLOAT32) != 0;
+    struct stat st;
+    if (::stat(path, &st) == 0 && S_ISDIR(st.st_mode)) return load_model_folder(path, device, f32, out);
+    if (f32) return fail(QUINTRIT_ERR_UNSUPPORTED, "32-bit mode is available for model folders; a GGUF file's arithmetic is that of its ternary encoding");
+    return load_gguf_model(path, device, out);
+}
 
 // Reads the file, checks what the decoder needs and places the ternary projections on GPU `device` (the loading half of
 // GpuModel::load, gpu.rs:183-260).
@@ -1535,6 +1573,17 @@ int load_gguf_model(const char* path, uint32_t device, GgufModel* out) {
 
 // A decoder (KV cache, buffers, copies of the dense tables) over a loaded model; the model keeps the projections.
 int decoder_from_model(const GgufModel& md, uint32_t ctx, quintrit_b200_decoder** out) {
+    if (md.layered) {
+        DeviceGuard g(static_cast<int>(md.device));
+        quintrit_b200_decoder* d = nullptr;
+        const int rc = layered_decoder_create(md.layered, ctx, &d);
+        if (rc != QUINTRIT_OK) {
+            destroy_decoder(d);
+            return rc;
+        }
+        *out = d;
+        return QUINTRIT_OK;
+    }
     const GgufModelShape& m = md.shape;
     quintrit_b200_decoder_desc_t desc;
     std::memset(&desc, 0, sizeof desc);
@@ -1563,16 +1612,17 @@ int decoder_from_model(const GgufModel& md, uint32_t ctx, quintrit_b200_decoder*
 }
 
 int open_gguf_impl(const char* path, const quintrit_gpu_options_t* options, quintrit_b200_decoder** out) {
-    uint32_t device = 0, want_ctx = 0;
+    uint32_t device = 0, want_ctx = 0, flags = 0;
     if (options != nullptr) {
         if (options->struct_size < sizeof(quintrit_gpu_options_t))
             return fail(QUINTRIT_ERR_INVALID_ARGUMENT, "struct_size %u is smaller than quintrit_gpu_options_t (%zu)", options->struct_size, sizeof(quintrit_gpu_options_t));
-        if (options->flags & ~1u) return fail(QUINTRIT_ERR_INVALID_ARGUMENT, "unknown flag bits 0x%x", options->flags);
+        if (options->flags & ~(1u | QUINTRIT_B200_OPEN_FLOAT32)) return fail(QUINTRIT_ERR_INVALID_ARGUMENT, "unknown flag bits 0x%x", options->flags);
         device = options->device_index;
         want_ctx = options->context_length;
+        flags = options->flags;
     }
     GgufModel md;
-    int rc = load_gguf_model(path, device, &md);
+    int rc = load_model(path, device, flags, &md);
     if (rc != QUINTRIT_OK) return rc;
     const uint32_t ctx = md.context_for(want_ctx);
     if (ctx == 0) return fail(QUINTRIT_ERR_INVALID_ARGUMENT, "the context window of the model is empty");
@@ -1755,6 +1805,7 @@ extern "C" int quintrit_b200_decoder_forward(quintrit_b200_decoder_t* decoder, u
         if (token >= static_cast<uint32_t>(d->vocab_full)) return fail(QUINTRIT_ERR_INVALID_ARGUMENT, "token id %u is not below the vocabulary size %d", token, d->vocab_full);
         if (pos >= static_cast<uint32_t>(d->ctx)) return fail(QUINTRIT_ERR_CONTEXT_OVERFLOW, "position %u does not fit the context window of %d tokens", pos, d->ctx);
         if (pos > d->host_pos) return fail(QUINTRIT_ERR_INVALID_ARGUMENT, "position %u skips positions: %u tokens are cached", pos, d->host_pos);
+        if (d->lay && (rc = layered_check_position(d, pos, d->host_pos)) != QUINTRIT_OK) return rc;
         if (logits != nullptr && logits_capacity < static_cast<size_t>(d->vocab)) return fail(QUINTRIT_ERR_BUFFER_TOO_SMALL, "logits hold %zu values, the vocabulary has %d", logits_capacity, d->vocab);
         DeviceGuard g(d->device);
         if ((rc = decoder_set(d, token, pos)) != QUINTRIT_OK || (rc = decoder_step(d)) != QUINTRIT_OK) return rc;
@@ -1783,8 +1834,8 @@ extern "C" int quintrit_b200_decoder_generate(quintrit_b200_decoder_t* decoder, 
         uint32_t* d_prompt = nullptr;
         QTB_CUDA(cudaMalloc(&d_prompt, prompt_len * sizeof(uint32_t)));
         cudaError_t e = cudaMemcpyAsync(d_prompt, prompt, prompt_len * sizeof(uint32_t), cudaMemcpyHostToDevice, d->stream);
-        if (e == cudaSuccess) rc = decoder_set(d, prompt[0], 0);
-        for (size_t i = 0; e == cudaSuccess && rc == QUINTRIT_OK && i < prompt_len; ++i) {
+        if (e == cudaSuccess) rc = d->lay ? layered_prefill(d, prompt, prompt_len, 0, nullptr, 0, nullptr, 0, nullptr) : decoder_set(d, prompt[0], 0);
+        for (size_t i = 0; e == cudaSuccess && rc == QUINTRIT_OK && i < prompt_len && !d->lay; ++i) {
             rc = decoder_step(d);
             if (rc == QUINTRIT_OK && i + 1 < prompt_len)  // the next prompt token replaces the prediction
                 e = cudaMemcpyAsync(d->d_token, d_prompt + i + 1, sizeof(uint32_t), cudaMemcpyDeviceToDevice, d->stream);
@@ -1819,6 +1870,7 @@ extern "C" int quintrit_b200_decoder_time_token(quintrit_b200_decoder_t* decoder
         QTB_CUDA(cudaEventCreate(&e1));
         float best = 1e30f;
         if (!d->use_mega && (rc = decoder_graph(d)) != QUINTRIT_OK) return rc;
+        if (d->lay && (rc = layered_save(d, false)) != QUINTRIT_OK) return rc;
         for (uint32_t b = 0; b < blocks; ++b) {
             cudaEventRecord(e0, d->stream);
             for (uint32_t i = 0; i < iters; ++i) {
@@ -1834,6 +1886,10 @@ extern "C" int quintrit_b200_decoder_time_token(quintrit_b200_decoder_t* decoder
         cudaEventDestroy(e0);
         cudaEventDestroy(e1);
         QTB_CUDA(cudaGetLastError());
+        if (d->lay) {
+            if ((rc = layered_save(d, true)) != QUINTRIT_OK) return rc;
+            QTB_CUDA(cudaStreamSynchronize(d->stream));
+        }
         *out_ms = best;
         return ok();
     });
@@ -2026,23 +2082,6 @@ namespace {
 std::mutex g_gemm_lock;
 constexpr int kGemmMaxParts = 8;
 constexpr size_t kGemmSmemLimit = 227 * 1024;  // dynamic shared memory a CTA may ask for on this device
-typedef CUresult (*TensorMapEncodeFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*, const cuuint32_t*, const cuuint32_t*,
-                                      CUtensorMapInterleave, CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
-
-// The driver's tensor-map encoder, fetched at run time so that the library loads on a machine without a driver.
-int tensor_map_encoder(TensorMapEncodeFn* out) {
-    static TensorMapEncodeFn fn = nullptr;
-    if (fn == nullptr) {
-        void* p = nullptr;
-        cudaDriverEntryPointQueryResult q = cudaDriverEntryPointSymbolNotFound;
-        const cudaError_t e = cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &p, cudaEnableDefault, &q);
-        if (e != cudaSuccess || q != cudaDriverEntryPointSuccess || p == nullptr) return fail(QUINTRIT_ERR_DEVICE, "the CUDA driver does not provide cuTensorMapEncodeTiled");
-        fn = reinterpret_cast<TensorMapEncodeFn>(p);
-    }
-    *out = fn;
-    return QUINTRIT_OK;
-}
-
 // Makes the two-bit copy of the weights and the call buffers of a matrix the first time it is used by the batched projection.
 int gemm_prepare(quintrit_b200_matrix* m) {
     std::lock_guard<std::mutex> hold(g_gemm_lock);
@@ -2286,7 +2325,7 @@ int decoder_gemm_prepare(quintrit_b200_decoder* d) {
 }
 
 int prefill_buffers(quintrit_b200_decoder* d) {
-    if (d->pf.x != nullptr) return QUINTRIT_OK;
+    if (d->pf.x != nullptr || d->lay) return QUINTRIT_OK;  // (a layered decoder made its buffers when it was created)
     const size_t B = kPrefillMax, H = d->hidden, I = d->inter, qd = d->q_dim, kvd = d->kv_dim, hd = d->head_dim;
     int rc;
     if ((rc = dev_alloc(d, &d->pf.tokens, B)) != QUINTRIT_OK || (rc = dev_alloc(d, &d->pf.pos, 4)) != QUINTRIT_OK || (rc = dev_alloc(d, &d->pf.x, B * H)) != QUINTRIT_OK ||
@@ -2310,6 +2349,8 @@ struct BatchTarget {
     const uint32_t* pos = nullptr;
     SeqIndex seq{nullptr, 0, 0};
     bool own = true;                      // the decoder's own cache: a full chunk may be replayed as the captured graph
+    const LayeredStore* layered = nullptr;  // layered models: the sequence store and the slot of a prompt's sequence
+    int slot = 0;
 };
 BatchTarget own_target(quintrit_b200_decoder* d) {
     BatchTarget t;
@@ -2455,10 +2496,11 @@ int enqueue_prefill_chunk(quintrit_b200_decoder* d, int n, uint32_t pos0, bool w
 
 // Whether a decoder can ingest prompts in chunks: per-tensor ternary projections on one GPU (the block-scaled and tensor-parallel decoders
 // take their prompts token by token).
-bool prefill_available(const quintrit_b200_decoder* d) { return !d->block_scaled && d->tp_world == 1 && d->hidden % 32 == 0 && d->inter % 32 == 0 && d->q_dim % 32 == 0; }
+bool prefill_available(const quintrit_b200_decoder* d) { return d->lay || (!d->block_scaled && d->tp_world == 1 && d->hidden % 32 == 0 && d->inter % 32 == 0 && d->q_dim % 32 == 0); }
 
 // Tokens at positions pos0 .. pos0 + count - 1, chunk by chunk; ends like a single step of the last token (logits, greedy token, position).
 int decoder_prefill(quintrit_b200_decoder* d, const uint32_t* tokens, size_t count, uint32_t pos0, const BatchTarget* target = nullptr) {
+    if (d->lay) return layered_prefill(d, tokens, count, pos0, target != nullptr ? target->layered : nullptr, target != nullptr ? target->slot : 0, nullptr, 0, nullptr);
     int rc = prefill_buffers(d);
     if (rc != QUINTRIT_OK) return rc;
     if ((rc = decoder_gemm_prepare(d)) != QUINTRIT_OK) return rc;
@@ -2489,6 +2531,7 @@ extern "C" int quintrit_b200_decoder_prefill(quintrit_b200_decoder_t* decoder, c
         if (!prefill_available(d)) return fail(QUINTRIT_ERR_UNSUPPORTED, "this decoder takes its prompt token by token (block-scaled or tensor-parallel model)");
         if (size_t(pos) + count > static_cast<size_t>(d->ctx)) return fail(QUINTRIT_ERR_CONTEXT_OVERFLOW, "%zu tokens from position %u do not fit the context window of %d tokens", count, pos, d->ctx);
         if (pos > d->host_pos) return fail(QUINTRIT_ERR_INVALID_ARGUMENT, "position %u skips positions: %u tokens are cached", pos, d->host_pos);
+        if (d->lay && (rc = layered_check_position(d, pos, d->host_pos)) != QUINTRIT_OK) return rc;
         for (size_t i = 0; i < count; ++i)
             if (tokens[i] >= static_cast<uint32_t>(d->vocab_full)) return fail(QUINTRIT_ERR_INVALID_ARGUMENT, "token id %u is not below the vocabulary size %d", tokens[i], d->vocab_full);
         if (logits != nullptr && logits_capacity < static_cast<size_t>(d->vocab)) return fail(QUINTRIT_ERR_BUFFER_TOO_SMALL, "logits hold %zu values, the vocabulary has %d", logits_capacity, d->vocab);
@@ -2860,6 +2903,7 @@ struct quintrit_b200_batch {
     uint32_t *d_pos = nullptr, *d_last = nullptr, *d_slot = nullptr, *d_chosen = nullptr;
     float* logits = nullptr;               // [n_seq][vocab] of the last step
     __half* x16 = nullptr;                 // [n_seq][hidden]: the final norm's output
+    LayeredStore layered;                  // layered models: states and windows of the sequences instead of kc / vc
     std::vector<uint32_t> host_pos;        // tokens cached per sequence
     std::vector<uint32_t> staged;          // host copy of the ids given to an asynchronous copy
     std::vector<void*> allocs;
@@ -2903,12 +2947,29 @@ int batch_alloc(quintrit_b200_batch* b, T** p, size_t count) {
     return QUINTRIT_OK;
 }
 
-size_t batch_cache_stride(const quintrit_b200_decoder* d) { return static_cast<size_t>(d->layers) * d->ctx * d->kv_dim; }
+size_t batch_cache_stride(const quintrit_b200_decoder* d) { return d->lay ? 0 : static_cast<size_t>(d->layers) * d->ctx * d->kv_dim; }
+
+// A step of several sequences of a layered model.
+int layered_batch_layers(quintrit_b200_batch* b, int n, const BatchTarget& tg) {
+    LayeredTarget t;
+    t.store = &b->layered, t.pos = tg.pos, t.seq = tg.seq;
+    return layered_run(b->d, b->d->lay->tokens, n, t);
+}
 
 // The output head for the n tokens of a step: final norm per token, then every vocabulary row against all tokens, then the greedy choice per token.
 int batch_head(quintrit_b200_batch* b, int n) {
     quintrit_b200_decoder* d = b->d;
     cudaStream_t s = d->stream;
+    if (d->lay) {
+        for (int t = 0; t < n; t += kDenseN) {
+            const int here = std::min(n - t, kDenseN);
+            const int rc = layered_logits_rows(d, t, here, b->logits + size_t(t) * d->vocab);
+            if (rc != QUINTRIT_OK) return rc;
+        }
+        argmax_kernel<<<n, 1024, 0, s>>>(b->logits, d->vocab, b->d_chosen);
+        QTB_LAUNCH_CHECK();
+        return QUINTRIT_OK;
+    }
     const int H = d->hidden;
     NormQuantArgs nf{};
     nf.x = d->pf.x, nf.b_x = H, nf.acc_prev = d->pf.acc_down, nf.b_acc = H, nf.scale_prev = d->pf.s_i, nf.b_scale = 1;
@@ -2944,13 +3005,17 @@ extern "C" int quintrit_b200_batch_create(quintrit_b200_decoder_t* decoder, uint
         if (!prefill_available(d)) return fail(QUINTRIT_ERR_UNSUPPORTED, "this decoder has no batched pass (block-scaled or tensor-parallel model)");
         DeviceGuard g(d->device);
         if ((rc = prefill_buffers(d)) != QUINTRIT_OK) return rc;
-        if ((rc = decoder_gemm_prepare(d)) != QUINTRIT_OK) return rc;
+        if (!d->lay && (rc = decoder_gemm_prepare(d)) != QUINTRIT_OK) return rc;
         quintrit_b200_batch* b = new quintrit_b200_batch();
         b->magic = kMagicBatch, b->d = d, b->device = d->device, b->n_seq = static_cast<int>(sequences);
         b->host_pos.assign(sequences, 0);
         b->graph.assign(sequences + 1, nullptr);
         b->warm.assign(sequences + 1, 0);
         const size_t n = sequences;
+        if (d->lay && (rc = layered_store_create(*d->lay->model, static_cast<int>(sequences), d->ctx, [&](void** p, size_t bytes) { return batch_alloc(b, reinterpret_cast<char**>(p), bytes); }, &b->layered)) != QUINTRIT_OK) {
+            destroy_batch(b);
+            return rc;
+        }
         if ((rc = batch_alloc(b, &b->kc, n * batch_cache_stride(d))) != QUINTRIT_OK || (rc = batch_alloc(b, &b->vc, n * batch_cache_stride(d))) != QUINTRIT_OK ||
             (rc = batch_alloc(b, &b->d_pos, n)) != QUINTRIT_OK || (rc = batch_alloc(b, &b->d_last, n)) != QUINTRIT_OK || (rc = batch_alloc(b, &b->d_slot, n)) != QUINTRIT_OK ||
             (rc = batch_alloc(b, &b->d_chosen, n)) != QUINTRIT_OK || (rc = batch_alloc(b, &b->logits, n * d->vocab)) != QUINTRIT_OK ||
@@ -2958,6 +3023,7 @@ extern "C" int quintrit_b200_batch_create(quintrit_b200_decoder_t* decoder, uint
             destroy_batch(b);
             return rc;
         }
+        QTB_CUDA(cudaDeviceSynchronize());
         *out_batch = b;
         return ok();
     });
@@ -2988,6 +3054,7 @@ extern "C" int quintrit_b200_batch_rewind(quintrit_b200_batch_t* batch, uint32_t
         if (rc != QUINTRIT_OK) return rc;
         if (sequence >= static_cast<uint32_t>(batch->n_seq)) return fail(QUINTRIT_ERR_INVALID_ARGUMENT, "sequence %u of %d", sequence, batch->n_seq);
         if (position > batch->host_pos[sequence]) return fail(QUINTRIT_ERR_INVALID_ARGUMENT, "position %u skips positions: %u tokens are cached", position, batch->host_pos[sequence]);
+        if (batch->d->lay && (rc = layered_check_position(batch->d, position, batch->host_pos[sequence])) != QUINTRIT_OK) return rc;
         DeviceGuard g(batch->d->device);
         QTB_CUDA(cudaMemcpyAsync(batch->d_pos + sequence, &position, sizeof position, cudaMemcpyHostToDevice, batch->d->stream));
         QTB_CUDA(cudaStreamSynchronize(batch->d->stream));
@@ -3015,6 +3082,7 @@ extern "C" int quintrit_b200_batch_prefill(quintrit_b200_batch_t* batch, uint32_
         b->staged.assign(tokens, tokens + count);
         BatchTarget tg;
         tg.kc = b->kc + sequence * batch_cache_stride(d), tg.vc = b->vc + sequence * batch_cache_stride(d), tg.pos = d->pf.pos, tg.own = false;
+        tg.layered = d->lay ? &b->layered : nullptr, tg.slot = static_cast<int>(sequence);
         if ((rc = decoder_prefill(d, b->staged.data(), count, pos, &tg)) != QUINTRIT_OK) return rc;
         const uint32_t next = pos + static_cast<uint32_t>(count);
         QTB_CUDA(cudaMemcpyAsync(b->d_pos + sequence, &next, sizeof next, cudaMemcpyHostToDevice, d->stream));
@@ -3064,18 +3132,19 @@ extern "C" int quintrit_b200_batch_step(quintrit_b200_batch_t* batch, const uint
             if (tokens != nullptr) b->staged[count + k] = tokens[order[k]];
         }
         const uint32_t* slot = b->d_slot;
+        uint32_t* step_tokens = d->lay ? d->lay->tokens : d->pf.tokens;
         QTB_CUDA(cudaMemcpyAsync(b->d_slot, b->staged.data(), count * sizeof(uint32_t), cudaMemcpyHostToDevice, s));
         if (tokens != nullptr) {
-            QTB_CUDA(cudaMemcpyAsync(d->pf.tokens, b->staged.data() + count, count * sizeof(uint32_t), cudaMemcpyHostToDevice, s));
+            QTB_CUDA(cudaMemcpyAsync(step_tokens, b->staged.data() + count, count * sizeof(uint32_t), cudaMemcpyHostToDevice, s));
         } else {
-            gather_tokens_kernel<<<(n + 255) / 256, 256, 0, s>>>(d->pf.tokens, b->d_last, slot, n);
+            gather_tokens_kernel<<<(n + 255) / 256, 256, 0, s>>>(step_tokens, b->d_last, slot, n);
             QTB_LAUNCH_CHECK();
         }
         BatchTarget tg;
         tg.kc = b->kc, tg.vc = b->vc, tg.pos = b->d_pos, tg.own = false;
         tg.seq.slot = slot, tg.seq.pos_stride = 1, tg.seq.cache_stride = batch_cache_stride(d);
         auto enqueue = [&]() -> int {
-            int r = prefill_layers(d, n, tg);
+            int r = d->lay ? layered_batch_layers(b, n, tg) : prefill_layers(d, n, tg);
             if (r == QUINTRIT_OK) r = batch_head(b, n);
             if (r != QUINTRIT_OK) return r;
             advance_batch_kernel<<<(n + 255) / 256, 256, 0, s>>>(b->d_pos, b->d_last, b->d_chosen, slot, n);

@@ -11,6 +11,9 @@
 #include "gemv_lut.cuh"
 #include "megakernel.cuh"
 
+namespace qtb {
+struct LayeredDecoder;  // layered.cuh: a model whose layers differ from one another
+}
 struct quintrit_b200_matrix;
 void qtb_release_stacked(quintrit_b200_matrix* m);  // capi.cu: deletes the host object of a stacked matrix
 
@@ -58,6 +61,7 @@ struct quintrit_b200_decoder {
     bool graph_ready;
     uint32_t host_pos;                         // tokens in the KV cache
     // tensor parallelism: this rank's share of a model split over tp_world GPUs (1 = none)
+    qtb::LayeredDecoder* lay = nullptr;        // weights, sequence store and buffers of a layered model; the ternary fields above stay empty
     bool block_scaled = false;                 // every projection is a block-scaled (Q2_0) matrix: Q8_0 activations, F32 results
     std::vector<const quintrit_b200_matrix*> mats;  // the projections (layers * 7), for the block-scaled launches
     float* q8_d = nullptr;                     // Q8_0 block scales of the current projection input
@@ -116,6 +120,9 @@ int dev_upload(quintrit_b200_decoder* d, T** p, const void* host, size_t count) 
     return QUINTRIT_OK;
 }
 
+void layered_release(quintrit_b200_decoder* d);
+int layered_enqueue_token(quintrit_b200_decoder* d, bool with_head);
+
 inline void destroy_decoder(quintrit_b200_decoder* d) {
     if (d == nullptr) return;
     int prev = -1;
@@ -128,6 +135,7 @@ inline void destroy_decoder(quintrit_b200_decoder* d) {
     for (quintrit_b200_matrix* m : d->pf.stacked_objects) qtb_release_stacked(m);
     if (d->stream) cudaStreamDestroy(d->stream);
     for (void* p : d->allocs) cudaFree(p);
+    if (d->lay) layered_release(d);
     if (prev >= 0) cudaSetDevice(prev);
     d->magic = 0;
     delete d;
@@ -182,6 +190,7 @@ inline void launch_attention(quintrit_b200_decoder* d, const AttnArgs& at, int n
 
 // The launch sequence of one token (gpu.rs:389-453 reshaped: 4 GEMV launches and 5 float kernels per layer).
 inline int enqueue_token(quintrit_b200_decoder* d, bool with_head) {
+    if (d->lay) return layered_enqueue_token(d, with_head);
     cudaStream_t s = d->stream;
     const int H = d->hidden, I = d->inter, qd = d->q_dim, kvd = d->kv_dim;
     const bool bs = d->block_scaled;  // Q2_0 model: the int32 result buffers hold F32 results, activations are Q8_0 blocks

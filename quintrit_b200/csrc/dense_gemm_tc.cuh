@@ -1,0 +1,268 @@
+// Dense projections of many tokens: out[t][r] = sum_k W[r][k] * h[t][k], with the endings of dense_gemv.cuh.
+//
+// 16-bit weights run on the 5th-generation tensor cores. A block makes one tile of 128 weight rows (the M of the instruction) x 128 tokens
+// (the N): one thread fetches 64-column slices of both operands with TMA (128-byte swizzle) into a ring of stages, one thread issues
+// tcgen05.mma.kind::f16 (bf16 operands, 32-bit sums in tensor memory), four warps read the sums with tcgen05.ld - a weight row per lane, so
+// that the 32 lanes of a warp write 32 neighbouring results of a token - and apply the ending. Two blocks share a multiprocessor: one's
+// ending overlaps the other's products. The grid runs over token tiles first, so the blocks that are resident together share weight rows.
+//
+// The dual form makes two products of one tile, W_o y and W_down m, in two accumulators and ends with both gates and the residual sum.
+// Every wait is bounded, as in gemm_tc.cuh, whose mbarrier, descriptor and status conventions are used here.
+//
+// 32-bit weights: a plain tiled kernel in 32-bit arithmetic with the same endings.
+#pragma once
+#include <cuda.h>
+
+#include "dense_gemv.cuh"
+#include "gemm_tc.cuh"
+
+namespace qtb {
+
+constexpr int kDenseM = 128, kDenseN = 128, kDenseK = 64;
+constexpr int kDenseStages = 3;
+constexpr int kDenseStageBytes = (kDenseM + kDenseN) * kDenseK * 2;
+constexpr int kDenseSmem = kDenseStages * kDenseStageBytes + 1024 + 256;
+constexpr int kDenseThreads = 192;  // TMA warp, MMA warp, four warps for the ending
+
+struct DenseGemmArgs {
+    int tokens;
+    int n_prob;              // plain form: 1 or 2 stacks, each over its own activations
+    int k_steps[2];          // 64-column slices
+    int row_tiles[2];
+    DenseStack stack[2];     // plain form: the endings
+    // dual form
+    float* x;
+    int width;
+    const float *gate1, *gate2;
+    unsigned int* status;
+    unsigned int spin_limit;
+};
+
+// One result of a plain-form tile. `pair` is the neighbouring row's value (SwiGLU: rows 2 i and 2 i + 1 are gate and up of channel i).
+template <typename T>
+__device__ __forceinline__ void dense_end(const DenseSeg& g, int row, int token, float v, float pair) {
+    if (row >= g.rows) return;
+    if (g.kind == kSegSwiGlu) {
+        if ((row & 1) == 0) static_cast<T*>(g.t)[size_t(token) * g.ld + (row >> 1)] = to_storage<T>(silu_f(v) * pair);
+    } else {
+        g.f[size_t(token) * g.ld + row] = g.kind == kSegSigmoid ? sigmoid_f(v + g.bias[row]) : v;
+    }
+}
+
+namespace dense_detail {
+__device__ __forceinline__ void tma_load_2d(uint32_t dst, const CUtensorMap* map, int x, int y, uint32_t bar) {
+    asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];" ::"r"(dst), "l"(map), "r"(x), "r"(y), "r"(bar) : "memory");
+}
+// kind::f16 with bf16 operands: F32 accumulator (1 at bit 4), BF16 A and B (1 at bits 7 and 10), both K-major, N / 8 at bit 17, M / 16 at bit 24.
+__device__ __forceinline__ uint32_t instr_desc_bf16(int m, int n) { return (1u << 4) | (1u << 7) | (1u << 10) | (uint32_t(n >> 3) << 17) | (uint32_t(m >> 4) << 24); }
+__device__ __forceinline__ void mma_bf16(uint32_t tmem_d, uint64_t desc_a, uint64_t desc_b, uint32_t idesc, uint32_t accumulate) {
+    const uint32_t zero = 0;  // no output lane is disabled
+    asm volatile(
+        "{\n\t.reg .pred p;\n\t"
+        "setp.ne.b32 p, %4, 0;\n\t"
+        "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, {%5, %5, %5, %5}, p;\n\t}" ::"r"(tmem_d),
+        "l"(desc_a), "l"(desc_b), "r"(idesc), "r"(accumulate), "r"(zero)
+        : "memory");
+}
+__device__ __forceinline__ void tmem_load16(uint32_t taddr, uint32_t (&v)[16]) {
+    asm volatile(
+        "tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0, %1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15}, [%16];"
+        : "=r"(v[0]), "=r"(v[1]), "=r"(v[2]), "=r"(v[3]), "=r"(v[4]), "=r"(v[5]), "=r"(v[6]), "=r"(v[7]), "=r"(v[8]), "=r"(v[9]), "=r"(v[10]), "=r"(v[11]), "=r"(v[12]), "=r"(v[13]),
+          "=r"(v[14]), "=r"(v[15])
+        : "r"(taddr));
+}
+}  // namespace dense_detail
+
+template <bool DUAL>
+__global__ void __launch_bounds__(kDenseThreads) dense_gemm_tc_kernel(const __grid_constant__ CUtensorMap w0, const __grid_constant__ CUtensorMap h0, const __grid_constant__ CUtensorMap w1,
+                                                                      const __grid_constant__ CUtensorMap h1, const __grid_constant__ DenseGemmArgs a) {
+    using namespace gemm_detail;
+    using namespace dense_detail;
+    extern __shared__ unsigned char dense_smem_raw[];
+    unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(dense_smem_raw) + 1023) & ~uintptr_t(1023));
+    constexpr int S = kDenseStages;
+    uint64_t* bars = reinterpret_cast<uint64_t*>(smem + S * kDenseStageBytes);
+    const uint32_t bar0 = smem_u32(bars), tiles0 = smem_u32(smem);
+    auto loaded = [&](int s) { return bar0 + 8u * s; };
+    auto empty = [&](int s) { return bar0 + 8u * (S + s); };
+    const uint32_t acc_full = bar0 + 8u * (2 * S);
+    volatile uint32_t* tmem_slot = reinterpret_cast<volatile uint32_t*>(bars + 2 * S + 1);
+    volatile unsigned int* abort_flag = reinterpret_cast<volatile unsigned int*>(bars + 2 * S + 2);
+
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int token0 = blockIdx.x * kDenseN;
+    const int prob = !DUAL && static_cast<int>(blockIdx.y) >= a.row_tiles[0] ? 1 : 0;
+    const int row0 = (static_cast<int>(blockIdx.y) - (prob ? a.row_tiles[0] : 0)) * kDenseM;
+    const int steps0 = a.k_steps[prob], steps = DUAL ? steps0 + a.k_steps[1] : steps0;
+    constexpr uint32_t tmem_cols = DUAL ? 2 * kDenseN : kDenseN;
+
+    if (tid == 0) {
+        for (int s = 0; s < S; ++s) {
+            mbar_init(loaded(s), 1);
+            mbar_init(empty(s), 1);
+        }
+        mbar_init(acc_full, 1);
+        *abort_flag = 0;
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    if (warp == 0) {
+        asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(const_cast<uint32_t*>(tmem_slot))), "r"(tmem_cols) : "memory");
+        asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
+    }
+    asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+    __syncthreads();
+    asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+    const uint32_t tmem_base = *tmem_slot;
+
+    if (warp == 0) {
+        if (lane == 0) {
+            int it = 0, s = 0;
+            uint32_t ph = 0;
+            for (; it < steps; ++it) {
+                if (!mbar_wait(empty(s), ph ^ 1, abort_flag, a.spin_limit)) break;
+                const bool second = DUAL ? it >= steps0 : prob != 0;
+                const int k = (DUAL && second ? it - steps0 : it) * kDenseK;
+                const uint32_t dst = tiles0 + s * kDenseStageBytes;
+                mbar_expect_tx(loaded(s), kDenseStageBytes);
+                tma_load_2d(dst, second ? &w1 : &w0, k, row0, loaded(s));
+                tma_load_2d(dst + kDenseM * kDenseK * 2, second ? &h1 : &h0, k, token0, loaded(s));
+                if (++s == S) s = 0, ph ^= 1;
+            }
+            for (int back = 0; back < min(it, S); ++back) {  // its copies in flight land before the block leaves
+                if (--s < 0) s = S - 1, ph ^= 1;
+                mbar_wait(loaded(s), ph, abort_flag, a.spin_limit, false);
+            }
+        }
+    } else if (warp == 1) {
+        if (lane == 0) {
+            const uint32_t idesc = instr_desc_bf16(kDenseM, kDenseN);
+            int s = 0;
+            uint32_t ph = 0;
+            for (int it = 0; it < steps; ++it) {
+                if (!mbar_wait(loaded(s), ph, abort_flag, a.spin_limit)) break;
+                asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+                const bool second = DUAL && it >= steps0;
+                const uint32_t at = tiles0 + s * kDenseStageBytes;
+                const uint64_t da = smem_desc(at, 16, 1024, 2), db = smem_desc(at + kDenseM * kDenseK * 2, 16, 1024, 2);  // 128-byte swizzle, 8-row groups 1024 bytes apart
+                const uint32_t acc = tmem_base + (second ? kDenseN : 0);
+                const bool first = it == 0 || (DUAL && it == steps0);
+#pragma unroll
+                for (int j = 0; j < kDenseK / 16; ++j) mma_bf16(acc, da + 2 * j, db + 2 * j, idesc, first && j == 0 ? 0u : 1u);
+                mma_commit(empty(s));
+                if (++s == S) s = 0, ph ^= 1;
+            }
+            mma_commit(acc_full);
+        }
+    } else {
+        const int r = (warp & 3) * 32 + lane;  // a warp reads the 32 lanes of tensor memory that its index modulo 4 selects
+        bool okay = true;
+        if (lane == 0) okay = mbar_wait(acc_full, 0, abort_flag, a.spin_limit);
+        okay = __shfl_sync(0xffffffffu, okay ? 1 : 0, 0) != 0 && *abort_flag == 0;
+        okay = __all_sync(0xffffffffu, okay);
+        if (okay) {
+            asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+            const uint32_t lane_base = tmem_base + (uint32_t((warp & 3) * 32) << 16);
+            const int n_here = min(kDenseN, a.tokens - token0);
+            if constexpr (DUAL) {
+                const int row = row0 + r;
+                const bool has2 = a.k_steps[1] > 0;
+                for (int c0 = 0; c0 < n_here; c0 += 16) {
+                    uint32_t v1[16], v2[16];
+                    tmem_load16(lane_base + c0, v1);
+                    if (has2) tmem_load16(lane_base + kDenseN + c0, v2);
+                    asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+                    if (row < a.width) {
+#pragma unroll
+                        for (int i = 0; i < 16; ++i)
+                            if (c0 + i < n_here) {
+                                const size_t at = size_t(token0 + c0 + i) * a.width + row;
+                                float add = __uint_as_float(v1[i]);
+                                if (a.gate1 != nullptr) add *= a.gate1[at];
+                                if (has2) add += __uint_as_float(v2[i]) * (a.gate2 != nullptr ? a.gate2[at] : 1.0f);
+                                a.x[at] += add;
+                            }
+                    }
+                }
+            } else {
+                const DenseStack& st = a.stack[prob];
+                const DenseSeg& g = st.seg[st.n_seg > 1 && row0 >= st.seg[1].row0 ? 1 : 0];
+                for (int c0 = 0; c0 < n_here; c0 += 16) {
+                    uint32_t v[16];
+                    tmem_load16(lane_base + c0, v);
+                    asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+#pragma unroll
+                    for (int i = 0; i < 16; ++i) {
+                        const float val = __uint_as_float(v[i]), pair = __shfl_xor_sync(0xffffffffu, val, 1);
+                        if (c0 + i < n_here) dense_end<bf16>(g, row0 + r - g.row0, token0 + c0 + i, val, pair);
+                    }
+                }
+            }
+        }
+    }
+    asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+    __syncthreads();
+    if (tid == 0 && *abort_flag) atomicExch(a.status, kGemmStatusTimeout);
+    if (warp == 0) {
+        asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+        asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem_base), "r"(tmem_cols) : "memory");
+    }
+}
+
+// ---- 32-bit products ------------------------------------------------------------------------------------------------------------------
+constexpr int kF32Tile = 64, kF32K = 16;
+
+template <bool DUAL>
+__global__ void __launch_bounds__(256) dense_gemm_f32_kernel(const float* w0, const float* h0, int pitch0, const float* w1, const float* h1, int pitch1, const __grid_constant__ DenseGemmArgs a) {
+    __shared__ float ws[kF32K][kF32Tile + 4], hs[kF32K][kF32Tile + 4];
+    const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
+    const int per = kDenseM / kF32Tile;  // row tiles are counted in units of kDenseM
+    const int token0 = blockIdx.x * kF32Tile;
+    const int prob = !DUAL && static_cast<int>(blockIdx.y) >= a.row_tiles[0] * per ? 1 : 0;
+    const int row0 = (static_cast<int>(blockIdx.y) - (prob ? a.row_tiles[0] * per : 0)) * kF32Tile;
+    float acc[2][4][4] = {};
+    for (int half = 0; half < (DUAL ? 2 : 1); ++half) {
+        const bool second = DUAL ? half == 1 : prob != 0;
+        const float *w = second ? w1 : w0, *h = second ? h1 : h0;
+        const int pitch = second ? pitch1 : pitch0, k_end = a.k_steps[second ? 1 : 0] * kDenseK;
+        for (int k0 = 0; k0 < k_end; k0 += kF32K) {
+            __syncthreads();
+            for (int i = tid; i < kF32Tile * kF32K; i += 256) {
+                const int r = i / kF32K, k = i % kF32K;
+                ws[k][r] = w[size_t(row0 + r) * pitch + k0 + k];
+                hs[k][r] = token0 + r < a.tokens ? h[size_t(token0 + r) * pitch + k0 + k] : 0.0f;
+            }
+            __syncthreads();
+#pragma unroll
+            for (int k = 0; k < kF32K; ++k) {
+                float wv[4], hv[4];
+#pragma unroll
+                for (int i = 0; i < 4; ++i) wv[i] = ws[k][tx * 4 + i], hv[i] = hs[k][ty * 4 + i];
+#pragma unroll
+                for (int i = 0; i < 4; ++i)
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) acc[half][i][j] = fmaf(wv[i], hv[j], acc[half][i][j]);
+            }
+        }
+    }
+    for (int j = 0; j < 4; ++j) {
+        const int token = token0 + ty * 4 + j;
+        if (token >= a.tokens) continue;
+        for (int i = 0; i < 4; ++i) {
+            const int row = row0 + tx * 4 + i;
+            if constexpr (DUAL) {
+                if (row >= a.width) continue;
+                const size_t at = size_t(token) * a.width + row;
+                float add = acc[0][i][j];
+                if (a.gate1 != nullptr) add *= a.gate1[at];
+                if (a.k_steps[1] > 0) add += acc[1][i][j] * (a.gate2 != nullptr ? a.gate2[at] : 1.0f);
+                a.x[at] += add;
+            } else {
+                const DenseStack& st = a.stack[prob];
+                const DenseSeg& g = st.seg[st.n_seg > 1 && row0 >= st.seg[1].row0 ? 1 : 0];
+                dense_end<float>(g, row - g.row0, token, acc[0][i][j], acc[0][i ^ 1][j]);
+            }
+        }
+    }
+}
+
+}  // namespace qtb

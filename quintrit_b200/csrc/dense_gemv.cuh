@@ -1,0 +1,289 @@
+// Dense (16- or 32-bit) projections of one token, fused with what stands before and after them: the kernels a layered decoder
+// (layered.cuh) takes a decode step with. Activations and sums are 32-bit; an activation is rounded to the storage type where the
+// batched path (dense_gemm_tc.cuh) stores it, so both paths round in the same places.
+//
+//   norm_project_kernel    RMS norms of the residual stream, then up to two stacked projections of them, each row range with its own
+//                          ending (plain, sigmoid of a gate, SwiGLU of interleaved gate | up rows)
+//   finish_project_kernel  the mixer's output norm, then output and down projection, both gates and the residual sum
+//
+// A warp owns two rows (one in the second kernel) and streams them with 16-byte loads, four per row in flight and lane; the activation
+// vector lies in shared memory as floats.
+#pragma once
+#include <cstdint>
+#include <cuda_bf16.h>
+#include <cuda_runtime.h>
+
+#include "decode.cuh"
+
+namespace qtb {
+
+typedef __nv_bfloat16 bf16;
+
+constexpr int kRowPad = 128;   // a stacked projection's row ranges start at multiples of this (the M of a tensor-core tile)
+constexpr int kColPad = 64;    // columns are padded with zeros to a multiple of this (a 128-byte swizzled TMA box)
+
+template <typename T> __device__ __forceinline__ T to_storage(float v);
+template <> __device__ __forceinline__ float to_storage<float>(float v) { return v; }
+template <> __device__ __forceinline__ bf16 to_storage<bf16>(float v) { return __float2bfloat16_rn(v); }
+__device__ __forceinline__ float from_storage(float v) { return v; }
+__device__ __forceinline__ float from_storage(bf16 v) { return __bfloat162float(v); }
+template <typename T> __device__ __forceinline__ float round_to(float v) { return from_storage(to_storage<T>(v)); }
+__device__ __forceinline__ float sigmoid_f(float v) { return 1.0f / (1.0f + expf(-v)); }
+__device__ __forceinline__ float silu_f(float v) { return v / (1.0f + expf(-v)); }
+
+// What becomes of the rows of one range of a stacked projection.
+enum SegKind : int { kSegPlain = 0, kSegSigmoid = 1, kSegSwiGlu = 2 };
+struct DenseSeg {
+    int row0, rows;      // rows of the stack (row0 a multiple of kRowPad)
+    int kind;
+    int ld;              // elements between the results of consecutive tokens
+    float* f;            // kSegPlain, kSegSigmoid: 32-bit results
+    void* t;             // kSegSwiGlu: silu(row 2 i) * row 2 i + 1, in the storage type
+    const float* bias;   // kSegSigmoid: added before the sigmoid
+};
+struct DenseStack {
+    const void* w;       // [rows padded][pitch], storage type
+    int pitch, cols;     // pitch: columns padded to kColPad
+    int n_seg;
+    DenseSeg seg[2];
+};
+
+// ---- reductions ---------------------------------------------------------------------------------------------------------------------
+__device__ __forceinline__ float warp_sum(float v) {
+    for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+    return v;
+}
+__device__ __forceinline__ float block_sum(float v, float* sh) {  // sh: one float per warp
+    v = warp_sum(v);
+    const int w = threadIdx.x >> 5, nw = blockDim.x >> 5;
+    __syncthreads();
+    if ((threadIdx.x & 31) == 0) sh[w] = v;
+    __syncthreads();
+    float t = 0.0f;
+    for (int i = 0; i < nw; ++i) t += sh[i];
+    return t;
+}
+
+// ---- activation vector in shared memory ----------------------------------------------------------------------------------------------
+// 16-bit weights: a lane multiplies eight columns per load; the two halves of an eight lie in two separate arrays so that its 16-byte
+// reads fall on different banks. 32-bit weights: four columns per load, plain order.
+template <typename T> __device__ __forceinline__ int act_index(int e, int pitch);
+template <> __device__ __forceinline__ int act_index<float>(int e, int) { return e; }
+template <> __device__ __forceinline__ int act_index<bf16>(int e, int pitch) { return ((e >> 2) & 1) * (pitch >> 1) + ((e >> 3) << 2) + (e & 3); }
+
+__device__ __forceinline__ uint4 load_stream(const void* p) {
+    uint4 v;
+    asm volatile("ld.global.nc.L1::no_allocate.v4.u32 {%0, %1, %2, %3}, [%4];" : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "l"(p));
+    return v;
+}
+__device__ __forceinline__ float dot_piece(const uint4& w, const float* h, int piece, int pitch, bf16) {
+    const float4 a = *reinterpret_cast<const float4*>(h + piece * 4), b = *reinterpret_cast<const float4*>(h + (pitch >> 1) + piece * 4);
+    float s = __uint_as_float(w.x << 16) * a.x;
+    s = fmaf(__uint_as_float(w.x & 0xffff0000u), a.y, s);
+    s = fmaf(__uint_as_float(w.y << 16), a.z, s);
+    s = fmaf(__uint_as_float(w.y & 0xffff0000u), a.w, s);
+    s = fmaf(__uint_as_float(w.z << 16), b.x, s);
+    s = fmaf(__uint_as_float(w.z & 0xffff0000u), b.y, s);
+    s = fmaf(__uint_as_float(w.w << 16), b.z, s);
+    return fmaf(__uint_as_float(w.w & 0xffff0000u), b.w, s);
+}
+__device__ __forceinline__ float dot_piece(const uint4& w, const float* h, int piece, int, float) {
+    const float4 a = *reinterpret_cast<const float4*>(h + piece * 4);
+    float s = __uint_as_float(w.x) * a.x;
+    s = fmaf(__uint_as_float(w.y), a.y, s);
+    s = fmaf(__uint_as_float(w.z), a.z, s);
+    return fmaf(__uint_as_float(w.w), a.w, s);
+}
+
+// Sums of R consecutive rows over the vector h (shared memory): every lane returns the whole sums.
+template <typename T, int R>
+__device__ __forceinline__ void dot_rows(const T* w, int pitch, const float* h, float (&sum)[R]) {
+    constexpr int kPer = 16 / sizeof(T), U = 4;
+    const int pieces = pitch / kPer, lane = threadIdx.x & 31;
+#pragma unroll
+    for (int r = 0; r < R; ++r) sum[r] = 0.0f;
+    for (int p0 = lane; p0 < pieces; p0 += 32 * U) {
+        uint4 v[R][U];
+#pragma unroll
+        for (int u = 0; u < U; ++u)
+#pragma unroll
+            for (int r = 0; r < R; ++r) v[r][u] = p0 + 32 * u < pieces ? load_stream(w + size_t(r) * pitch + size_t(p0 + 32 * u) * kPer) : make_uint4(0, 0, 0, 0);
+#pragma unroll
+        for (int u = 0; u < U; ++u)
+            if (p0 + 32 * u < pieces) {
+#pragma unroll
+                for (int r = 0; r < R; ++r) sum[r] += dot_piece(v[r][u], h, p0 + 32 * u, pitch, T());
+            }
+    }
+#pragma unroll
+    for (int r = 0; r < R; ++r) sum[r] = warp_sum(sum[r]);
+}
+
+// ---- norms and the projections of their results ----------------------------------------------------------------------------------------
+struct NormProjectArgs {
+    const float* x;             // residual stream, [tokens][width]
+    const float* norm_w[2];     // weights of the two norms
+    float eps;
+    int width, n_stack;         // projections: 1 or 2, each over its own norm of x
+    DenseStack stack[2];
+};
+
+constexpr int kProjectThreads = 256;
+
+template <typename T>
+__global__ void __launch_bounds__(kProjectThreads) norm_project_kernel(NormProjectArgs a) {
+    extern __shared__ float act_smem[];
+    __shared__ float red[kProjectThreads / 32];
+    const int tid = threadIdx.x, token = blockIdx.y, pitch = a.stack[0].pitch;
+    const float* x = a.x + size_t(token) * a.width;
+    float ss = 0.0f;
+    for (int i = tid; i < a.width; i += kProjectThreads) ss += x[i] * x[i];
+    ss = block_sum(ss, red);
+    const float inv = 1.0f / sqrtf(ss / static_cast<float>(a.width) + a.eps);
+    for (int s = 0; s < a.n_stack; ++s)
+        for (int i = tid; i < pitch; i += kProjectThreads)
+            act_smem[s * pitch + act_index<T>(i, pitch)] = i < a.width ? round_to<T>(x[i] * inv * a.norm_w[s][i]) : 0.0f;
+    __syncthreads();
+    const int warps = gridDim.x * (kProjectThreads / 32);
+    int unit = blockIdx.x * (kProjectThreads / 32) + (tid >> 5);
+    for (int s = 0; s < a.n_stack; ++s)
+        for (int k = 0; k < a.stack[s].n_seg; ++k) {
+            const DenseSeg& g = a.stack[s].seg[k];
+            const int units = (g.rows + 1) / 2;
+            for (; unit < units; unit += warps) {
+                const int r = unit * 2;
+                float v[2];  // (an odd last row has a row of padding behind it: row ranges are padded to kRowPad)
+                dot_rows<T, 2>(static_cast<const T*>(a.stack[s].w) + size_t(g.row0 + r) * pitch, pitch, act_smem + s * pitch, v);
+                if ((tid & 31) != 0) continue;
+                if (g.kind == kSegSwiGlu) {
+                    static_cast<T*>(g.t)[size_t(token) * g.ld + unit] = to_storage<T>(silu_f(v[0]) * v[1]);
+                } else {
+                    float* f = g.f + size_t(token) * g.ld + r;
+                    for (int j = 0; j < 2 && r + j < g.rows; ++j) f[j] = g.kind == kSegSigmoid ? sigmoid_f(v[j] + g.bias[r + j]) : v[j];
+                }
+            }
+            unit -= units;
+        }
+}
+
+// ---- output norm of a mixer -----------------------------------------------------------------------------------------------------------
+// y of one token in `parts` equal parts, each divided by its own root mean square, times w[i % w_len]; in place in shared memory, in the
+// order act_index<T>. red: one float per warp.
+template <typename T>
+__device__ __forceinline__ void parts_norm(float* y, int n, int pitch, int parts, float eps, const float* w, int w_len, float* red) {
+    const int len = n / parts, warps = blockDim.x >> 5, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    if (parts >= warps) {  // a warp per part
+        for (int p = warp; p < parts; p += warps) {
+            float ss = 0.0f;
+            for (int i = lane; i < len; i += 32) {
+                const float v = y[act_index<T>(p * len + i, pitch)];
+                ss += v * v;
+            }
+            const float inv = 1.0f / sqrtf(warp_sum(ss) / static_cast<float>(len) + eps);
+            for (int i = lane; i < len; i += 32) {
+                const int e = p * len + i, at = act_index<T>(e, pitch);
+                y[at] = round_to<T>(y[at] * inv * w[e % w_len]);
+            }
+        }
+        __syncthreads();
+        return;
+    }
+    for (int p = 0; p < parts; ++p) {
+        float ss = 0.0f;
+        for (int i = threadIdx.x; i < len; i += blockDim.x) {
+            const float v = y[act_index<T>(p * len + i, pitch)];
+            ss += v * v;
+        }
+        const float inv = 1.0f / sqrtf(block_sum(ss, red) / static_cast<float>(len) + eps);
+        for (int i = threadIdx.x; i < len; i += blockDim.x) {
+            const int e = p * len + i, at = act_index<T>(e, pitch);
+            y[at] = round_to<T>(y[at] * inv * w[e % w_len]);
+        }
+    }
+    __syncthreads();
+}
+
+// ---- output and down projection, gates, residual ------------------------------------------------------------------------------------------
+struct FinishProjectArgs {
+    float* x;                   // residual stream, updated in place: x += (W_o y) * gate1 + (W_down m) * gate2
+    int width;
+    const float* y;             // the mixer's output, 32-bit; normed here when norm_parts > 0
+    int inner;
+    int norm_parts, norm_len;   // norm_len: length of the weight vector (inner, or a head's vdim)
+    const float* norm_w;
+    float eps;
+    const void* o;              // [width][o_pitch]
+    int o_pitch;
+    const void* m;              // feed-forward activations in the storage type, [tokens][down_pitch]; nullptr: no feed-forward
+    const void* down;           // [width][down_pitch]
+    int down_pitch;
+    const float *gate1, *gate2; // sigmoids, [tokens][width]; nullptr: no gate
+};
+
+template <typename T>
+__global__ void __launch_bounds__(kProjectThreads) finish_project_kernel(FinishProjectArgs a) {
+    extern __shared__ float act_smem[];
+    __shared__ float red[kProjectThreads / 32];
+    const int tid = threadIdx.x, lane = tid & 31, token = blockIdx.y;
+    float *y = act_smem, *m = act_smem + a.o_pitch;
+    for (int i = tid; i < a.o_pitch; i += kProjectThreads) {
+        const float v = i < a.inner ? a.y[size_t(token) * a.inner + i] : 0.0f;
+        y[act_index<T>(i, a.o_pitch)] = a.norm_parts > 0 ? v : round_to<T>(v);
+    }
+    if (a.m != nullptr)
+        for (int i = tid; i < a.down_pitch; i += kProjectThreads) m[act_index<T>(i, a.down_pitch)] = from_storage(static_cast<const T*>(a.m)[size_t(token) * a.down_pitch + i]);
+    __syncthreads();
+    if (a.norm_parts > 0) parts_norm<T>(y, a.inner, a.o_pitch, a.norm_parts, a.eps, a.norm_w, a.norm_len, red);
+    const int warps = gridDim.x * (kProjectThreads / 32);
+    for (int row = blockIdx.x * (kProjectThreads / 32) + (tid >> 5); row < a.width; row += warps) {
+        float so[1], sd[1] = {0.0f};
+        dot_rows<T, 1>(static_cast<const T*>(a.o) + size_t(row) * a.o_pitch, a.o_pitch, y, so);
+        if (a.m != nullptr) dot_rows<T, 1>(static_cast<const T*>(a.down) + size_t(row) * a.down_pitch, a.down_pitch, m, sd);
+        if (lane == 0) {
+            const size_t at = size_t(token) * a.width + row;
+            const float g1 = a.gate1 != nullptr ? a.gate1[at] : 1.0f, g2 = a.gate2 != nullptr ? a.gate2[at] : 1.0f;
+            a.x[at] += so[0] * g1 + sd[0] * g2;
+        }
+    }
+}
+
+// ---- batched counterparts of the steps around the projections ------------------------------------------------------------------------------
+// x = embed[token] * scale + pos[position] (pos may be nullptr)
+template <typename T>
+__global__ void embed_scaled_kernel(const T* embed, int pitch, const T* pos_table, const uint32_t* tokens, const uint32_t* pos, SeqIndex seq, float scale, int width, float* x) {
+    const int i = blockIdx.x * blockDim.x + threadIdx.x, t = blockIdx.y;
+    if (i >= width) return;
+    float v = from_storage(embed[size_t(tokens[t]) * pitch + i]) * scale;
+    if (pos_table != nullptr) v += from_storage(pos_table[size_t(seq_position(seq, pos, t)) * width + i]);
+    x[size_t(t) * width + i] = v;
+}
+
+// h_s = RMS norm of x with the weights w_s, in the storage type; rows (optional) picks tokens
+template <typename T>
+__global__ void __launch_bounds__(256) norm_rows_kernel(const float* x, int width, float eps, const float* w0, T* h0, const float* w1, T* h1, int pitch, const uint32_t* rows) {
+    __shared__ float red[8];
+    const int t = blockIdx.x;
+    const float* xr = x + size_t(rows != nullptr ? rows[t] : t) * width;
+    float ss = 0.0f;
+    for (int i = threadIdx.x; i < width; i += blockDim.x) ss += xr[i] * xr[i];
+    const float inv = 1.0f / sqrtf(block_sum(ss, red) / static_cast<float>(width) + eps);
+    for (int i = threadIdx.x; i < width; i += blockDim.x) {
+        const float v = xr[i] * inv;
+        h0[size_t(t) * pitch + i] = to_storage<T>(v * w0[i]);
+        if (h1 != nullptr) h1[size_t(t) * pitch + i] = to_storage<T>(v * w1[i]);
+    }
+}
+
+// The mixer's output norm of many tokens (parts_norm), into the storage type; without a norm a plain conversion.
+template <typename T>
+__global__ void __launch_bounds__(256) finish_rows_kernel(const float* y, int inner, int parts, float eps, const float* w, int w_len, T* out, int pitch) {
+    extern __shared__ float act_smem[];
+    __shared__ float red[8];
+    const int t = blockIdx.x;
+    for (int i = threadIdx.x; i < inner; i += blockDim.x) act_smem[i] = y[size_t(t) * inner + i];
+    __syncthreads();
+    if (parts > 0) parts_norm<float>(act_smem, inner, inner, parts, eps, w, w_len, red);
+    for (int i = threadIdx.x; i < inner; i += blockDim.x) out[size_t(t) * pitch + i] = to_storage<T>(act_smem[i]);
+}
+
+}  // namespace qtb

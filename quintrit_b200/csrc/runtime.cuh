@@ -261,6 +261,36 @@ int rt_feed(quintrit_session* s, const uint32_t* ids, size_t n, uint32_t pos0, b
     return rt_forward(s, ids[n - 1], pos0 + static_cast<uint32_t>(n - 1), want_logits, greedy, false, sample);
 }
 
+// As rt_feed, and the logits at the places `want` (ascending indices into the tokens): [want_n][vocab] floats. A layered model computes them
+// with the tokens they belong to; other models feed the tokens in pieces that end at the places asked for.
+int rt_feed_at(quintrit_session* s, const uint32_t* ids, size_t n, uint32_t pos0, const uint32_t* want, size_t want_n, float* out) {
+    quintrit_b200_decoder* d = s->dec;
+    int rc;
+    if (d->lay && n >= 8) {
+        DeviceGuard g(d->device);
+        if ((rc = layered_prefill(d, ids, n, pos0, nullptr, 0, want, want_n, out)) != QUINTRIT_OK) return rc;
+        QTB_CUDA(cudaMemcpyAsync(s->logits.data(), d->logits, size_t(d->vocab) * sizeof(float), cudaMemcpyDeviceToHost, d->stream));
+        if ((rc = decoder_check_status(d)) != QUINTRIT_OK) return rc;
+        if (s->cached.size() >= pos0) {
+            s->cached.resize(pos0);
+            s->cached.insert(s->cached.end(), ids, ids + n);
+        } else {
+            s->cached.clear();
+        }
+        d->host_pos = pos0 + static_cast<uint32_t>(n);
+        s->logits_valid = true;
+        return QUINTRIT_OK;
+    }
+    size_t from = 0;
+    for (size_t i = 0; i <= want_n; ++i) {
+        const size_t to = i < want_n ? size_t(want[i]) + 1 : n;
+        if (to > from && (rc = rt_feed(s, ids + from, to - from, pos0 + static_cast<uint32_t>(from), true, nullptr)) != QUINTRIT_OK) return rc;
+        from = to;
+        if (i < want_n) std::copy(s->logits.begin(), s->logits.end(), out + i * s->logits.size());
+    }
+    return QUINTRIT_OK;
+}
+
 // engine.rs:869-879: the first index of `pending` from which the rest could still be the beginning of a stop sequence.
 size_t rt_safe_flush(const std::string& pending, const std::vector<std::string>& stops) {
     for (size_t idx = 0; idx < pending.size(); ++idx) {
@@ -345,15 +375,16 @@ std::string rt_build_tokenizer(const GgufFile& g, qtb::BpeTokenizer* tok) {
 }
 
 int rt_open_gpu(const char* path, const quintrit_gpu_options_t* options, quintrit_model** out) {
-    uint32_t device = 0, want_ctx = 0;
+    uint32_t device = 0, want_ctx = 0, flags = 0;
     if (options != nullptr) {
         int rc = rt_struct(options, "options");
         if (rc != QUINTRIT_OK) return rc;
-        if (options->flags & ~uint32_t(QUINTRIT_MODEL_OPEN_VERBOSE)) return fail(QUINTRIT_ERR_INVALID_ARGUMENT, "options.flags has unknown bits set: 0x%x", options->flags);
+        if (options->flags & ~uint32_t(QUINTRIT_MODEL_OPEN_VERBOSE | QUINTRIT_B200_OPEN_FLOAT32)) return fail(QUINTRIT_ERR_INVALID_ARGUMENT, "options.flags has unknown bits set: 0x%x", options->flags);
+        flags = options->flags;
         device = options->device_index, want_ctx = options->context_length;  // the library never prints: VERBOSE changes nothing
     }
     auto inner = std::make_shared<RtModelInner>();
-    int rc = load_gguf_model(path, device, &inner->data);
+    int rc = load_model(path, device, flags, &inner->data);
     if (rc != QUINTRIT_OK) return rc;
     const GgufFile& g = inner->data.file;
     const GgufModelShape& m = inner->data.shape;
@@ -363,7 +394,8 @@ int rt_open_gpu(const char* path, const quintrit_gpu_options_t* options, quintri
         std::string name = meta_str(g, "general.name", ""), base = meta_str(g, "general.basename", "");
         for (char& c : name) c = static_cast<char>(std::tolower(static_cast<unsigned char>(c)));
         for (char& c : base) c = static_cast<char>(std::tolower(static_cast<unsigned char>(c)));
-        inner->arch = m.arch_id == QUINTRIT_B200_ARCH_BITNET ? "bitnet"
+        inner->arch = inner->data.layered ? m.arch
+                      : m.arch_id == QUINTRIT_B200_ARCH_BITNET ? "bitnet"
                       : m.arch == "qwen3" ? "qwen3"
                       : (m.arch == "falcon3" || name.find("falcon") != std::string::npos || base.find("falcon") != std::string::npos) ? "falcon3" : "llama";
     }
@@ -905,7 +937,7 @@ extern "C" int quintrit_session_create(const quintrit_model_t* model, const quin
         uint32_t ctx = options != nullptr ? options->context_length : 0;
         if (ctx == 0) ctx = m->max_ctx;
         if (ctx > m->max_ctx) return fail(QUINTRIT_ERR_INVALID_ARGUMENT, "context_length %u exceeds the GPU context of the model (%u)", ctx, m->max_ctx);
-        ctx = ctx >= 256 ? ctx / 256 * 256 : ctx;
+        if (!m->data.layered) ctx = ctx >= 256 ? ctx / 256 * 256 : ctx;
         std::unique_ptr<quintrit_session> s(new quintrit_session());
         {
             std::lock_guard<std::mutex> hold(m->lock);
@@ -987,6 +1019,8 @@ int rt_generate(quintrit_session* s, const std::string& prompt, const quintrit_g
     size_t common = 0;
     if (!keep && s->cached.size() == s->dec->host_pos && std::getenv("QUINTRIT_B200_NO_PREFIX_REUSE") == nullptr)
         while (common < s->cached.size() && common + 1 < tokens.size() && s->cached[common] == tokens[common]) ++common;
+    // A layered model's recurrent state stands at the end of what is cached: it can be continued there, not at an earlier difference.
+    if (s->dec->lay && common != s->cached.size()) common = 0;
     s->last_reused = static_cast<uint32_t>(common);
     const uint32_t pos0 = keep ? base : static_cast<uint32_t>(common);
     if (!keep) {
@@ -1147,6 +1181,28 @@ extern "C" int quintrit_session_feed_tokens(quintrit_session_t* session, const u
         if (size_t(pos0) + count > session->ctx) return fail(QUINTRIT_ERR_CONTEXT_OVERFLOW, "%zu tokens do not fit: the context window holds %u tokens and %u are already used", count, session->ctx, pos0);
         if (pos0 == 0) session->dec->host_pos = 0;
         if ((rc = rt_feed(session, tokens, count, pos0, true, nullptr)) != QUINTRIT_OK) return rc;
+        return ok();
+    });
+}
+extern "C" int quintrit_b200_session_feed_at(quintrit_session_t* session, const uint32_t* tokens, size_t count, uint32_t flags, const uint32_t* want, size_t want_count, float* out,
+                                             size_t capacity) {
+    return guard([&]() -> int {
+        int rc = rt_check(session, kMagicSession, "session");
+        if (rc != QUINTRIT_OK) return rc;
+        if (tokens == nullptr || (want_count != 0 && (want == nullptr || out == nullptr))) return fail(QUINTRIT_ERR_NULL_POINTER, "a buffer is NULL");
+        if (count == 0) return fail(QUINTRIT_ERR_INVALID_ARGUMENT, "no tokens to feed");
+        if (flags & ~uint32_t(QUINTRIT_GENERATE_KEEP_CONTEXT)) return fail(QUINTRIT_ERR_INVALID_ARGUMENT, "unknown flags 0x%x", flags);
+        for (size_t i = 0; i < want_count; ++i)
+            if (want[i] >= count || (i > 0 && want[i] <= want[i - 1])) return fail(QUINTRIT_ERR_INVALID_ARGUMENT, "want[%zu] = %u is not an ascending index below %zu", i, want[i], count);
+        RtSessionLock lk(session);
+        if ((rc = lk.check()) != QUINTRIT_OK) return rc;
+        if (capacity / session->logits.size() < want_count) return fail(QUINTRIT_ERR_BUFFER_TOO_SMALL, "out holds %zu values, %zu rows of %zu are needed", capacity, want_count, session->logits.size());
+        const uint32_t pos0 = (flags & QUINTRIT_GENERATE_KEEP_CONTEXT) ? session->dec->host_pos : 0;
+        for (size_t i = 0; i < count; ++i)
+            if (tokens[i] >= static_cast<uint32_t>(session->dec->vocab_full)) return fail(QUINTRIT_ERR_INVALID_ARGUMENT, "token id %u is outside the vocabulary of %d", tokens[i], session->dec->vocab_full);
+        if (size_t(pos0) + count > session->ctx) return fail(QUINTRIT_ERR_CONTEXT_OVERFLOW, "%zu tokens do not fit: the context window holds %u tokens and %u are already used", count, session->ctx, pos0);
+        if (pos0 == 0) session->dec->host_pos = 0;
+        if ((rc = rt_feed_at(session, tokens, count, pos0, want, want_count, out)) != QUINTRIT_OK) return rc;
         return ok();
     });
 }

@@ -17,6 +17,7 @@ import numpy as np
 from .api import QuintritError, _check, load_library
 
 _sz = C.c_size_t
+_OPEN_FLOAT32 = 0x100
 FINISH = {0: "length", 1: "eos", 2: "stop", 3: "callback", 4: "context"}
 
 
@@ -107,6 +108,7 @@ def _lib() -> C.CDLL:
     l.quintrit_session_generate.argtypes = [vp, C.c_char_p, _sz, C.POINTER(_GenerateParams), TOKEN_CALLBACK, vp, C.c_char_p, _sz, C.POINTER(_sz),
                                             C.POINTER(_GenerateResult)]
     l.quintrit_session_feed_tokens.argtypes = [vp, u32p, _sz, C.c_uint32]
+    l.quintrit_b200_session_feed_at.argtypes = [vp, u32p, _sz, C.c_uint32, u32p, _sz, C.POINTER(C.c_float), _sz]
     l.quintrit_session_logits.argtypes = [vp, C.POINTER(C.c_float), _sz]
     l.quintrit_session_generate_tokens.argtypes = [vp, u32p, _sz, _sz, u32p, _sz, C.POINTER(_sz)]
     l.quintrit_b200_tokenizer_open.argtypes = [C.c_char_p, C.POINTER(vp)]
@@ -223,6 +225,53 @@ class TokenStream:
         return self._pieces.pop(0)
 
 
+class Session:
+    """One conversation of a model: its cache and state on the device, driven by token ids (quintrit_session_create, _feed_tokens).
+    A model has one of its own; ``Model.new_session`` makes more, over the same weights."""
+
+    def __init__(self, model: "Model", context: int | None = None):
+        self._l, self.model = model._l, model  # (the model's weights outlive its handle as long as a session exists)
+        self._s = C.c_void_p()
+        opts = _SessionOptions(struct_size=C.sizeof(_SessionOptions), context_length=context or 0)
+        _check(self._l.quintrit_session_create(model._h, C.byref(opts), C.byref(self._s)))
+
+    @property
+    def position(self) -> int:
+        si = _SessionInfo(struct_size=C.sizeof(_SessionInfo))
+        _check(self._l.quintrit_session_info(self._s, C.byref(si)))
+        return si.position
+
+    def reset(self) -> None:
+        _check(self._l.quintrit_session_reset(self._s))
+
+    def feed(self, ids, want=(), keep_context: bool = True) -> np.ndarray:
+        """Feeds token ids after those already held (``keep_context=False``: from position 0) and returns the logits at the places
+        ``want`` (ascending indices into ``ids``) as [len(want), vocab]."""
+        a, w = _ids(ids), _ids(want)
+        out = np.zeros((w.size, self.model.vocab_size), np.float32)
+        _check(self._l.quintrit_b200_session_feed_at(self._s, _u32p(a), a.size, 1 if keep_context else 0, _u32p(w), w.size,
+                                                     out.ctypes.data_as(C.POINTER(C.c_float)), out.size))
+        return out
+
+    def generate_tokens(self, prompt_ids, max_new: int) -> np.ndarray:
+        """Greedy tokens after the prompt, from position 0, without leaving the device between them."""
+        a = _ids(prompt_ids)
+        out, n = np.zeros(max_new, np.uint32), _sz(0)
+        _check(self._l.quintrit_session_generate_tokens(self._s, _u32p(a), a.size, max_new, _u32p(out), out.size, C.byref(n)))
+        return out[:n.value]
+
+    def close(self) -> None:
+        if self._s.value is not None:
+            self._l.quintrit_session_free(self._s)
+            self._s = C.c_void_p()
+
+    def __del__(self):
+        try:
+            self.close()
+        except Exception:
+            pass
+
+
 class Model:
     """A model on a B200 with one session (quintrit_model_open_gpu + quintrit_session_create)."""
 
@@ -241,7 +290,11 @@ class Model:
         self.tokenizer = Tokenizer(_model=self)
 
     @staticmethod
-    def load(path, *, device: str = "cuda", context: int | None = None, verbose: bool = False) -> "Model":
+    def load(path, *, device: str = "cuda", context: int | None = None, verbose: bool = False, dtype: str | None = None) -> "Model":
+        """``path``: a GGUF file or a model folder. ``dtype``: "float32" opens a folder in 32-bit arithmetic; the default serves it in
+        bfloat16 (a GGUF file has the arithmetic of its encoding)."""
+        if dtype not in (None, "bfloat16", "float32"):
+            raise QuintritError(2, f"dtype {dtype!r} is neither 'bfloat16' nor 'float32'")
         if device == "cuda":
             index = 0
         elif device.startswith("cuda:") and device[5:].isdigit():
@@ -249,10 +302,13 @@ class Model:
         else:
             raise QuintritError(2, f"device {device!r} is not 'cuda' or 'cuda:N' (this library has no CPU engine)")
         l = _lib()
-        opts = _GpuOptions(struct_size=C.sizeof(_GpuOptions), device_index=index, context_length=context or 0, flags=1 if verbose else 0)
+        opts = _GpuOptions(struct_size=C.sizeof(_GpuOptions), device_index=index, context_length=context or 0, flags=(1 if verbose else 0) | (_OPEN_FLOAT32 if dtype == "float32" else 0))
         h = C.c_void_p()
         _check(l.quintrit_model_open_gpu(os.fsencode(str(path)), C.byref(opts), C.byref(h)))
         return Model(h, l, path)
+
+    def new_session(self, context: int | None = None) -> Session:
+        return Session(self, context)
 
     architecture = property(lambda self: self._info.architecture.decode())
     vocab_size = property(lambda self: self._info.vocab_size)
