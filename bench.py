@@ -455,6 +455,81 @@ def run_block_scaled_decode(args, local_rank: int):
     return out
 
 
+# Layered models of random weights at the widths of real models: a third of the layers each mamba2 (inner 2 x width, heads of 64, state 128),
+# hgrn2 (heads of 128 x 128) and attention (heads of 128, four query heads per KV head, window 2048, blocks of 32).
+LAYERED_SIZES = {"1k": (1024, 2816, 12), "2k": (2048, 5632, 12), "4k": (4096, 11264, 6)}
+
+
+def layered_config(size: str, layers=None, positions: int = 8192):
+    from quintrit_b200 import model_folder as mf
+
+    W, ff, L = LAYERED_SIZES[size]
+    kinds = [lambda: mf.mamba2(W // 32, 64, 128, groups=8, conv=4, norm_groups=8, ff=ff), lambda: mf.hgrn2(W // 128, 128, 128, ff=ff),
+             lambda: mf.attention(W // 128, W // 512, 128, 128, 2048, 32, ff=ff)]
+    return mf.lasosun_config([kinds[i % 3]() for i in range(layers or L)], W, 32768, positions)
+
+
+def run_layered(args, local_rank: int):
+    """Prompt ingestion and decoding of layered models (Lasosun) beside a ternary LLaMA-form model of the same width, feed-forward, layer count and
+    vocabulary: tokens/s of a 4096-token prompt (wall clock around the call that ends with the logits on the host, best of three), and device
+    time of a decode step at that context. Fractions are of the measured HBM rate (bytes of the weights a step reads) and of the measured dense
+    bf16 rate (multiply-adds of the projections)."""
+    import shutil
+    import tempfile
+
+    import torch
+
+    import quintrit_b200 as q
+    from quintrit_b200 import model_folder as mf
+
+    hbm, tensor = measured_peaks()[0], 1590.0
+    try:
+        tensor = float(json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json")))["bf16_tflops"])
+    except Exception:  # the fallback rate of a dense bf16 product
+        pass
+    out = []
+    for size in args.layered_sizes.split(","):
+        cfg = layered_config(size, args.decode_layers)
+        W, ff = cfg["width"], cfg["layers"][0]["mlp"]["ff"]
+        shapes = mf.lasosun_shapes(cfg)
+        matrix = sum(int(np.prod(s)) for n, s in shapes.items() if len(s) == 2 and n not in ("embed", "pos") and not n.endswith("conv"))
+        head = cfg["vocab"] * W
+        tmp = tempfile.mkdtemp()
+        try:
+            mf.write_folder(tmp, cfg, mf.random_lasosun(cfg, 5))
+            dec = q.Decoder.open(tmp, device=local_rank)
+        finally:
+            shutil.rmtree(tmp)
+        prompt = synth.prompt_tokens(6, args.layered_prompt, cfg["vocab"])
+
+        def ingest(dec):
+            best = 1e9
+            for _ in range(4):
+                t0 = time.perf_counter()
+                dec.prefill(prompt)
+                best = min(best, time.perf_counter() - t0)
+            return best
+
+        def row(dec, weight_bytes, macs):
+            t = ingest(dec)
+            ms = dec.time_token(5, max(args.steps, 20))
+            return {"prefill_tokens_per_s": round(len(prompt) / t), "prefill_ms": round(t * 1e3, 2), "prefill_frac_of_bf16": round(2 * macs * len(prompt) / t / tensor / 1e12, 3),
+                    "decode_ms": round(ms, 4), "decode_tokens_per_s": round(1e3 / ms, 1), "weight_bytes": int(weight_bytes), "decode_frac_of_hbm": round(weight_bytes / (ms * 1e-3) / hbm / 1e9, 3)}
+
+        r = {"size": size, "width": W, "ff": ff, "layers": len(cfg["layers"]), "prompt": len(prompt), "lasosun_bf16": row(dec, 2 * (matrix + head), matrix)}
+        dec.free()
+        if not args.no_decode:  # the ternary model
+            dims = dict(hidden=W, inter=ff, layers=len(cfg["layers"]), q_heads=W // 128, kv_heads=W // 512, head_dim=128, vocab=cfg["vocab"])
+            spec = synth.torch_model(dims, torch.device("cuda", local_rank), min(8192, len(prompt) + 256))
+            torch.cuda.empty_cache()
+            dec = q.Decoder(spec, device=local_rank)
+            tern = dims["layers"] * (2 * W * W + 2 * W * W // 4 + 3 * W * ff)
+            r["ternary_llama"] = row(dec, tern * BYTES_PER_WEIGHT + 2 * head, tern)
+            dec.free()
+        out.append(r)
+    return out
+
+
 def run_moe(args, local_rank: int):
     """One mixture-of-experts feed-forward block of the Qwen3-30B-A3B shape (hidden 2048, 128 experts of width 768, top-8 softmax routing,
     BF16 router, ternary experts) for a batch of 16 tokens on one GPU: device time of the block's launches, the time of the C call with host
@@ -956,6 +1031,9 @@ def main():
     ap.add_argument("--block-scaled-decode", action="store_true", help="run only a whole-token decode of a block-scaled (Q2_0) model of the decode shape (profiling aid)")
     ap.add_argument("--decode-shape", default="falcon3_10b", choices=["falcon3_10b", "bitnet_2b"])
     ap.add_argument("--decode-layers", type=int, default=None, help="fewer layers than the shape has (experiments)")
+    ap.add_argument("--layered-model", action="store_true", help="run only prompt ingestion and decoding of layered models (Lasosun) beside a ternary model of equal size")
+    ap.add_argument("--layered-sizes", default="1k,2k,4k", help="with --layered-model: which of %s" % ", ".join(LAYERED_SIZES))
+    ap.add_argument("--layered-prompt", type=int, default=4096, help="with --layered-model: prompt tokens")
     ap.add_argument("--moe-only", action="store_true", help="run only the mixture-of-experts block leg and print its object")
     ap.add_argument("--no-moe", action="store_true", help="skip the mixture-of-experts block leg")
     ap.add_argument("--batch-seqs", type=int, default=32, help="sequences of the batched-decode leg (0 skips it)")
@@ -989,6 +1067,9 @@ def main():
         return
     if args.block_scaled_decode:
         print(json.dumps({"block_scaled_decode": run_block_scaled_decode(args, local_rank)}), flush=True)
+        return
+    if args.layered_model:
+        print(json.dumps({"layered_model": run_layered(args, local_rank)}), flush=True)
         return
     if args.moe_only:
         print(json.dumps({"moe": run_moe(args, local_rank)}), flush=True)

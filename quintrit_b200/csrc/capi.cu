@@ -2961,8 +2961,8 @@ int batch_head(quintrit_b200_batch* b, int n) {
     quintrit_b200_decoder* d = b->d;
     cudaStream_t s = d->stream;
     if (d->lay) {
-        for (int t = 0; t < n; t += kDenseN) {
-            const int here = std::min(n - t, kDenseN);
+        for (int t = 0; t < n; t += kDenseBox) {
+            const int here = std::min(n - t, kDenseBox);
             const int rc = layered_logits_rows(d, t, here, b->logits + size_t(t) * d->vocab);
             if (rc != QUINTRIT_OK) return rc;
         }

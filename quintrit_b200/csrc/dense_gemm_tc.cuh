@@ -1,10 +1,11 @@
 // Dense projections of many tokens: out[t][r] = sum_k W[r][k] * h[t][k], with the endings of dense_gemv.cuh.
 //
-// 16-bit weights run on the 5th-generation tensor cores. A block makes one tile of 128 weight rows (the M of the instruction) x 128 tokens
-// (the N): one thread fetches 64-column slices of both operands with TMA (128-byte swizzle) into a ring of stages, one thread issues
-// tcgen05.mma.kind::f16 (bf16 operands, 32-bit sums in tensor memory), four warps read the sums with tcgen05.ld - a weight row per lane, so
-// that the 32 lanes of a warp write 32 neighbouring results of a token - and apply the ending. Two blocks share a multiprocessor: one's
-// ending overlaps the other's products. The grid runs over token tiles first, so the blocks that are resident together share weight rows.
+// 16-bit weights run on the 5th-generation tensor cores. A tile is 128 weight rows (the M of the instruction) x 128 or 256 tokens (the N):
+// one thread fetches 64-column slices of both operands with TMA (128-byte swizzle) into a ring of stages, one thread issues
+// tcgen05.mma.kind::f16 (bf16 operands, 32-bit sums in tensor memory), eight warps read the sums with tcgen05.ld - a weight row per lane, so
+// that the 32 lanes of a warp write 32 neighbouring results of a token - and apply the ending. One block per multiprocessor takes tiles in
+// turn; two sets of accumulators let the ending of a tile overlap the products of the next. Tiles run over the tokens first, so the blocks
+// that are at work together share weight rows.
 //
 // The dual form makes two products of one tile, W_o y and W_down m, in two accumulators and ends with both gates and the residual sum.
 // Every wait is bounded, as in gemm_tc.cuh, whose mbarrier, descriptor and status conventions are used here.
@@ -18,11 +19,12 @@
 
 namespace qtb {
 
-constexpr int kDenseM = 128, kDenseN = 128, kDenseK = 64;
-constexpr int kDenseStages = 3;
-constexpr int kDenseStageBytes = (kDenseM + kDenseN) * kDenseK * 2;
-constexpr int kDenseSmem = kDenseStages * kDenseStageBytes + 1024 + 256;
-constexpr int kDenseThreads = 192;  // TMA warp, MMA warp, four warps for the ending
+constexpr int kDenseM = 128, kDenseBox = 128, kDenseK = 64;  // kDenseBox: rows of an activation box; a tile's N is a multiple of it
+constexpr int kDenseEndWarps = 8;
+constexpr int kDenseThreads = 64 + 32 * kDenseEndWarps;  // TMA warp, MMA warp, warps for the ending
+__host__ __device__ constexpr int dense_stages(int n) { return n > 128 ? 4 : 6; }
+__host__ __device__ constexpr int dense_stage_bytes(int n) { return (kDenseM + n) * kDenseK * 2; }
+__host__ __device__ constexpr int dense_smem(int n) { return dense_stages(n) * dense_stage_bytes(n) + 1024 + 256; }
 
 struct DenseGemmArgs {
     int tokens;
@@ -73,40 +75,49 @@ __device__ __forceinline__ void tmem_load16(uint32_t taddr, uint32_t (&v)[16]) {
 }
 }  // namespace dense_detail
 
-template <bool DUAL>
-__global__ void __launch_bounds__(kDenseThreads) dense_gemm_tc_kernel(const __grid_constant__ CUtensorMap w0, const __grid_constant__ CUtensorMap h0, const __grid_constant__ CUtensorMap w1,
-                                                                      const __grid_constant__ CUtensorMap h1, const __grid_constant__ DenseGemmArgs a) {
+template <int N, bool DUAL>
+__global__ void __launch_bounds__(kDenseThreads, 1) dense_gemm_tc_kernel(const __grid_constant__ CUtensorMap w0, const __grid_constant__ CUtensorMap h0, const __grid_constant__ CUtensorMap w1,
+                                                                         const __grid_constant__ CUtensorMap h1, const __grid_constant__ DenseGemmArgs a) {
     using namespace gemm_detail;
     using namespace dense_detail;
     extern __shared__ unsigned char dense_smem_raw[];
     unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(dense_smem_raw) + 1023) & ~uintptr_t(1023));
-    constexpr int S = kDenseStages;
-    uint64_t* bars = reinterpret_cast<uint64_t*>(smem + S * kDenseStageBytes);
+    constexpr int S = dense_stages(N), kStage = dense_stage_bytes(N), kAcc = DUAL ? 2 * N : N;  // kAcc: tensor-memory columns of a tile
+    static_assert(2 * kAcc <= 512, "two sets of accumulators fit tensor memory");
+    uint64_t* bars = reinterpret_cast<uint64_t*>(smem + S * kStage);
     const uint32_t bar0 = smem_u32(bars), tiles0 = smem_u32(smem);
     auto loaded = [&](int s) { return bar0 + 8u * s; };
     auto empty = [&](int s) { return bar0 + 8u * (S + s); };
-    const uint32_t acc_full = bar0 + 8u * (2 * S);
-    volatile uint32_t* tmem_slot = reinterpret_cast<volatile uint32_t*>(bars + 2 * S + 1);
-    volatile unsigned int* abort_flag = reinterpret_cast<volatile unsigned int*>(bars + 2 * S + 2);
+    auto acc_full = [&](int i) { return bar0 + 8u * (2 * S + i); };
+    auto acc_empty = [&](int i) { return bar0 + 8u * (2 * S + 2 + i); };
+    volatile uint32_t* tmem_slot = reinterpret_cast<volatile uint32_t*>(bars + 2 * S + 4);
+    volatile unsigned int* abort_flag = reinterpret_cast<volatile unsigned int*>(bars + 2 * S + 5);
 
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const int token0 = blockIdx.x * kDenseN;
-    const int prob = !DUAL && static_cast<int>(blockIdx.y) >= a.row_tiles[0] ? 1 : 0;
-    const int row0 = (static_cast<int>(blockIdx.y) - (prob ? a.row_tiles[0] : 0)) * kDenseM;
-    const int steps0 = a.k_steps[prob], steps = DUAL ? steps0 + a.k_steps[1] : steps0;
-    constexpr uint32_t tmem_cols = DUAL ? 2 * kDenseN : kDenseN;
+    const int token_tiles = (a.tokens + N - 1) / N;
+    const int items = token_tiles * (a.row_tiles[0] + (!DUAL && a.n_prob > 1 ? a.row_tiles[1] : 0));
+    // tile `item`: its problem, first row and first token
+    auto locate = [&](int item, int* prob, int* row0, int* token0) {
+        const int tile = item / token_tiles;
+        *prob = !DUAL && tile >= a.row_tiles[0] ? 1 : 0;
+        *row0 = (tile - (*prob ? a.row_tiles[0] : 0)) * kDenseM;
+        *token0 = (item % token_tiles) * N;
+    };
 
     if (tid == 0) {
         for (int s = 0; s < S; ++s) {
             mbar_init(loaded(s), 1);
             mbar_init(empty(s), 1);
         }
-        mbar_init(acc_full, 1);
+        for (int i = 0; i < 2; ++i) {
+            mbar_init(acc_full(i), 1);
+            mbar_init(acc_empty(i), kDenseEndWarps);
+        }
         *abort_flag = 0;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
     if (warp == 0) {
-        asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(const_cast<uint32_t*>(tmem_slot))), "r"(tmem_cols) : "memory");
+        asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(const_cast<uint32_t*>(tmem_slot))), "r"(512u) : "memory");
         asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
     }
     asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
@@ -118,15 +129,23 @@ __global__ void __launch_bounds__(kDenseThreads) dense_gemm_tc_kernel(const __gr
         if (lane == 0) {
             int it = 0, s = 0;
             uint32_t ph = 0;
-            for (; it < steps; ++it) {
-                if (!mbar_wait(empty(s), ph ^ 1, abort_flag, a.spin_limit)) break;
-                const bool second = DUAL ? it >= steps0 : prob != 0;
-                const int k = (DUAL && second ? it - steps0 : it) * kDenseK;
-                const uint32_t dst = tiles0 + s * kDenseStageBytes;
-                mbar_expect_tx(loaded(s), kDenseStageBytes);
-                tma_load_2d(dst, second ? &w1 : &w0, k, row0, loaded(s));
-                tma_load_2d(dst + kDenseM * kDenseK * 2, second ? &h1 : &h0, k, token0, loaded(s));
-                if (++s == S) s = 0, ph ^= 1;
+            bool okay = true;
+            for (int item = blockIdx.x; item < items && okay; item += gridDim.x) {
+                int prob, row0, token0;
+                locate(item, &prob, &row0, &token0);
+                const int steps0 = a.k_steps[prob], steps = DUAL ? steps0 + a.k_steps[1] : steps0;
+                for (int k = 0; k < steps; ++k, ++it) {
+                    if (!(okay = mbar_wait(empty(s), ph ^ 1, abort_flag, a.spin_limit))) break;
+                    const bool second = DUAL ? k >= steps0 : prob != 0;
+                    const int x = (DUAL && second ? k - steps0 : k) * kDenseK;
+                    const uint32_t dst = tiles0 + s * kStage;
+                    mbar_expect_tx(loaded(s), kStage);
+                    tma_load_2d(dst, second ? &w1 : &w0, x, row0, loaded(s));
+#pragma unroll
+                    for (int b = 0; b < N / kDenseBox; ++b)
+                        tma_load_2d(dst + (kDenseM + b * kDenseBox) * kDenseK * 2, second ? &h1 : &h0, x, token0 + b * kDenseBox, loaded(s));
+                    if (++s == S) s = 0, ph ^= 1;
+                }
             }
             for (int back = 0; back < min(it, S); ++back) {  // its copies in flight land before the block leaves
                 if (--s < 0) s = S - 1, ph ^= 1;
@@ -135,60 +154,75 @@ __global__ void __launch_bounds__(kDenseThreads) dense_gemm_tc_kernel(const __gr
         }
     } else if (warp == 1) {
         if (lane == 0) {
-            const uint32_t idesc = instr_desc_bf16(kDenseM, kDenseN);
-            int s = 0;
+            const uint32_t idesc = instr_desc_bf16(kDenseM, N);
+            int s = 0, j = 0;
             uint32_t ph = 0;
-            for (int it = 0; it < steps; ++it) {
-                if (!mbar_wait(loaded(s), ph, abort_flag, a.spin_limit)) break;
+            bool okay = true;
+            for (int item = blockIdx.x; item < items && okay; item += gridDim.x, ++j) {
+                int prob, row0, token0;
+                locate(item, &prob, &row0, &token0);
+                const int steps0 = a.k_steps[prob], steps = DUAL ? steps0 + a.k_steps[1] : steps0;
+                const int set = j & 1;
+                if (!(okay = mbar_wait(acc_empty(set), ((j >> 1) & 1) ^ 1, abort_flag, a.spin_limit))) break;
                 asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-                const bool second = DUAL && it >= steps0;
-                const uint32_t at = tiles0 + s * kDenseStageBytes;
-                const uint64_t da = smem_desc(at, 16, 1024, 2), db = smem_desc(at + kDenseM * kDenseK * 2, 16, 1024, 2);  // 128-byte swizzle, 8-row groups 1024 bytes apart
-                const uint32_t acc = tmem_base + (second ? kDenseN : 0);
-                const bool first = it == 0 || (DUAL && it == steps0);
+                for (int k = 0; k < steps; ++k) {
+                    if (!(okay = mbar_wait(loaded(s), ph, abort_flag, a.spin_limit))) break;
+                    asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+                    const uint32_t at = tiles0 + s * kStage;
+                    const uint64_t da = smem_desc(at, 16, 1024, 2), db = smem_desc(at + kDenseM * kDenseK * 2, 16, 1024, 2);  // 128-byte swizzle, 8-row groups 1024 bytes apart
+                    const uint32_t acc = tmem_base + set * kAcc + (DUAL && k >= steps0 ? N : 0);
+                    const bool first = k == 0 || (DUAL && k == steps0);
 #pragma unroll
-                for (int j = 0; j < kDenseK / 16; ++j) mma_bf16(acc, da + 2 * j, db + 2 * j, idesc, first && j == 0 ? 0u : 1u);
-                mma_commit(empty(s));
-                if (++s == S) s = 0, ph ^= 1;
+                    for (int q = 0; q < kDenseK / 16; ++q) mma_bf16(acc, da + 2 * q, db + 2 * q, idesc, first && q == 0 ? 0u : 1u);
+                    mma_commit(empty(s));
+                    if (++s == S) s = 0, ph ^= 1;
+                }
+                mma_commit(acc_full(set));  // (also on the way out after a failed wait)
             }
-            mma_commit(acc_full);
         }
     } else {
-        const int r = (warp & 3) * 32 + lane;  // a warp reads the 32 lanes of tensor memory that its index modulo 4 selects
-        bool okay = true;
-        if (lane == 0) okay = mbar_wait(acc_full, 0, abort_flag, a.spin_limit);
-        okay = __shfl_sync(0xffffffffu, okay ? 1 : 0, 0) != 0 && *abort_flag == 0;
-        okay = __all_sync(0xffffffffu, okay);
-        if (okay) {
+        // the ending: a warp reads the 32 lanes of tensor memory that its index modulo 4 selects; the two warps of a quarter take 16-column pieces in turn
+        const int r = (warp & 3) * 32 + lane, turn = (warp - 2) >> 2;
+        int j = 0;
+        for (int item = blockIdx.x; item < items; item += gridDim.x, ++j) {
+            int prob, row0, token0;
+            locate(item, &prob, &row0, &token0);
+            const int set = j & 1;
+            bool okay = true;
+            if (lane == 0) okay = mbar_wait(acc_full(set), (j >> 1) & 1, abort_flag, a.spin_limit) && *abort_flag == 0;
+            okay = __shfl_sync(0xffffffffu, okay ? 1 : 0, 0) != 0;
+            if (!okay) break;
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-            const uint32_t lane_base = tmem_base + (uint32_t((warp & 3) * 32) << 16);
-            const int n_here = min(kDenseN, a.tokens - token0);
+            const uint32_t acc = tmem_base + (uint32_t((warp & 3) * 32) << 16) + set * kAcc;
+            const int n_here = min(N, a.tokens - token0);
             if constexpr (DUAL) {
                 const int row = row0 + r;
                 const bool has2 = a.k_steps[1] > 0;
-                for (int c0 = 0; c0 < n_here; c0 += 16) {
+                for (int c0 = turn * 16; c0 < n_here; c0 += 32) {
                     uint32_t v1[16], v2[16];
-                    tmem_load16(lane_base + c0, v1);
-                    if (has2) tmem_load16(lane_base + kDenseN + c0, v2);
+                    tmem_load16(acc + c0, v1);
+                    if (has2) tmem_load16(acc + N + c0, v2);
                     asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
                     if (row < a.width) {
+                        float add[16], x[16];
+#pragma unroll
+                        for (int i = 0; i < 16; ++i) {
+                            const size_t at = size_t(token0 + min(c0 + i, n_here - 1)) * a.width + row;
+                            add[i] = __uint_as_float(v1[i]) * (a.gate1 != nullptr ? a.gate1[at] : 1.0f);
+                            if (has2) add[i] += __uint_as_float(v2[i]) * (a.gate2 != nullptr ? a.gate2[at] : 1.0f);
+                            x[i] = a.x[at];
+                        }
 #pragma unroll
                         for (int i = 0; i < 16; ++i)
-                            if (c0 + i < n_here) {
-                                const size_t at = size_t(token0 + c0 + i) * a.width + row;
-                                float add = __uint_as_float(v1[i]);
-                                if (a.gate1 != nullptr) add *= a.gate1[at];
-                                if (has2) add += __uint_as_float(v2[i]) * (a.gate2 != nullptr ? a.gate2[at] : 1.0f);
-                                a.x[at] += add;
-                            }
+                            if (c0 + i < n_here) a.x[size_t(token0 + c0 + i) * a.width + row] = x[i] + add[i];
                     }
                 }
             } else {
                 const DenseStack& st = a.stack[prob];
                 const DenseSeg& g = st.seg[st.n_seg > 1 && row0 >= st.seg[1].row0 ? 1 : 0];
-                for (int c0 = 0; c0 < n_here; c0 += 16) {
+                for (int c0 = turn * 16; c0 < n_here; c0 += 32) {
                     uint32_t v[16];
-                    tmem_load16(lane_base + c0, v);
+                    tmem_load16(acc + c0, v);
                     asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
 #pragma unroll
                     for (int i = 0; i < 16; ++i) {
@@ -197,6 +231,9 @@ __global__ void __launch_bounds__(kDenseThreads) dense_gemm_tc_kernel(const __gr
                     }
                 }
             }
+            asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+            __syncwarp();
+            if (lane == 0) mbar_arrive(acc_empty(set));
         }
     }
     asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
@@ -204,7 +241,7 @@ __global__ void __launch_bounds__(kDenseThreads) dense_gemm_tc_kernel(const __gr
     if (tid == 0 && *abort_flag) atomicExch(a.status, kGemmStatusTimeout);
     if (warp == 0) {
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-        asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem_base), "r"(tmem_cols) : "memory");
+        asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem_base), "r"(512u) : "memory");
     }
 }
 

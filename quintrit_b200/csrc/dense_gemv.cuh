@@ -274,13 +274,17 @@ __global__ void __launch_bounds__(256) norm_rows_kernel(const float* x, int widt
     }
 }
 
-// The mixer's output norm of many tokens (parts_norm), into the storage type; without a norm a plain conversion.
+// The mixer's output norm of many tokens (parts_norm), into the storage type; without a norm a plain conversion. gate (may be nullptr):
+// y is first multiplied by silu(gate[token * gate_ld + i]).
 template <typename T>
-__global__ void __launch_bounds__(256) finish_rows_kernel(const float* y, int inner, int parts, float eps, const float* w, int w_len, T* out, int pitch) {
+__global__ void __launch_bounds__(256) finish_rows_kernel(const float* y, const float* gate, int gate_ld, int inner, int parts, float eps, const float* w, int w_len, T* out, int pitch) {
     extern __shared__ float act_smem[];
     __shared__ float red[8];
     const int t = blockIdx.x;
-    for (int i = threadIdx.x; i < inner; i += blockDim.x) act_smem[i] = y[size_t(t) * inner + i];
+    for (int i = threadIdx.x; i < inner; i += blockDim.x) {
+        const float v = y[size_t(t) * inner + i];
+        act_smem[i] = gate != nullptr ? v * silu_f(gate[size_t(t) * gate_ld + i]) : v;
+    }
     __syncthreads();
     if (parts > 0) parts_norm<float>(act_smem, inner, inner, parts, eps, w, w_len, red);
     for (int i = threadIdx.x; i < inner; i += blockDim.x) out[size_t(t) * pitch + i] = to_storage<T>(act_smem[i]);

@@ -11,16 +11,18 @@
 #pragma once
 #include <memory>
 
+#include "chunk_scan.cuh"
 #include "dense_gemm_tc.cuh"
 #include "dense_gemv.cuh"
 #include "gated_scan.cuh"
 #include "layered_spec.hpp"
 #include "pooled_attention.cuh"
+#include "pooled_attention_mma.cuh"
 #include "tensor_map.cuh"
 
 namespace qtb {
 
-constexpr int kLayeredChunk = 1024;     // tokens of a prompt chunk
+constexpr int kLayeredChunk = 2048;     // tokens of a prompt chunk
 constexpr int kLayeredLogitRows = 64;   // rows of logits computed at a time when several positions of a chunk are asked for
 constexpr int kLayeredMaxBatch = 256;   // sequences of a batched step
 
@@ -91,6 +93,7 @@ struct LayeredDecoder {
     std::vector<CUtensorMap> map_y, map_m;  // per layer: the pitches differ
     float *part_acc = nullptr, *part_ml = nullptr;
     unsigned int* done = nullptr;
+    char* work = nullptr;               // chunked recurrences: operands of one layer (ChunkWork)
 };
 
 // Where the tokens of a pass sit: consecutive tokens of one sequence (`slot` of the store, position in pos[0]), or one token for each of
@@ -332,10 +335,15 @@ inline int layered_decoder_setup(quintrit_b200_decoder* d, const std::shared_ptr
     int rc = layered_store_create(m, 1, d->ctx, alloc, &y->store);
     if (rc != QUINTRIT_OK) return rc;
     const size_t C = kLayeredChunk, W = m.spec.width, wp = m.embed.pitch, e = m.elem();
-    size_t p1 = 0, inner = 0, op = 0, mp = kColPad, parts = 1, groups = 1, acc = 4;
+    size_t work = 0, p1 = 0, inner = 0, op = 0, mp = kColPad, parts = 1, groups = 1, acc = 4;
     for (const LayeredLayer& l : m.layers) {
         p1 = std::max<size_t>(p1, l.spec.in_rows()), inner = std::max<size_t>(inner, l.spec.inner()), op = std::max<size_t>(op, l.o.pitch), mp = std::max<size_t>(mp, l.down.pitch);
-        if (l.spec.kind != MixerKind::kAttention) continue;
+        if (l.spec.kind != MixerKind::kAttention) {
+            ChunkWork cw;
+            if (!m.f32 && chunk_scan_rows(l.spec.key_dim()) != 0)
+                work = std::max(work, chunk_work(nullptr, l.spec.kind == MixerKind::kMamba2, l.spec.heads, l.spec.vdim, l.spec.key_dim(), l.spec.groups, kLayeredChunk, &cw));
+            continue;
+        }
         groups = std::max<size_t>(groups, size_t(l.spec.kv_heads) * ((l.spec.heads / l.spec.kv_heads + kPaHeads - 1) / kPaHeads));
         for (int n = 1; n <= kLayeredMaxBatch; ++n) {
             const size_t sp = pooled_splits(l.spec, d->ctx, n, m.sm_count);
@@ -344,18 +352,19 @@ inline int layered_decoder_setup(quintrit_b200_decoder* d, const std::shared_ptr
     }
     if ((rc = dev_alloc(d, &y->tokens, C)) || (rc = dev_alloc(d, &y->pos, 4)) || (rc = dev_alloc(d, &y->rows, C)) || (rc = dev_alloc(d, &y->x, C * W)) || (rc = dev_alloc(d, &y->p1, C * p1)) ||
         (rc = dev_alloc(d, &y->g1, C * W)) || (rc = dev_alloc(d, &y->g2, C * W)) || (rc = dev_alloc(d, &y->y, C * inner)) || (rc = alloc(&y->h1, C * wp * e)) ||
-        (rc = alloc(&y->h2, C * wp * e)) || (rc = alloc(&y->y_t, C * op * e)) || (rc = alloc(&y->m, C * mp * e)) || (rc = alloc(&y->h_head, size_t(kDenseN) * wp * e)) ||
-        (rc = dev_alloc(d, &y->part_acc, acc)) || (rc = dev_alloc(d, &y->part_ml, 2 * parts)) || (rc = dev_alloc(d, &y->done, groups * kLayeredMaxBatch)))
+        (rc = alloc(&y->h2, C * wp * e)) || (rc = alloc(&y->y_t, C * op * e)) || (rc = alloc(&y->m, C * mp * e)) || (rc = alloc(&y->h_head, size_t(kDenseBox) * wp * e)) ||
+        (rc = dev_alloc(d, &y->part_acc, acc)) || (rc = dev_alloc(d, &y->part_ml, 2 * parts)) || (rc = dev_alloc(d, &y->done, groups * kLayeredMaxBatch)) ||
+        (rc = dev_alloc(d, &y->work, work)))
         return rc;
     if (!m.f32) {
-        if ((rc = tensor_map_2d_bf16(&y->map_h1, y->h1, m.embed.pitch, C, kDenseK, kDenseN)) || (rc = tensor_map_2d_bf16(&y->map_h2, y->h2, m.embed.pitch, C, kDenseK, kDenseN)) ||
-            (rc = tensor_map_2d_bf16(&y->map_head, y->h_head, m.embed.pitch, kDenseN, kDenseK, kDenseN)))
+        if ((rc = tensor_map_2d_bf16(&y->map_h1, y->h1, m.embed.pitch, C, kDenseK, kDenseBox)) || (rc = tensor_map_2d_bf16(&y->map_h2, y->h2, m.embed.pitch, C, kDenseK, kDenseBox)) ||
+            (rc = tensor_map_2d_bf16(&y->map_head, y->h_head, m.embed.pitch, kDenseBox, kDenseK, kDenseBox)))
             return rc;
         y->map_y.resize(m.layers.size()), y->map_m.resize(m.layers.size());
         for (size_t i = 0; i < m.layers.size(); ++i) {
-            if ((rc = tensor_map_2d_bf16(&y->map_y[i], y->y_t, m.layers[i].o.pitch, C, kDenseK, kDenseN))) return rc;
+            if ((rc = tensor_map_2d_bf16(&y->map_y[i], y->y_t, m.layers[i].o.pitch, C, kDenseK, kDenseBox))) return rc;
             y->map_m[i] = y->map_y[i];
-            if (m.layers[i].spec.ff > 0 && (rc = tensor_map_2d_bf16(&y->map_m[i], y->m, m.layers[i].down.pitch, C, kDenseK, kDenseN))) return rc;
+            if (m.layers[i].spec.ff > 0 && (rc = tensor_map_2d_bf16(&y->map_m[i], y->m, m.layers[i].down.pitch, C, kDenseK, kDenseBox))) return rc;
         }
     }
     // shared-memory limits are a property of the kernel: set to the most a block may have
@@ -373,7 +382,13 @@ inline int layered_decoder_setup(quintrit_b200_decoder* d, const std::shared_ptr
                              reinterpret_cast<const void*>(gated_scan_kernel<kScanMamba2>), reinterpret_cast<const void*>(gated_scan_kernel<kScanHgrn2>),
                              reinterpret_cast<const void*>(pooled_attention_kernel<bf16, true>), reinterpret_cast<const void*>(pooled_attention_kernel<bf16, false>),
                              reinterpret_cast<const void*>(pooled_attention_kernel<float, true>), reinterpret_cast<const void*>(pooled_attention_kernel<float, false>),
-                             reinterpret_cast<const void*>(dense_gemm_tc_kernel<true>), reinterpret_cast<const void*>(dense_gemm_tc_kernel<false>)};
+                             reinterpret_cast<const void*>(dense_gemm_tc_kernel<128, true>), reinterpret_cast<const void*>(dense_gemm_tc_kernel<128, false>),
+                             reinterpret_cast<const void*>(dense_gemm_tc_kernel<256, false>),
+                             reinterpret_cast<const void*>(chunk_scan_kernel<kScanMamba2, 32>), reinterpret_cast<const void*>(chunk_scan_kernel<kScanMamba2, 64>),
+                             reinterpret_cast<const void*>(chunk_scan_kernel<kScanMamba2, 128>), reinterpret_cast<const void*>(chunk_scan_kernel<kScanHgrn2, 32>),
+                             reinterpret_cast<const void*>(chunk_scan_kernel<kScanHgrn2, 64>), reinterpret_cast<const void*>(chunk_scan_kernel<kScanHgrn2, 128>),
+                             reinterpret_cast<const void*>(pooled_attention_mma_kernel<32>), reinterpret_cast<const void*>(pooled_attention_mma_kernel<64>),
+                             reinterpret_cast<const void*>(pooled_attention_mma_kernel<128>)};
     for (const void* k : kernels)
         if ((rc = allow(k)) != QUINTRIT_OK) return rc;
     // the largest requests of this model against what a block may have
@@ -416,6 +431,37 @@ inline int layered_in_stacks(const LayeredDecoder& y, const LayeredLayer& l, Den
 inline int layered_norm_parts(const LayerSpec& l) { return l.kind == MixerKind::kMamba2 ? l.norm_groups : l.kind == MixerKind::kHgrn2 ? l.heads : 0; }
 inline int layered_norm_len(const LayerSpec& l) { return l.kind == MixerKind::kMamba2 ? l.inner() : l.vdim; }
 
+// Many tokens of a recurrence in 16-token chunks.
+inline int layered_chunk_scan(quintrit_b200_decoder* d, const LayerSpec& l, const ScanArgs& a) {
+    cudaStream_t s = d->stream;
+    const bool mamba = l.kind == MixerKind::kMamba2;
+    ChunkWork w;
+    chunk_work(d->lay->work, mamba, l.heads, l.vdim, a.n, l.groups, a.tokens, &w);
+    const int chunks = chunk_count(a.tokens), rows = w.rows;
+    if (mamba) {
+        ssd_conv_kernel<<<dim3((l.heads * w.v_pad + 2 * l.groups * rows + 127) / 128, chunks), 128, 0, s>>>(a, w);
+        QTB_LAUNCH_CHECK();
+        ssd_gram_kernel<<<dim3(l.groups + 1, chunks), 256, size_t(2 * kChunkT) * (rows + 1) * sizeof(float), s>>>(a, w);
+        QTB_LAUNCH_CHECK();
+    } else {
+        hgrn_prep_kernel<<<dim3(l.heads, chunks), 128, size_t(3 * kChunkT) * rows * sizeof(float), s>>>(a, w);
+        QTB_LAUNCH_CHECK();
+    }
+    const dim3 grid(l.heads, w.v_pad / kChunkV);
+    auto go = [&](auto kernel, size_t smem) { kernel<<<grid, 128, smem, s>>>(a, w); };
+    if (mamba) {
+        const size_t smem = chunk_scan_smem<kScanMamba2>(rows);
+        rows == 32 ? go(chunk_scan_kernel<kScanMamba2, 32>, smem) : rows == 64 ? go(chunk_scan_kernel<kScanMamba2, 64>, smem) : go(chunk_scan_kernel<kScanMamba2, 128>, smem);
+        QTB_LAUNCH_CHECK();
+        conv_tail_kernel<<<(l.conv_dim() + 255) / 256, 256, 0, s>>>(a);
+    } else {
+        const size_t smem = chunk_scan_smem<kScanHgrn2>(rows);
+        rows == 32 ? go(chunk_scan_kernel<kScanHgrn2, 32>, smem) : rows == 64 ? go(chunk_scan_kernel<kScanHgrn2, 64>, smem) : go(chunk_scan_kernel<kScanHgrn2, 128>, smem);
+    }
+    QTB_LAUNCH_CHECK();
+    return QUINTRIT_OK;
+}
+
 template <typename T>
 int layered_mixer(quintrit_b200_decoder* d, size_t li, int n, const LayeredTarget& tg) {
     LayeredDecoder& y = *d->lay;
@@ -432,6 +478,7 @@ int layered_mixer(quintrit_b200_decoder* d, size_t li, int n, const LayeredTarge
         a.conv_w = w.conv_w, a.conv_b = w.conv_b, a.dt_bias = w.dt_bias, a.a_log = w.a_log, a.d_skip = w.d_skip, a.f_bias = w.f_bias, a.lower = w.lower;
         a.state = st.state, a.conv = st.conv, a.y = y.y;
         const dim3 grid(l.heads, (l.vdim + kScanRows - 1) / kScanRows, seqs);
+        if (sizeof(T) == 2 && tokens > kChunkT / 2 && chunk_scan_rows(a.n) != 0) return layered_chunk_scan(d, l, a);
         if (l.kind == MixerKind::kMamba2) {
             gated_scan_kernel<kScanMamba2><<<grid, kScanThreads, scan_smem(a.n), s>>>(a);
             QTB_LAUNCH_CHECK();
@@ -459,9 +506,19 @@ int layered_mixer(quintrit_b200_decoder* d, size_t li, int n, const LayeredTarge
         return QUINTRIT_OK;
     }
     const int unit = l.pool > 0 ? l.pool : 64;
-    pooled_append_kernel<T><<<dim3(tokens / unit + 2, l.kv_heads, 1), 128, 0, s>>>(a);
+    pooled_append_kernel<T><<<dim3(tokens / unit + 2, l.kv_heads, 1), 256, 0, s>>>(a);
     QTB_LAUNCH_CHECK();
     a.splits = 1;
+    if constexpr (sizeof(T) == 2) {
+        const int dims = pooled_mma_dims(l.dim, l.vdim);
+        if (dims != 0) {
+            const dim3 grid((tokens + kPmRows - 1) / kPmRows, l.heads);
+            auto go = [&](auto kernel) { kernel<<<grid, kPmThreads, pooled_mma_smem(dims), s>>>(a); };
+            dims == 32 ? go(pooled_attention_mma_kernel<32>) : dims == 64 ? go(pooled_attention_mma_kernel<64>) : go(pooled_attention_mma_kernel<128>);
+            QTB_LAUNCH_CHECK();
+            return QUINTRIT_OK;
+        }
+    }
     pooled_attention_kernel<T, false><<<dim3(hg, 1, tokens), kPaThreads, smem, s>>>(a);
     QTB_LAUNCH_CHECK();
     return QUINTRIT_OK;
@@ -478,7 +535,10 @@ int layered_gemm(quintrit_b200_decoder* d, int n, const LayeredMatrix* const (&w
     for (int i = 0; i < n_stack; ++i) a.stack[i] = st[i], a.k_steps[i] = w[i]->pitch / kDenseK, a.row_tiles[i] = w[i]->rows_pad / kDenseM, tiles += a.row_tiles[i];
     const int j = n_stack > 1 ? 1 : 0;
     if constexpr (sizeof(T) == 2)
-        dense_gemm_tc_kernel<false><<<dim3((n + kDenseN - 1) / kDenseN, tiles), kDenseThreads, kDenseSmem, d->stream>>>(w[0]->map, *hmap[0], w[j]->map, *hmap[j], a);
+        if (n > kDenseBox)
+            dense_gemm_tc_kernel<256, false><<<std::min(d->sm_count, (n + 255) / 256 * tiles), kDenseThreads, dense_smem(256), d->stream>>>(w[0]->map, *hmap[0], w[j]->map, *hmap[j], a);
+        else
+            dense_gemm_tc_kernel<128, false><<<std::min(d->sm_count, tiles), kDenseThreads, dense_smem(128), d->stream>>>(w[0]->map, *hmap[0], w[j]->map, *hmap[j], a);
     else
         dense_gemm_f32_kernel<false><<<dim3((n + kF32Tile - 1) / kF32Tile, tiles * (kDenseM / kF32Tile)), 256, 0, d->stream>>>(
             static_cast<const float*>(w[0]->w), static_cast<const float*>(h[0]), w[0]->pitch, static_cast<const float*>(w[j]->w), static_cast<const float*>(h[j]), w[j]->pitch, a);
@@ -528,7 +588,8 @@ int layered_layers(quintrit_b200_decoder* d, const uint32_t* tokens, int n, cons
         const CUtensorMap* const hm[2] = {&y.map_h1, &y.map_h2};
         const void* const hs[2] = {y.h1, y.h2};
         if ((rc = layered_gemm<T>(d, n, ws, hm, hs, st, n_stack)) != QUINTRIT_OK || (rc = layered_mixer<T>(d, li, n, tg)) != QUINTRIT_OK) return rc;
-        finish_rows_kernel<T><<<n, 256, size_t(l.spec.inner()) * sizeof(float), s>>>(y.y, l.spec.inner(), parts, m.spec.eps, l.mix_norm, norm_len, static_cast<T*>(y.y_t), l.o.pitch);
+        const float* gate = sizeof(T) == 2 && l.spec.kind == MixerKind::kMamba2 && !tg.step() && n > kChunkT / 2 && chunk_scan_rows(l.spec.state) != 0 ? y.p1 : nullptr;  // silu(z)
+        finish_rows_kernel<T><<<n, 256, size_t(l.spec.inner()) * sizeof(float), s>>>(y.y, gate, l.spec.in_rows(), l.spec.inner(), parts, m.spec.eps, l.mix_norm, norm_len, static_cast<T*>(y.y_t), l.o.pitch);
         QTB_LAUNCH_CHECK();
         DenseGemmArgs a{};
         a.tokens = n, a.n_prob = 1, a.status = d->d_counters + 2, a.spin_limit = kDenseSpinLimit;
@@ -536,7 +597,7 @@ int layered_layers(quintrit_b200_decoder* d, const uint32_t* tokens, int n, cons
         a.x = y.x, a.width = W;
         if (l.spec.gated_residual) a.gate1 = y.g1, a.gate2 = y.g2;
         if constexpr (sizeof(T) == 2)
-            dense_gemm_tc_kernel<true><<<dim3((n + kDenseN - 1) / kDenseN, a.row_tiles[0]), kDenseThreads, kDenseSmem, s>>>(l.o.map, y.map_y[li], l.spec.ff > 0 ? l.down.map : l.o.map, y.map_m[li], a);
+            dense_gemm_tc_kernel<128, true><<<std::min(d->sm_count, (n + 127) / 128 * a.row_tiles[0]), kDenseThreads, dense_smem(128), s>>>(l.o.map, y.map_y[li], l.spec.ff > 0 ? l.down.map : l.o.map, y.map_m[li], a);
         else
             dense_gemm_f32_kernel<true><<<dim3((n + kF32Tile - 1) / kF32Tile, a.row_tiles[0] * (kDenseM / kF32Tile)), 256, 0, s>>>(
                 static_cast<const float*>(l.o.w), static_cast<const float*>(y.y_t), l.o.pitch, static_cast<const float*>(l.down.w), static_cast<const float*>(y.m), l.down.pitch, a);
@@ -560,7 +621,7 @@ int layered_head(quintrit_b200_decoder* d, int row, float* logits) {
     return QUINTRIT_OK;
 }
 
-// The same for n <= kDenseN rows - those listed in `rows`, or first .. first + n - 1 where it is nullptr -> logits[n][vocab].
+// The same for n <= kDenseBox rows - those listed in `rows`, or first .. first + n - 1 where it is nullptr -> logits[n][vocab].
 template <typename T>
 int layered_head_rows(quintrit_b200_decoder* d, const uint32_t* rows, int first, int n, float* logits) {
     LayeredDecoder& y = *d->lay;

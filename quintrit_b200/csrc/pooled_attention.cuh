@@ -40,7 +40,7 @@ __device__ __forceinline__ int pooled_blocks_seen(int pos, int window, int pool)
 // Writes keys and values of the launch's tokens to the ring and the means of the blocks that become complete.
 // grid: (aligned groups of tokens, kv heads, sequences); the groups are `pool` tokens long (64 without pooling).
 template <typename T>
-__global__ void __launch_bounds__(128) pooled_append_kernel(const __grid_constant__ PooledAttnArgs a) {
+__global__ void __launch_bounds__(256) pooled_append_kernel(const __grid_constant__ PooledAttnArgs a) {
     const int z = blockIdx.z, kvh = blockIdx.y, unit = a.pool > 0 ? a.pool : 64;
     const uint32_t slot = a.seq.pos_stride != 0 ? seq_of(a.seq, z) : 0;
     const int pos0 = static_cast<int>(seq_position(a.seq, a.pos, z)), end = pos0 + a.tokens;
@@ -57,10 +57,17 @@ __global__ void __launch_bounds__(128) pooled_append_kernel(const __grid_constan
         float sum = 0.0f;
         if (complete)
             for (int j = b0; j < min(pos0, b1); ++j) sum += from_storage(ring[size_t(j % a.cache.ring) * step]);
-        for (int j = max(b0, pos0); j < min(b1, end); ++j) {
-            const T v = to_storage<T>(e < width ? rows[size_t(j - pos0) * a.ld + src] : 0.0f);
-            ring[size_t(j % a.cache.ring) * step] = v;
-            sum += from_storage(v);
+        for (int j0 = max(b0, pos0); j0 < min(b1, end); j0 += 8) {
+            float v[8];  // eight loads in flight
+#pragma unroll
+            for (int k = 0; k < 8; ++k) v[k] = e < width && j0 + k < min(b1, end) ? rows[size_t(j0 + k - pos0) * a.ld + src] : 0.0f;
+#pragma unroll
+            for (int k = 0; k < 8; ++k)
+                if (j0 + k < min(b1, end)) {
+                    const T t = to_storage<T>(v[k]);
+                    ring[size_t((j0 + k) % a.cache.ring) * step] = t;
+                    sum += from_storage(t);
+                }
         }
         if (complete) {
             T* pool = static_cast<T*>(key ? a.cache.pk : a.cache.pv) + ((size_t(slot) * a.cache.blocks + block) * a.kv_heads + kvh) * pad + e;

@@ -172,12 +172,15 @@ def torch_normal_f16_bits(seed: int, n: int, std: float, device, chunk: int = 1 
     return out
 
 
-def torch_model(shape: str, device, ctx: int, f32_values: bool = False, config: int = 2, layers: int | None = None, tp=None) -> dict:
+def torch_model(shape, device, ctx: int, f32_values: bool = False, config: int = 2, layers: int | None = None, tp=None) -> dict:
     """The Falcon3-10B-shape or BitNet-2B-shape model with seeded random-init weights, built on a torch device."""
     if shape == "falcon3_10b":
         arch, hidden, inter, L, qh, kvh, hd, vocab, theta, eps, tied = 0, 3072, 23040, 40, 12, 4, 256, 131072, 1000042.0, 1e-6, False
     elif shape == "bitnet_2b":
         arch, hidden, inter, L, qh, kvh, hd, vocab, theta, eps, tied = 1, 2560, 6912, 30, 20, 5, 128, 128256, 500000.0, 1e-5, True
+    elif isinstance(shape, dict):  # LLaMA form at sizes of the caller's
+        arch, theta, eps, tied = 0, 500000.0, 1e-6, True
+        hidden, inter, L, qh, kvh, hd, vocab = (shape[k] for k in ("hidden", "inter", "layers", "q_heads", "kv_heads", "head_dim", "vocab"))
     else:
         raise ValueError(shape)
     L = layers or L
