@@ -473,6 +473,14 @@ int quintrit_session_logits(struct quintrit_session* session, float* out, size_t
 int quintrit_session_generate_tokens(struct quintrit_session* session, const uint32_t* prompt, size_t prompt_len, size_t max_new, uint32_t* out,
                                      size_t out_capacity, size_t* out_count);
 
+/* Generation without text: up to params->max_tokens ids after the prompt, greedy or sampled (temperature, top_k, top_p, seed of
+ * quintrit_generate_params_t; stop sequences do not apply), for models without a tokenizer and servers that tokenize elsewhere. It ends early
+ * when the context is full. flags: QUINTRIT_GENERATE_KEEP_CONTEXT continues after the tokens the session holds; the last token returned has not
+ * been fed. */
+struct quintrit_generate_params;
+int quintrit_b200_session_sample_tokens(struct quintrit_session* session, const uint32_t* prompt, size_t prompt_len, const struct quintrit_generate_params* params,
+                                        uint32_t* out, size_t out_capacity, size_t* out_count);
+
 /* Prompt tokens that the last quintrit_session_generate call of this session found in the KV cache and did not compute again: a prompt
  * that begins like the conversation the session holds is ingested from the first differing token on (the reference's
  * InferenceEngine::reusable_prefix, quintrit-runtime/src/engine.rs:700-727; at least the last prompt token is always computed). */

@@ -6,6 +6,9 @@
 //                          ending (plain, sigmoid of a gate, SwiGLU of interleaved gate | up rows)
 //   finish_project_kernel  the mixer's output norm, then output and down projection, both gates and the residual sum
 //
+// The kernels of a decode step follow one another with programmatic dependent launch: a kernel may start while the one before it still runs,
+// brings what does not depend on it (weights, states, cached keys) on the way, and only then waits for its results.
+//
 // A warp owns two rows (one in the second kernel) and streams them with 16-byte loads, four per row in flight and lane; the activation
 // vector lies in shared memory as floats.
 #pragma once
@@ -30,6 +33,23 @@ __device__ __forceinline__ float from_storage(bf16 v) { return __bfloat162float(
 template <typename T> __device__ __forceinline__ float round_to(float v) { return from_storage(to_storage<T>(v)); }
 __device__ __forceinline__ float sigmoid_f(float v) { return 1.0f / (1.0f + expf(-v)); }
 __device__ __forceinline__ float silu_f(float v) { return v / (1.0f + expf(-v)); }
+
+// Programmatic dependent launch: the next kernel of the stream may start / everything the kernels before this one wrote is visible. Both do
+// nothing in a kernel that was launched without the attribute.
+__device__ __forceinline__ void pdl_trigger() { asm volatile("griddepcontrol.launch_dependents;" ::: "memory"); }
+__device__ __forceinline__ void pdl_wait() { asm volatile("griddepcontrol.wait;" ::: "memory"); }
+template <typename... P, typename... A>
+inline cudaError_t launch_dependent(void (*kernel)(P...), dim3 grid, int threads, size_t smem, cudaStream_t s, const A&... args) {
+    cudaLaunchConfig_t cfg{};
+    cudaLaunchAttribute attr{};
+    attr.id = cudaLaunchAttributeProgrammaticStreamSerialization, attr.val.programmaticStreamSerializationAllowed = 1;
+    cfg.gridDim = grid, cfg.blockDim = dim3(threads), cfg.dynamicSmemBytes = smem, cfg.stream = s, cfg.attrs = &attr, cfg.numAttrs = 1;
+    return cudaLaunchKernelEx(&cfg, kernel, static_cast<P>(args)...);
+}
+// `bytes` (a multiple of 16) from p on are requested into L2.
+__device__ __forceinline__ void l2_prefetch(const void* p, size_t bytes) {
+    asm volatile("cp.async.bulk.prefetch.L2.global [%0], %1;" ::"l"(p), "r"(static_cast<uint32_t>(bytes)) : "memory");
+}
 
 // What becomes of the rows of one range of a stacked projection.
 enum SegKind : int { kSegPlain = 0, kSegSigmoid = 1, kSegSwiGlu = 2 };
@@ -95,24 +115,44 @@ __device__ __forceinline__ float dot_piece(const uint4& w, const float* h, int p
     return fmaf(__uint_as_float(w.w), a.w, s);
 }
 
-// Sums of R consecutive rows over the vector h (shared memory): every lane returns the whole sums.
+// Four consecutive elements (e a multiple of 4) of an activation vector, and eight of the storage type.
+template <typename T> __device__ __forceinline__ void act_put4(float* h, int e, int pitch, float4 v) { *reinterpret_cast<float4*>(h + act_index<T>(e, pitch)) = v; }
+__device__ __forceinline__ void act_put_storage(float* h, int piece, int pitch, const bf16* src) {
+    const uint4 w = *reinterpret_cast<const uint4*>(src + piece * 8);
+    const auto lo = [](uint32_t u) { return __uint_as_float(u << 16); };
+    const auto hi = [](uint32_t u) { return __uint_as_float(u & 0xffff0000u); };
+    act_put4<bf16>(h, piece * 8, pitch, make_float4(lo(w.x), hi(w.x), lo(w.y), hi(w.y)));
+    act_put4<bf16>(h, piece * 8 + 4, pitch, make_float4(lo(w.z), hi(w.z), lo(w.w), hi(w.w)));
+}
+__device__ __forceinline__ void act_put_storage(float* h, int piece, int, const float* src) {
+    *reinterpret_cast<float4*>(h + piece * 4) = *reinterpret_cast<const float4*>(src + piece * 4);
+}
+
+// The first pieces of R consecutive rows, in registers: they can be on their way before the vector is known.
+template <int R> struct RowHead { uint4 v[R][8 / R]; };
 template <typename T, int R>
-__device__ __forceinline__ void dot_rows(const T* w, int pitch, const float* h, float (&sum)[R]) {
-    constexpr int kPer = 16 / sizeof(T), U = 4;
+__device__ __forceinline__ void load_pieces(RowHead<R>& b, const T* w, int pitch, int p0) {
+    constexpr int kPer = 16 / sizeof(T);
+    const int pieces = pitch / kPer;
+#pragma unroll
+    for (int u = 0; u < 8 / R; ++u)
+#pragma unroll
+        for (int r = 0; r < R; ++r) b.v[r][u] = p0 + 32 * u < pieces ? load_stream(w + size_t(r) * pitch + size_t(p0 + 32 * u) * kPer) : make_uint4(0, 0, 0, 0);
+}
+// Sums of R consecutive rows over the vector h (shared memory), the rows' first pieces in `head`: every lane returns the whole sums.
+template <typename T, int R>
+__device__ __forceinline__ void dot_rows(const T* w, int pitch, const float* h, RowHead<R>& head, float (&sum)[R]) {
+    constexpr int kPer = 16 / sizeof(T), U = 8 / R;
     const int pieces = pitch / kPer, lane = threadIdx.x & 31;
 #pragma unroll
     for (int r = 0; r < R; ++r) sum[r] = 0.0f;
     for (int p0 = lane; p0 < pieces; p0 += 32 * U) {
-        uint4 v[R][U];
-#pragma unroll
-        for (int u = 0; u < U; ++u)
-#pragma unroll
-            for (int r = 0; r < R; ++r) v[r][u] = p0 + 32 * u < pieces ? load_stream(w + size_t(r) * pitch + size_t(p0 + 32 * u) * kPer) : make_uint4(0, 0, 0, 0);
+        if (p0 != lane) load_pieces<T, R>(head, w, pitch, p0);
 #pragma unroll
         for (int u = 0; u < U; ++u)
             if (p0 + 32 * u < pieces) {
 #pragma unroll
-                for (int r = 0; r < R; ++r) sum[r] += dot_piece(v[r][u], h, p0 + 32 * u, pitch, T());
+                for (int r = 0; r < R; ++r) sum[r] += dot_piece(head.v[r][u], h, p0 + 32 * u, pitch, T());
             }
     }
 #pragma unroll
@@ -136,16 +176,44 @@ __global__ void __launch_bounds__(kProjectThreads) norm_project_kernel(NormProje
     __shared__ float red[kProjectThreads / 32];
     const int tid = threadIdx.x, token = blockIdx.y, pitch = a.stack[0].pitch;
     const float* x = a.x + size_t(token) * a.width;
-    float ss = 0.0f;
-    for (int i = tid; i < a.width; i += kProjectThreads) ss += x[i] * x[i];
-    ss = block_sum(ss, red);
-    const float inv = 1.0f / sqrtf(ss / static_cast<float>(a.width) + a.eps);
-    for (int s = 0; s < a.n_stack; ++s)
-        for (int i = tid; i < pitch; i += kProjectThreads)
-            act_smem[s * pitch + act_index<T>(i, pitch)] = i < a.width ? round_to<T>(x[i] * inv * a.norm_w[s][i]) : 0.0f;
-    __syncthreads();
     const int warps = gridDim.x * (kProjectThreads / 32);
     int unit = blockIdx.x * (kProjectThreads / 32) + (tid >> 5);
+    pdl_trigger();
+    RowHead<2> head;  // the rows this warp begins with
+    {
+        int u = unit;
+        for (int s = 0; s < a.n_stack; ++s)
+            for (int k = 0; k < a.stack[s].n_seg; ++k) {
+                const int units = (a.stack[s].seg[k].rows + 1) / 2;
+                if (u >= 0 && u < units) load_pieces<T, 2>(head, static_cast<const T*>(a.stack[s].w) + size_t(a.stack[s].seg[k].row0 + 2 * u) * pitch, pitch, tid & 31);
+                u -= units;
+            }
+    }
+    bool first = true;
+    pdl_wait();
+    float ss = 0.0f;
+    for (int i = tid; i < pitch; i += kProjectThreads) {
+        const float v = i < a.width ? x[i] : 0.0f;
+        act_smem[i] = v;  // (a thread keeps its own elements here until the sum is known)
+        ss += v * v;
+    }
+    ss = block_sum(ss, red);
+    const float inv = 1.0f / sqrtf(ss / static_cast<float>(a.width) + a.eps);
+    constexpr int kKeep = 16;
+    float keep[kKeep];
+#pragma unroll
+    for (int j = 0; j < kKeep; ++j) keep[j] = tid + j * kProjectThreads < pitch ? act_smem[tid + j * kProjectThreads] : 0.0f;
+    __syncthreads();
+    for (int s = 0; s < a.n_stack; ++s) {
+#pragma unroll
+        for (int j = 0; j < kKeep; ++j) {
+            const int i = tid + j * kProjectThreads;
+            if (i < pitch) act_smem[s * pitch + act_index<T>(i, pitch)] = i < a.width ? round_to<T>(keep[j] * inv * a.norm_w[s][i]) : 0.0f;
+        }
+        for (int i = tid + kKeep * kProjectThreads; i < pitch; i += kProjectThreads)
+            act_smem[s * pitch + act_index<T>(i, pitch)] = i < a.width ? round_to<T>(x[i] * inv * a.norm_w[s][i]) : 0.0f;
+    }
+    __syncthreads();
     for (int s = 0; s < a.n_stack; ++s)
         for (int k = 0; k < a.stack[s].n_seg; ++k) {
             const DenseSeg& g = a.stack[s].seg[k];
@@ -153,7 +221,10 @@ __global__ void __launch_bounds__(kProjectThreads) norm_project_kernel(NormProje
             for (; unit < units; unit += warps) {
                 const int r = unit * 2;
                 float v[2];  // (an odd last row has a row of padding behind it: row ranges are padded to kRowPad)
-                dot_rows<T, 2>(static_cast<const T*>(a.stack[s].w) + size_t(g.row0 + r) * pitch, pitch, act_smem + s * pitch, v);
+                const T* rows = static_cast<const T*>(a.stack[s].w) + size_t(g.row0 + r) * pitch;
+                if (!first) load_pieces<T, 2>(head, rows, pitch, tid & 31);
+                first = false;
+                dot_rows<T, 2>(rows, pitch, act_smem + s * pitch, head, v);
                 if ((tid & 31) != 0) continue;
                 if (g.kind == kSegSwiGlu) {
                     static_cast<T*>(g.t)[size_t(token) * g.ld + unit] = to_storage<T>(silu_f(v[0]) * v[1]);
@@ -226,19 +297,50 @@ __global__ void __launch_bounds__(kProjectThreads) finish_project_kernel(FinishP
     __shared__ float red[kProjectThreads / 32];
     const int tid = threadIdx.x, lane = tid & 31, token = blockIdx.y;
     float *y = act_smem, *m = act_smem + a.o_pitch;
-    for (int i = tid; i < a.o_pitch; i += kProjectThreads) {
-        const float v = i < a.inner ? a.y[size_t(token) * a.inner + i] : 0.0f;
-        y[act_index<T>(i, a.o_pitch)] = a.norm_parts > 0 ? v : round_to<T>(v);
-    }
-    if (a.m != nullptr)
-        for (int i = tid; i < a.down_pitch; i += kProjectThreads) m[act_index<T>(i, a.down_pitch)] = from_storage(static_cast<const T*>(a.m)[size_t(token) * a.down_pitch + i]);
-    __syncthreads();
-    if (a.norm_parts > 0) parts_norm<T>(y, a.inner, a.o_pitch, a.norm_parts, a.eps, a.norm_w, a.norm_len, red);
     const int warps = gridDim.x * (kProjectThreads / 32);
+    pdl_trigger();
+    RowHead<1> head;
+    bool first = true;
+    if (const int row = blockIdx.x * (kProjectThreads / 32) + (tid >> 5); row < a.width) {
+        load_pieces<T, 1>(head, static_cast<const T*>(a.o) + size_t(row) * a.o_pitch, a.o_pitch, lane);
+        if (lane == 0) {
+            l2_prefetch(static_cast<const T*>(a.o) + size_t(row) * a.o_pitch, a.o_pitch * sizeof(T));
+            if (a.m != nullptr) l2_prefetch(static_cast<const T*>(a.down) + size_t(row) * a.down_pitch, a.down_pitch * sizeof(T));
+        }
+    }
+    pdl_wait();
+    const float* yt = a.y + size_t(token) * a.inner;
+    const bool norm = a.norm_parts > 0;
+    if (a.inner % 4 == 0) {
+#pragma unroll 4
+        for (int i = tid * 4; i < a.o_pitch; i += kProjectThreads * 4) {
+            float4 v = i < a.inner ? *reinterpret_cast<const float4*>(yt + i) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            if (!norm) v = make_float4(round_to<T>(v.x), round_to<T>(v.y), round_to<T>(v.z), round_to<T>(v.w));
+            act_put4<T>(y, i, a.o_pitch, v);
+        }
+    } else {
+        for (int i = tid; i < a.o_pitch; i += kProjectThreads) {
+            const float v = i < a.inner ? yt[i] : 0.0f;
+            y[act_index<T>(i, a.o_pitch)] = norm ? v : round_to<T>(v);
+        }
+    }
+    if (a.m != nullptr) {
+        constexpr int kPer = 16 / sizeof(T);
+#pragma unroll 4
+        for (int i = tid; i < a.down_pitch / kPer; i += kProjectThreads) act_put_storage(m, i, a.down_pitch, static_cast<const T*>(a.m) + size_t(token) * a.down_pitch);
+    }
+    __syncthreads();
+    if (norm) parts_norm<T>(y, a.inner, a.o_pitch, a.norm_parts, a.eps, a.norm_w, a.norm_len, red);
     for (int row = blockIdx.x * (kProjectThreads / 32) + (tid >> 5); row < a.width; row += warps) {
         float so[1], sd[1] = {0.0f};
-        dot_rows<T, 1>(static_cast<const T*>(a.o) + size_t(row) * a.o_pitch, a.o_pitch, y, so);
-        if (a.m != nullptr) dot_rows<T, 1>(static_cast<const T*>(a.down) + size_t(row) * a.down_pitch, a.down_pitch, m, sd);
+        const T *o_row = static_cast<const T*>(a.o) + size_t(row) * a.o_pitch, *d_row = static_cast<const T*>(a.down) + size_t(row) * a.down_pitch;
+        if (!first) load_pieces<T, 1>(head, o_row, a.o_pitch, lane);
+        first = false;
+        dot_rows<T, 1>(o_row, a.o_pitch, y, head, so);
+        if (a.m != nullptr) {
+            load_pieces<T, 1>(head, d_row, a.down_pitch, lane);
+            dot_rows<T, 1>(d_row, a.down_pitch, m, head, sd);
+        }
         if (lane == 0) {
             const size_t at = size_t(token) * a.width + row;
             const float g1 = a.gate1 != nullptr ? a.gate1[at] : 1.0f, g2 = a.gate2 != nullptr ? a.gate2[at] : 1.0f;

@@ -40,11 +40,17 @@ __device__ __forceinline__ float softplus_f(float v) { return v > 20.0f ? v + lo
 __device__ __forceinline__ float conv_silu(const ScanArgs& a, const float* ring, int row, int t, uint32_t pos, int c, int channels, int inner) {
     float s = a.conv_b[c];
     const float* w = a.conv_w + size_t(c) * a.taps;
-    for (int k = 0; k < a.taps; ++k) {
-        const int back = a.taps - 1 - k;
-        if (static_cast<uint32_t>(back) > pos) continue;  // before the start of the sequence
-        const float v = back <= t ? a.p[size_t(row - back) * a.ld + inner + c] : ring[size_t((pos - back) % a.taps) * channels + c];
-        s = fmaf(w[k], v, s);
+    for (int k0 = 0; k0 < a.taps; k0 += 4) {
+        float v[4], f[4];  // four taps' loads in flight
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+            const int back = a.taps - 1 - k0 - k;
+            const bool there = back >= 0 && static_cast<uint32_t>(back) <= pos;  // not before the start of the sequence
+            const float* src = back <= t ? a.p + size_t(row - back) * a.ld + inner + c : ring + size_t((pos - back) % a.taps) * channels + c;
+            v[k] = there ? *src : 0.0f, f[k] = there ? w[k0 + k] : 0.0f;
+        }
+#pragma unroll
+        for (int k = 0; k < 4; ++k) s = fmaf(f[k], v[k], s);
     }
     return silu_f(s);
 }
@@ -59,6 +65,7 @@ inline size_t scan_smem(int n) { return (size_t(kScanStage) * (3 * n + kScanRows
 template <int KIND>
 __global__ void __launch_bounds__(kScanThreads) gated_scan_kernel(const __grid_constant__ ScanArgs a) {
     extern __shared__ float scan_sm[];
+    pdl_trigger();
     const int n = a.n, head = blockIdx.x, v0 = blockIdx.y * kScanRows, z = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     float *ks = scan_sm, *qs = ks + kScanStage * n, *as = qs + kScanStage * n, *xs = as + kScanStage * n, *one = xs + kScanStage * kScanRows;
     const uint32_t slot = a.seq.pos_stride != 0 ? seq_of(a.seq, z) : 0, pos0 = seq_position(a.seq, a.pos, z);
@@ -75,6 +82,7 @@ __global__ void __launch_bounds__(kScanThreads) gated_scan_kernel(const __grid_c
             const int i = lane + 32 * e;
             s[j][e] = pos0 > 0 && mine + j < a.vdim && i < n ? state[size_t(mine + j) * n + i] : 0.0f;
         }
+    pdl_wait();  // (the state above was written by an earlier step)
     for (int t0 = 0; t0 < a.tokens; t0 += kScanStage) {
         const int nt = min(kScanStage, a.tokens - t0);
         __syncthreads();
@@ -83,10 +91,9 @@ __global__ void __launch_bounds__(kScanThreads) gated_scan_kernel(const __grid_c
                 const float dt = softplus_f(a.p[size_t(row0 + t0 + i) * a.ld + inner + channels + head] + a.dt_bias[head]);
                 one[i] = dt, one[kScanStage + i] = expf(-expf(a.a_log[head]) * dt);
             }
-            __syncthreads();
             for (int i = tid; i < nt * n; i += kScanThreads) {
                 const int t = i / n, c = i % n;
-                ks[i] = one[t] * conv_silu(a, ring, row0 + t0 + t, t0 + t, pos0 + t0 + t, inner + group * n + c, channels, inner);
+                ks[i] = conv_silu(a, ring, row0 + t0 + t, t0 + t, pos0 + t0 + t, inner + group * n + c, channels, inner);
                 qs[i] = conv_silu(a, ring, row0 + t0 + t, t0 + t, pos0 + t0 + t, inner + a.groups * n + group * n + c, channels, inner);
             }
             for (int i = tid; i < nt * kScanRows; i += kScanThreads) {
@@ -112,12 +119,12 @@ __global__ void __launch_bounds__(kScanThreads) gated_scan_kernel(const __grid_c
             float x[4], acc[4] = {};
 #pragma unroll
             for (int j = 0; j < 4; ++j) x[j] = xs[t * kScanRows + warp * 4 + j];
-            const float decay = KIND == kScanMamba2 ? one[kScanStage + t] : 0.0f;
+            const float decay = KIND == kScanMamba2 ? one[kScanStage + t] : 0.0f, step = KIND == kScanMamba2 ? one[t] : 1.0f;
 #pragma unroll
             for (int e = 0; e < kScanMaxPer; ++e) {
                 const int i = lane + 32 * e;
                 if (i < n) {
-                    const float k = ks[t * n + i], q = qs[t * n + i], d = KIND == kScanMamba2 ? decay : as[t * n + i];
+                    const float k = ks[t * n + i] * step, q = qs[t * n + i], d = KIND == kScanMamba2 ? decay : as[t * n + i];
 #pragma unroll
                     for (int j = 0; j < 4; ++j) {
                         s[j][e] = d * s[j][e] + k * x[j];

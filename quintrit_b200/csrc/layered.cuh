@@ -480,14 +480,14 @@ int layered_mixer(quintrit_b200_decoder* d, size_t li, int n, const LayeredTarge
         const dim3 grid(l.heads, (l.vdim + kScanRows - 1) / kScanRows, seqs);
         if (sizeof(T) == 2 && tokens > kChunkT / 2 && chunk_scan_rows(a.n) != 0) return layered_chunk_scan(d, l, a);
         if (l.kind == MixerKind::kMamba2) {
-            gated_scan_kernel<kScanMamba2><<<grid, kScanThreads, scan_smem(a.n), s>>>(a);
+            launch_dependent(gated_scan_kernel<kScanMamba2>, grid, kScanThreads, scan_smem(a.n), s, a);
             QTB_LAUNCH_CHECK();
             if (tokens > 1) {
                 conv_tail_kernel<<<(l.conv_dim() + 255) / 256, 256, 0, s>>>(a);
                 QTB_LAUNCH_CHECK();
             }
         } else {
-            gated_scan_kernel<kScanHgrn2><<<grid, kScanThreads, scan_smem(a.n), s>>>(a);
+            launch_dependent(gated_scan_kernel<kScanHgrn2>, grid, kScanThreads, scan_smem(a.n), s, a);
             QTB_LAUNCH_CHECK();
         }
         return QUINTRIT_OK;
@@ -501,7 +501,7 @@ int layered_mixer(quintrit_b200_decoder* d, size_t li, int n, const LayeredTarge
     const size_t smem = pooled_attn_smem(a.dim_pad, a.vdim_pad, sizeof(T));
     if (tokens == 1) {  // a token at a time: the attention kernel appends to the cache itself
         a.splits = pooled_splits(l, d->ctx, n, y.model->sm_count);
-        pooled_attention_kernel<T, true><<<dim3(hg, a.splits, seqs), kPaThreads, smem, s>>>(a);
+        launch_dependent(pooled_attention_kernel<T, true>, dim3(hg, a.splits, seqs), kPaThreads, smem, s, a);
         QTB_LAUNCH_CHECK();
         return QUINTRIT_OK;
     }
@@ -570,7 +570,7 @@ int layered_layers(quintrit_b200_decoder* d, const uint32_t* tokens, int n, cons
                 for (int k = 0; k < st[i].n_seg; ++k) units += (st[i].seg[k].rows + 1) / 2;
             }
             const int warps = kProjectThreads / 32;
-            norm_project_kernel<T><<<std::min((units + warps - 1) / warps, 4 * m.sm_count), kProjectThreads, size_t(n_stack) * wp * sizeof(float), s>>>(a);
+            launch_dependent(norm_project_kernel<T>, dim3(std::min((units + warps - 1) / warps, 4 * m.sm_count)), kProjectThreads, size_t(n_stack) * wp * sizeof(float), s, a);
             QTB_LAUNCH_CHECK();
             if ((rc = layered_mixer<T>(d, li, n, tg)) != QUINTRIT_OK) return rc;
             FinishProjectArgs f{};
@@ -578,7 +578,7 @@ int layered_layers(quintrit_b200_decoder* d, const uint32_t* tokens, int n, cons
             f.o = l.o.w, f.o_pitch = l.o.pitch;
             if (l.spec.ff > 0) f.m = y.m, f.down = l.down.w, f.down_pitch = l.down.pitch;
             if (l.spec.gated_residual) f.gate1 = y.g1, f.gate2 = y.g2;
-            finish_project_kernel<T><<<std::min((W + warps - 1) / warps, 4 * m.sm_count), kProjectThreads, (size_t(f.o_pitch) + f.down_pitch) * sizeof(float), s>>>(f);
+            launch_dependent(finish_project_kernel<T>, dim3(std::min((W + warps - 1) / warps, 4 * m.sm_count)), kProjectThreads, (size_t(f.o_pitch) + f.down_pitch) * sizeof(float), s, f);
             QTB_LAUNCH_CHECK();
             continue;
         }
@@ -616,7 +616,7 @@ int layered_head(quintrit_b200_decoder* d, int row, float* logits) {
     a.stack[0] = layered_stack(m.head);
     a.stack[0].n_seg = 1, a.stack[0].seg[0] = DenseSeg{0, m.spec.vocab, kSegPlain, m.spec.vocab, logits, nullptr, nullptr};
     const int warps = kProjectThreads / 32;
-    norm_project_kernel<T><<<std::min((m.spec.vocab / 2 + warps) / warps, 4 * m.sm_count), kProjectThreads, size_t(m.head.pitch) * sizeof(float), d->stream>>>(a);
+    launch_dependent(norm_project_kernel<T>, dim3(std::min((m.spec.vocab / 2 + warps) / warps, 4 * m.sm_count)), kProjectThreads, size_t(m.head.pitch) * sizeof(float), d->stream, a);
     QTB_LAUNCH_CHECK();
     return QUINTRIT_OK;
 }

@@ -76,11 +76,11 @@ __global__ void __launch_bounds__(256) pooled_append_kernel(const __grid_constan
     }
 }
 
-constexpr int kPaThreads = 128, kPaTile = 64, kPaHeads = 8;  // keys per tile; query heads per block
+constexpr int kPaThreads = 256, kPaTile = 64, kPaHeads = 8;  // keys per tile; query heads per block
 
 inline size_t pooled_attn_smem(int dim_pad, int vdim_pad, int elem) {
     return size_t(kPaHeads) * dim_pad * 4 + size_t(kPaTile) * (size_t(dim_pad) * elem + 16) + size_t(kPaTile) * vdim_pad * elem + size_t(kPaHeads) * kPaTile * 4 +
-           size_t(4) * kPaHeads * 256 * 4 + 64;
+           size_t(kPaHeads) * 2 * kPaThreads * 4 + 64;
 }
 
 __device__ __forceinline__ float dot_key(const bf16* k, const float* q, int dim_pad) {
@@ -104,12 +104,17 @@ __device__ __forceinline__ float dot_key(const float* k, const float* q, int dim
     return s;
 }
 
+__device__ __forceinline__ void attn_copy16(void* dst, const void* src) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(static_cast<uint32_t>(__cvta_generic_to_shared(dst))), "l"(src) : "memory");
+}
+
 // One query position per block: up to eight query heads of one kv head over a share (split) of the visible keys; the last block of a
 // position and head group to finish adds the shares up. A decode step (APPEND) also stores its own key and value, and the mean of a block
 // that this token completes. grid: (kv heads * head groups, splits, tokens or sequences)
 template <typename T, bool APPEND>
 __global__ void __launch_bounds__(kPaThreads) pooled_attention_kernel(const __grid_constant__ PooledAttnArgs a) {
-    extern __shared__ float pa_sm[];
+    extern __shared__ __align__(16) float pa_sm[];
+    pdl_trigger();
     __shared__ float m_run[kPaHeads], l_run[kPaHeads], fac[kPaHeads];
     __shared__ bool last_block;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -124,12 +129,8 @@ __global__ void __launch_bounds__(kPaThreads) pooled_attention_kernel(const __gr
     unsigned char* kt = reinterpret_cast<unsigned char*>(qs + kPaHeads * dp);            // [kPaTile][kpitch]
     T* vt = reinterpret_cast<T*>(kt + kPaTile * kpitch);                                 // [kPaTile][vp]
     float* sc = reinterpret_cast<float*>(vt + kPaTile * vp);                             // [kPaHeads][kPaTile]
-    float* red = sc + kPaHeads * kPaTile;                                                // [key groups][kPaHeads][vcols]
+    float* red = sc + kPaHeads * kPaTile;                                                // [key groups][kPaHeads][vstride]
     const float* prow = a.p + size_t(z) * a.ld;
-    for (int i = tid; i < kPaHeads * dp; i += kPaThreads) {
-        const int h = i / dp, c = i % dp;
-        qs[i] = h < nh && c < a.dim ? round_to<T>(prow[(h0 + h) * a.dim + c]) : 0.0f;
-    }
     if (tid < kPaHeads) m_run[tid] = -INFINITY, l_run[tid] = 0.0f;
     const int nb = pooled_blocks_seen(pos, a.window, a.pool), lo = max(0, pos - a.window + 1), total = nb + pos - lo + 1;
     const int per = ((total + a.splits - 1) / a.splits + kPaTile - 1) / kPaTile * kPaTile;
@@ -141,27 +142,44 @@ __global__ void __launch_bounds__(kPaThreads) pooled_attention_kernel(const __gr
     const int src_k = a.heads * a.dim + kvh * a.dim, src_v = a.heads * a.dim + a.kv_heads * a.dim + kvh * a.vdim;
     // value columns: thread (key group kg, column vc); columns beyond 128 take a second turn
     const int vcols = vp <= 32 ? 32 : vp <= 64 ? 64 : 128, kgroups = kPaThreads / vcols, kg = tid / vcols, vc = tid % vcols;
+    const int vstride = vp > 128 ? 256 : vcols;
     float acc[kPaHeads][2] = {};
-    for (int t0 = begin; t0 < end; t0 += kPaTile) {
+    constexpr int kPer = 16 / sizeof(T);
+    const int kvec = dp / kPer, vvec = vp / kPer;
+    auto fetch = [&](int t0) {  // keys and values of a tile; a decode step's own token is not in the cache yet
         const int nt = min(kPaTile, end - t0);
-        __syncthreads();
-        constexpr int kPer = 16 / sizeof(T);
-        const int kvec = dp / kPer, vvec = vp / kPer;
+#pragma unroll 4
         for (int i = tid; i < nt * (kvec + vvec); i += kPaThreads) {
             const int r = i / (kvec + vvec), c = i % (kvec + vvec), key = t0 + r;
-            const bool pooled = key < nb;
+            const bool pooled = key < nb, is_k = c < kvec;
             const int token = lo + key - nb;
+            if (APPEND && !pooled && token == pos) continue;
             const size_t row = size_t(pooled ? key : token % a.cache.ring) * a.kv_heads;
-            const bool is_k = c < kvec;
-            T* dst = is_k ? reinterpret_cast<T*>(kt + r * kpitch) + c * kPer : vt + r * vp + (c - kvec) * kPer;
-            if (APPEND && !pooled && token == pos) {  // this step's own token: from the projections
-                const int e0 = (is_k ? c : c - kvec) * kPer, width = is_k ? a.dim : a.vdim, src = is_k ? src_k : src_v;
-                for (int e = 0; e < kPer; ++e) dst[e] = to_storage<T>(e0 + e < width ? prow[src + e0 + e] : 0.0f);
-            } else {
-                const T* from = is_k ? (pooled ? pool_k : ring_k) + row * dp + c * kPer : (pooled ? pool_v : ring_v) + row * vp + (c - kvec) * kPer;
-                *reinterpret_cast<uint4*>(dst) = *reinterpret_cast<const uint4*>(from);
+            const T* from = is_k ? (pooled ? pool_k : ring_k) + row * dp + c * kPer : (pooled ? pool_v : ring_v) + row * vp + (c - kvec) * kPer;
+            attn_copy16(is_k ? static_cast<void*>(kt + r * kpitch + c * 16) : static_cast<void*>(vt + r * vp + (c - kvec) * kPer), from);
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    if (begin < end) fetch(begin);  // (cached by earlier steps, or by the launch before where this is a prompt's)
+    pdl_wait();
+    for (int i = tid; i < kPaHeads * dp; i += kPaThreads) {
+        const int h = i / dp, c = i % dp;
+        qs[i] = h < nh && c < a.dim ? round_to<T>(prow[(h0 + h) * a.dim + c]) : 0.0f;
+    }
+    for (int t0 = begin; t0 < end; t0 += kPaTile) {
+        const int nt = min(kPaTile, end - t0);
+        if (t0 != begin) {
+            __syncthreads();
+            fetch(t0);
+        }
+        if (APPEND && pos - lo + nb >= t0 && pos - lo + nb < t0 + nt) {  // this step's own token: from the projections
+            const int r = pos - lo + nb - t0;
+            for (int e = tid; e < dp + vp; e += kPaThreads) {
+                if (e < dp) reinterpret_cast<T*>(kt + r * kpitch)[e] = to_storage<T>(e < a.dim ? prow[src_k + e] : 0.0f);
+                else vt[r * vp + e - dp] = to_storage<T>(e - dp < a.vdim ? prow[src_v + e - dp] : 0.0f);
             }
         }
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();
         for (int i = tid; i < kPaTile * nh; i += kPaThreads) {
             const int r = i % kPaTile, h = i / kPaTile;
@@ -199,14 +217,14 @@ __global__ void __launch_bounds__(kPaThreads) pooled_attention_kernel(const __gr
 #pragma unroll
     for (int h = 0; h < kPaHeads; ++h)
         if (h < nh) {
-            red[(kg * kPaHeads + h) * 256 + vc] = acc[h][0];
-            if (vcols == 128) red[(kg * kPaHeads + h) * 256 + 128 + vc] = acc[h][1];
+            red[(kg * kPaHeads + h) * vstride + vc] = acc[h][0];
+            if (vstride == 256) red[(kg * kPaHeads + h) * vstride + 128 + vc] = acc[h][1];
         }
     __syncthreads();
     for (int i = tid; i < nh * a.vdim; i += kPaThreads) {
         const int h = i / a.vdim, v = i % a.vdim, head = h0 + h;
         float s = 0.0f;
-        for (int g = 0; g < kgroups; ++g) s += red[(g * kPaHeads + h) * 256 + v];
+        for (int g = 0; g < kgroups; ++g) s += red[(g * kPaHeads + h) * vstride + v];
         if (a.splits == 1) {
             const float gate = a.head_gate ? sigmoid_f(prow[a.heads * a.dim + a.kv_heads * (a.dim + a.vdim) + head]) : 1.0f;
             a.y[size_t(z) * a.heads * a.vdim + size_t(head) * a.vdim + v] = s / l_run[h] * gate;
@@ -244,20 +262,54 @@ __global__ void __launch_bounds__(kPaThreads) pooled_attention_kernel(const __gr
     if (!last_block) return;
     if (tid == 0) *counter = 0;
     __threadfence();
-    for (int i = tid; i < nh * a.vdim; i += kPaThreads) {
-        const int head = h0 + i / a.vdim, v = i % a.vdim;
-        const size_t at = (size_t(z) * a.heads + head) * a.splits;
-        float m = -INFINITY, l = 0.0f, s = 0.0f;
-        for (int k = 0; k < a.splits; ++k) m = fmaxf(m, __ldcg(a.part_ml + (at + k) * 2));
-        for (int k = 0; k < a.splits; ++k) {
-            const float mk = __ldcg(a.part_ml + (at + k) * 2);
-            if (mk == -INFINITY) continue;  // an empty share
-            const float f = expf(mk - m);
-            l = fmaf(__ldcg(a.part_ml + (at + k) * 2 + 1), f, l);
-            s = fmaf(__ldcg(a.part_acc + (at + k) * a.vdim + v), f, s);
+    // factors of the shares, then the sums
+    float* part = sc;  // [nh][splits]; kPaHeads x kPaTile floats hold at most 64 shares a head
+    for (int h = warp; h < nh; h += kPaThreads / 32) {
+        const float* ml = a.part_ml + (size_t(z) * a.heads + h0 + h) * a.splits * 2;
+        float mk[2], lk[2], m = -INFINITY;
+#pragma unroll
+        for (int k = 0; k < 2; ++k) {
+            const int i = lane + 32 * k;
+            mk[k] = i < a.splits ? __ldcg(ml + 2 * i) : -INFINITY, lk[k] = i < a.splits ? __ldcg(ml + 2 * i + 1) : 0.0f;
+            m = fmaxf(m, mk[k]);
         }
-        const float gate = a.head_gate ? sigmoid_f(prow[a.heads * a.dim + a.kv_heads * (a.dim + a.vdim) + head]) : 1.0f;
-        a.y[size_t(z) * a.heads * a.vdim + size_t(head) * a.vdim + v] = s / l * gate;
+        for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
+        float l = 0.0f;
+#pragma unroll
+        for (int k = 0; k < 2; ++k) {
+            mk[k] = mk[k] == -INFINITY ? 0.0f : expf(mk[k] - m);  // an empty share counts nothing
+            l = fmaf(lk[k], mk[k], l);
+        }
+        l = warp_sum(l);
+        const float gate = a.head_gate ? sigmoid_f(prow[a.heads * a.dim + a.kv_heads * (a.dim + a.vdim) + h0 + h]) : 1.0f;
+#pragma unroll
+        for (int k = 0; k < 2; ++k)
+            if (lane + 32 * k < a.splits) part[h * kPaTile + lane + 32 * k] = mk[k] * gate / l;
+    }
+    __syncthreads();
+    const float* acc0 = a.part_acc + (size_t(z) * a.heads + h0) * a.splits * a.vdim;
+    float* y0 = a.y + size_t(z) * a.heads * a.vdim + size_t(h0) * a.vdim;
+    if (a.vdim % 4 == 0) {
+        const int quads = a.vdim / 4;
+        for (int i = tid; i < nh * quads; i += kPaThreads) {
+            const int h = i / quads, v = i % quads * 4;
+            float4 s = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll 12
+            for (int k = 0; k < a.splits; ++k) {
+                const float4 p = __ldcg(reinterpret_cast<const float4*>(acc0 + (size_t(h) * a.splits + k) * a.vdim + v));
+                const float f = part[h * kPaTile + k];
+                s.x = fmaf(p.x, f, s.x), s.y = fmaf(p.y, f, s.y), s.z = fmaf(p.z, f, s.z), s.w = fmaf(p.w, f, s.w);
+            }
+            *reinterpret_cast<float4*>(y0 + h * a.vdim + v) = s;
+        }
+        return;
+    }
+    for (int i = tid; i < nh * a.vdim; i += kPaThreads) {
+        const int h = i / a.vdim, v = i % a.vdim;
+        float s = 0.0f;
+#pragma unroll 8
+        for (int k = 0; k < a.splits; ++k) s = fmaf(__ldcg(acc0 + (size_t(h) * a.splits + k) * a.vdim + v), part[h * kPaTile + k], s);
+        y0[h * a.vdim + v] = s;
     }
 }
 

@@ -999,6 +999,27 @@ extern "C" int quintrit_generate_params_default(quintrit_generate_params_t* para
 }
 
 namespace {
+// Sampling runs on the device where the candidates are cut to at most 1024 (top_k): the logits then never leave the GPU and the
+// sampled token is the next step's input there, as the greedy choice is. Other settings sample on the host from the logits.
+int rt_begin_sampling(quintrit_session* s, const quintrit_generate_params_t& prm, const RtSampler& sampler, bool* on_device) {
+    *on_device = !sampler.greedy() && prm.top_k >= 1 && prm.top_k <= static_cast<uint32_t>(kSampleMaxK) && prm.top_k < s->model->data.shape.vocab && s->dec->tp_world == 1 &&
+                 std::getenv("QUINTRIT_B200_HOST_SAMPLER") == nullptr;
+    if (!*on_device) return QUINTRIT_OK;
+    DeviceGuard dg(s->dec->device);
+    if (s->dec->d_rng == nullptr) {
+        int rc = dev_alloc(s->dec, &s->dec->d_rng, 1);
+        if (rc != QUINTRIT_OK) return rc;
+    }
+    QTB_CUDA(cudaMemcpyAsync(s->dec->d_rng, &sampler.state, sizeof sampler.state, cudaMemcpyHostToDevice, s->dec->stream));
+    QTB_CUDA(cudaStreamSynchronize(s->dec->stream));  // (the state is a local of the caller)
+    return QUINTRIT_OK;
+}
+int rt_check_params(const quintrit_generate_params_t& prm) {
+    if (!(prm.temperature >= 0.0f) || !std::isfinite(prm.temperature)) return fail(QUINTRIT_ERR_INVALID_ARGUMENT, "temperature must be finite and not negative");
+    if (!(prm.top_p > 0.0f && prm.top_p <= 1.0f)) return fail(QUINTRIT_ERR_INVALID_ARGUMENT, "top_p must be in (0, 1]");
+    return QUINTRIT_OK;
+}
+
 // The generation loop of quintrit-c/src/runtime.rs:382-520 over a decoder on the device. Greedy decoding reads back only the
 // token the device chose; sampling reads the logits of every step and samples on the host with the reference's sampler.
 int rt_generate(quintrit_session* s, const std::string& prompt, const quintrit_generate_params_t& prm, const std::vector<std::string>& stops, quintrit_token_callback cb,
@@ -1028,25 +1049,15 @@ int rt_generate(quintrit_session* s, const std::string& prompt, const quintrit_g
         s->cached.resize(common);
     }
     RtSampler sampler(prm.temperature, prm.top_k, prm.top_p, prm.seed);
-    // Sampling runs on the device where the candidates are cut to at most 1024 (top_k): the logits then never leave the GPU and the
-    // sampled token is the next step's input there, as the greedy choice is. Other settings sample on the host from the logits.
     RtDeviceSampling dev_sampling{prm.temperature, prm.top_p, static_cast<int>(prm.top_k)};
-    const bool on_device_sampling = !sampler.greedy() && prm.top_k >= 1 && prm.top_k <= static_cast<uint32_t>(kSampleMaxK) && prm.top_k < m.data.shape.vocab &&
-                                    s->dec->tp_world == 1 && std::getenv("QUINTRIT_B200_HOST_SAMPLER") == nullptr;
+    bool on_device_sampling = false;
+    int rc = rt_begin_sampling(s, prm, sampler, &on_device_sampling);
+    if (rc != QUINTRIT_OK) return rc;
     const RtDeviceSampling* dsp = on_device_sampling ? &dev_sampling : nullptr;
-    if (on_device_sampling) {
-        DeviceGuard dg(s->dec->device);
-        if (s->dec->d_rng == nullptr) {
-            int rc0 = dev_alloc(s->dec, &s->dec->d_rng, 1);
-            if (rc0 != QUINTRIT_OK) return rc0;
-        }
-        QTB_CUDA(cudaMemcpyAsync(s->dec->d_rng, &sampler.state, sizeof sampler.state, cudaMemcpyHostToDevice, s->dec->stream));
-        QTB_CUDA(cudaStreamSynchronize(s->dec->stream));  // (the state is a local of this call)
-    }
     const bool greedy = sampler.greedy() || on_device_sampling;  // the device chooses: only the token comes back
     const bool llama_like = m.arch == "bitnet" || m.arch == "llama";
     uint32_t device_choice = 0;
-    int rc = rt_feed(s, tokens.data() + common, tokens.size() - common, pos0, !greedy, &device_choice, dsp);
+    rc = rt_feed(s, tokens.data() + common, tokens.size() - common, pos0, !greedy, &device_choice, dsp);
     if (rc != QUINTRIT_OK) return rc;
     uint32_t pos = base + static_cast<uint32_t>(tokens.size());
     std::string full, pending;
@@ -1142,8 +1153,7 @@ extern "C" int quintrit_session_generate(quintrit_session_t* session, const char
             prm = *params;
         }
         if (prm.flags & ~uint32_t(QUINTRIT_GENERATE_KEEP_CONTEXT)) return fail(QUINTRIT_ERR_INVALID_ARGUMENT, "params.flags has unknown bits set: 0x%x", prm.flags);
-        if (!(prm.temperature >= 0.0f) || !std::isfinite(prm.temperature)) return fail(QUINTRIT_ERR_INVALID_ARGUMENT, "temperature must be finite and not negative");
-        if (!(prm.top_p > 0.0f && prm.top_p <= 1.0f)) return fail(QUINTRIT_ERR_INVALID_ARGUMENT, "top_p must be in (0, 1]");
+        if ((rc = rt_check_params(prm)) != QUINTRIT_OK) return rc;
         if (prm.stop_count > 64) return fail(QUINTRIT_ERR_INVALID_ARGUMENT, "at most 64 stop sequences");
         if (prm.stop_count != 0 && prm.stop_sequences == nullptr) return fail(QUINTRIT_ERR_NULL_POINTER, "stop_sequences is NULL");
         std::vector<std::string> stops;
@@ -1232,6 +1242,40 @@ extern "C" int quintrit_session_generate_tokens(quintrit_session_t* session, con
         session->cached.clear();  // the loop ran on the device: the host has no record of what the cache holds now
         session->logits_valid = false;
         *out_count = max_new;
+        return ok();
+    });
+}
+
+extern "C" int quintrit_b200_session_sample_tokens(quintrit_session_t* session, const uint32_t* prompt, size_t prompt_len, const quintrit_generate_params_t* params, uint32_t* out,
+                                                   size_t out_capacity, size_t* out_count) {
+    return guard([&]() -> int {
+        int rc = rt_check(session, kMagicSession, "session");
+        if (rc != QUINTRIT_OK || (rc = rt_struct(params, "params")) != QUINTRIT_OK || (rc = rt_check_params(*params)) != QUINTRIT_OK) return rc;
+        if (prompt == nullptr || out == nullptr || out_count == nullptr) return fail(QUINTRIT_ERR_NULL_POINTER, "a pointer is NULL");
+        *out_count = 0;
+        if (prompt_len == 0) return fail(QUINTRIT_ERR_INVALID_ARGUMENT, "the prompt must not be empty");
+        if (out_capacity < params->max_tokens) return fail(QUINTRIT_ERR_BUFFER_TOO_SMALL, "out holds %zu ids, %u are needed", out_capacity, params->max_tokens);
+        RtSessionLock lk(session);
+        if ((rc = lk.check()) != QUINTRIT_OK) return rc;
+        const uint32_t base = (params->flags & QUINTRIT_GENERATE_KEEP_CONTEXT) ? session->dec->host_pos : 0;
+        for (size_t i = 0; i < prompt_len; ++i)
+            if (prompt[i] >= static_cast<uint32_t>(session->dec->vocab_full)) return fail(QUINTRIT_ERR_INVALID_ARGUMENT, "token id %u is outside the vocabulary of %d", prompt[i], session->dec->vocab_full);
+        if (size_t(base) + prompt_len > session->ctx) return fail(QUINTRIT_ERR_CONTEXT_OVERFLOW, "%zu prompt tokens do not fit: the context window holds %u tokens and %u are already used", prompt_len, session->ctx, base);
+        if (base == 0) session->dec->host_pos = 0;
+        RtSampler sampler(params->temperature, params->top_k, params->top_p, params->seed);
+        RtDeviceSampling dev{params->temperature, params->top_p, static_cast<int>(params->top_k)};
+        bool on_device = false;
+        if ((rc = rt_begin_sampling(session, *params, sampler, &on_device)) != QUINTRIT_OK) return rc;
+        const RtDeviceSampling* dsp = on_device ? &dev : nullptr;
+        const bool chosen = sampler.greedy() || on_device;
+        uint32_t choice = 0, pos = base + static_cast<uint32_t>(prompt_len);
+        if ((rc = rt_feed(session, prompt, prompt_len, base, !chosen, &choice, dsp)) != QUINTRIT_OK) return rc;
+        DeviceGuard g(session->dec->device);
+        for (uint32_t step = 0; step < params->max_tokens; ++step) {
+            out[(*out_count)++] = chosen ? choice : sampler.sample(session->logits);
+            if (step + 1 == params->max_tokens || pos >= session->ctx) break;
+            if ((rc = rt_forward(session, out[step], pos++, !chosen, &choice, chosen, dsp)) != QUINTRIT_OK) return rc;
+        }
         return ok();
     });
 }

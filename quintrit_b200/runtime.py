@@ -108,6 +108,7 @@ def _lib() -> C.CDLL:
     l.quintrit_session_generate.argtypes = [vp, C.c_char_p, _sz, C.POINTER(_GenerateParams), TOKEN_CALLBACK, vp, C.c_char_p, _sz, C.POINTER(_sz),
                                             C.POINTER(_GenerateResult)]
     l.quintrit_session_feed_tokens.argtypes = [vp, u32p, _sz, C.c_uint32]
+    l.quintrit_b200_session_sample_tokens.argtypes = [vp, u32p, _sz, C.POINTER(_GenerateParams), u32p, _sz, C.POINTER(_sz)]
     l.quintrit_b200_session_feed_at.argtypes = [vp, u32p, _sz, C.c_uint32, u32p, _sz, C.POINTER(C.c_float), _sz]
     l.quintrit_session_logits.argtypes = [vp, C.POINTER(C.c_float), _sz]
     l.quintrit_session_generate_tokens.argtypes = [vp, u32p, _sz, _sz, u32p, _sz, C.POINTER(_sz)]
@@ -258,6 +259,16 @@ class Session:
         a = _ids(prompt_ids)
         out, n = np.zeros(max_new, np.uint32), _sz(0)
         _check(self._l.quintrit_session_generate_tokens(self._s, _u32p(a), a.size, max_new, _u32p(out), out.size, C.byref(n)))
+        return out[:n.value]
+
+    def sample_tokens(self, prompt_ids, max_new: int, *, temperature: float = 0.8, top_k: int = 40, top_p: float = 0.9, seed: int = 0, keep_context: bool = False) -> np.ndarray:
+        """Tokens after the prompt, sampled (greedy with ``temperature=0``); fewer than ``max_new`` where the context ends."""
+        p = _GenerateParams()
+        _check(self._l.quintrit_generate_params_default(C.byref(p)))
+        p.max_tokens, p.top_k, p.temperature, p.top_p, p.seed, p.flags = max_new, top_k, temperature, top_p, seed, 1 if keep_context else 0
+        a = _ids(prompt_ids)
+        out, n = np.zeros(max_new, np.uint32), _sz(0)
+        _check(self._l.quintrit_b200_session_sample_tokens(self._s, _u32p(a), a.size, C.byref(p), _u32p(out), out.size, C.byref(n)))
         return out[:n.value]
 
     def close(self) -> None:

@@ -137,11 +137,14 @@ def needle(window, pool, width=160, vocab=40, seed=5):
     h = plain.rms_norm(w["embed"].astype(np.float64), w["l0.norm1"], config["norm"]["eps"])
     u = np.random.default_rng(seed).normal(0, 1, 32)
     u /= np.linalg.norm(u)
+    w["l0.mix.o"] *= 12.0
+    w["l0.rg1.b"][:] = 4.0
     w["l0.mix.q"] *= 0.05
     w["l0.mix.k"] *= 0.05
     alpha = (4.5 * pool) ** 0.5 if pool > 1 else 3.0  # a score of 4.5 through the mean of a block
-    w["l0.mix.q"] += alpha * np.outer(np.tile(u, 2), h[1] / (h[1] @ h[1]))
-    w["l0.mix.k"] += alpha * np.outer(u, h[0] / (h[0] @ h[0]))
+    probe = np.linalg.pinv(h)  # column t answers 1 to token t and 0 to the others
+    w["l0.mix.q"] += alpha * np.outer(np.tile(u, 2), probe[:, 1])
+    w["l0.mix.k"] += alpha * np.outer(u, probe[:, 0])
     return config, {k: mf.bf16_bits(v) for k, v in w.items()}
 
 
@@ -166,7 +169,7 @@ def test_keys_just_inside_and_outside_the_window_and_its_blocks(tmp_path, window
                 if cut:
                     s.feed(ids[:cut])
                 check(s.feed(ids[cut:], [len(ids) - cut - 1]), want, dtype)
-    assert shown >= 12  # the needle is seen at many of these distances (and must not be at the others)
+    assert shown >= 20  # the needle is seen at many of these distances (and must not be at the others)
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
@@ -274,7 +277,7 @@ def test_greedy_and_sampled_generation_through_sessions(tmp_path):
     assert s.sample_tokens(prompt, 30, temperature=0.0).tolist() == want
     assert s.sample_tokens(prompt, 30, temperature=1.0, top_k=1).tolist() == want
     one, two = s.sample_tokens(prompt, 20, temperature=1.5, top_k=20, top_p=0.95, seed=7), s.sample_tokens(prompt, 20, temperature=1.5, top_k=20, top_p=0.95, seed=7)
-    assert one.tolist() == two.tolist() and one.tolist() != s.sample_tokens(prompt, 20, temperature=1.5, top_k=20, top_p=0.95, seed=8).tolist()
+    assert one.tolist() == two.tolist() and one.tolist() != s.sample_tokens(prompt, 20, temperature=1.5, top_k=20, top_p=0.95, seed=0x9E3779B97F4A7C15).tolist()
     fresh = model.new_session()
     row, state = fresh.feed(prompt, [len(prompt) - 1])[0], 7
     for t in one:
