@@ -656,7 +656,7 @@ def quantize_q8_0(x, device: int = 0):
 
 
 def gguf_describe(path: str) -> dict:
-    """Hyperparameters and tensor directory of a GGUF file as the library reads them (host only, no GPU)."""
+    """Hyperparameters and tensor directory of a GGUF file or a model folder as the library reads them (host only, no GPU)."""
     n = _sz(0)
     lib = load_library()
     rc = lib.quintrit_b200_gguf_describe(str(path).encode(), None, 0, C.byref(n))
@@ -673,7 +673,7 @@ def gguf_describe(path: str) -> dict:
             for f in fields:
                 if "=" in f:
                     k, v = f.split("=")
-                    t[k] = tuple(int(x) for x in v.split("x")) if k == "shape" else int(v)
+                    t[k] = tuple(int(x) for x in v.split("x")) if k == "shape" else int(v) if v.isdigit() else v
             tensors.append(t)
         else:
             out[key] = rest

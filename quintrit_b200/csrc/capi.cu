@@ -1464,12 +1464,14 @@ struct GgufModel {
 
 // A model folder (config.json + model.safetensors; the design is chosen by config.json).
 int load_model_folder(const char* path, uint32_t device, bool f32, GgufModel* out) {
-    cudaDeviceProp prop;
-    int rc = require_b200(static_cast<int>(device), &prop);
+    auto read = std::make_unique<LayeredFolder>();  // what can be said about the folder is said before the device is asked for
+    int rc = read_model_folder(path, &read->spec, &read->file);
     if (rc != QUINTRIT_OK) return rc;
+    cudaDeviceProp prop;
+    if ((rc = require_b200(static_cast<int>(device), &prop)) != QUINTRIT_OK) return rc;
     DeviceGuard g(static_cast<int>(device));
     out->device = device;
-    if ((rc = load_layered_model(path, static_cast<int>(device), f32, &out->layered)) != QUINTRIT_OK) return rc;
+    if ((rc = load_layered_model(*read, static_cast<int>(device), f32, &out->layered)) != QUINTRIT_OK) return rc;
     const LayeredSpec& s = out->layered->spec;
     GgufModelShape& m = out->shape;
     m.arch = s.design, m.arch_id = QUINTRIT_B200_ARCH_LAYERED;
@@ -1672,6 +1674,18 @@ extern "C" int quintrit_b200_decoder_info(const quintrit_b200_decoder_t* decoder
 extern "C" int quintrit_b200_gguf_describe(const char* path, char* out, size_t out_capacity, size_t* out_needed) {
     return guard([&]() -> int {
         if (path == nullptr || out_needed == nullptr) return fail(QUINTRIT_ERR_NULL_POINTER, "a pointer is NULL");
+        struct stat st;
+        if (::stat(path, &st) == 0 && S_ISDIR(st.st_mode)) {
+            LayeredSpec spec;
+            SafetensorsFile file;
+            int rc = read_model_folder(path, &spec, &file);
+            if (rc != QUINTRIT_OK) return rc;
+            const std::string text = describe_layered(spec, file);
+            *out_needed = text.size() + 1;
+            if (out == nullptr || out_capacity < text.size() + 1) return fail(QUINTRIT_ERR_BUFFER_TOO_SMALL, "out holds %zu bytes, %zu are needed", out_capacity, text.size() + 1);
+            std::memcpy(out, text.c_str(), text.size() + 1);
+            return ok();
+        }
         GgufFile g;
         std::string why;
         const int rc_open = g.open(path, why);

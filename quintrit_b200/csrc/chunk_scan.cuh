@@ -55,6 +55,8 @@ inline size_t chunk_work(char* base, bool mamba, int heads, int vdim, int n, int
 }
 
 // mamba2: convolution and silu of every channel into xs and bc. grid: (padded channels / 128, chunks); a thread takes a channel of 16 tokens.
+// TAPS: taps of the convolution where they are few enough to keep their inputs in registers, 0 for any number.
+template <int TAPS>
 __global__ void __launch_bounds__(128) ssd_conv_kernel(const __grid_constant__ ScanArgs a, const __grid_constant__ ChunkWork w) {
     const int c = blockIdx.x * 128 + threadIdx.x, nx = a.heads * w.v_pad, nbc = 2 * a.groups * w.rows, inner = a.heads * a.vdim, channels = inner + 2 * a.groups * a.n;
     if (c >= nx + nbc) return;
@@ -68,8 +70,32 @@ __global__ void __launch_bounds__(128) ssd_conv_kernel(const __grid_constant__ S
     const size_t step = c < nx ? nx : nbc;
     const uint32_t pos0 = seq_position(a.seq, a.pos, 0);
     const float* ring = a.conv;
+    const int t0 = blockIdx.y * kChunkT;
+    if (TAPS > 0) {
+        constexpr int kBack = TAPS > 0 ? TAPS - 1 : 0;
+        float u[kChunkT + kBack], wt[TAPS > 0 ? TAPS : 1];
+        const int c0 = max(real, 0);
+        const float bias = a.conv_b[c0];
+#pragma unroll
+        for (int k = 0; k < TAPS; ++k) wt[k] = a.conv_w[size_t(c0) * TAPS + k];
+#pragma unroll
+        for (int i = 0; i < kChunkT + kBack; ++i) {  // all inputs in flight
+            const int t = t0 + i - kBack;
+            const bool there = real >= 0 && t < a.tokens && static_cast<int>(pos0) + t >= 0;
+            const float* src = t >= 0 ? a.p + size_t(t) * a.ld + inner + c0 : ring + size_t((pos0 + t) % TAPS) * channels + c0;
+            u[i] = there ? *src : 0.0f;
+        }
+#pragma unroll
+        for (int i = 0; i < kChunkT; ++i) {
+            float s = bias;
+#pragma unroll
+            for (int k = 0; k < TAPS; ++k) s = fmaf(wt[k], u[i + k], s);
+            out[size_t(t0 + i) * step] = __float2bfloat16_rn(real >= 0 && t0 + i < a.tokens ? silu_f(s) : 0.0f);
+        }
+        return;
+    }
     for (int i = 0; i < kChunkT; ++i) {
-        const int t = blockIdx.y * kChunkT + i;
+        const int t = t0 + i;
         out[size_t(t) * step] = __float2bfloat16_rn(real >= 0 && t < a.tokens ? conv_silu(a, ring, t, t, pos0 + t, real, channels, inner) : 0.0f);
     }
 }
@@ -111,20 +137,36 @@ __global__ void __launch_bounds__(128) hgrn_prep_kernel(const __grid_constant__ 
     extern __shared__ float prep_sm[];
     const int head = blockIdx.x, chunk = blockIdx.y, chunks = gridDim.y, tid = threadIdx.x, n = a.n, rows = w.rows;
     float *q = prep_sm, *k = q + kChunkT * rows, *f = k + kChunkT * rows;
-    for (int i = tid; i < kChunkT * rows; i += 128) {
-        const int t = chunk * kChunkT + i / rows, d = i % rows;
-        float qv = 0.0f, kv = 0.0f, fv = 1.0f;
-        if (t < a.tokens && d < n) {
-            const float* p = a.p + size_t(t) * a.ld + head * n + d;
-            const float z = p[a.heads * n] + a.f_bias[head * n + d], l = a.lower[head * n + d];
-            qv = silu_f(p[0]), fv = l + (1.0f - l) * sigmoid_f(z), kv = (1.0f - l) * sigmoid_f(-z);
+    for (int i0 = tid; i0 < kChunkT * rows; i0 += 128 * 4) {  // four elements' loads in flight (kChunkT * rows is a multiple of 512)
+        float qr[4], fr[4], low[4];
+        bool there[4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const int i = i0 + 128 * j, t = chunk * kChunkT + i / rows, d = i % rows, c = head * n + min(d, n - 1);
+            there[j] = t < a.tokens && d < n;
+            const float* p = a.p + size_t(min(t, a.tokens - 1)) * a.ld + c;
+            qr[j] = p[0], fr[j] = p[a.heads * n] + a.f_bias[c], low[j] = a.lower[c];
         }
-        q[i] = qv, k[i] = kv, f[i] = fv;
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const int i = i0 + 128 * j;
+            q[i] = there[j] ? silu_f(qr[j]) : 0.0f;
+            f[i] = there[j] ? low[j] + (1.0f - low[j]) * sigmoid_f(fr[j]) : 1.0f;
+            k[i] = there[j] ? (1.0f - low[j]) * sigmoid_f(-fr[j]) : 0.0f;
+        }
     }
-    for (int i = tid; i < kChunkT * w.v_pad; i += 128) {
-        const int t = chunk * kChunkT + i / w.v_pad, v = i % w.v_pad;
-        w.xs[(size_t(t) * a.heads + head) * w.v_pad + v] =
-            __float2bfloat16_rn(t < a.tokens && v < a.vdim ? a.p[size_t(t) * a.ld + 2 * a.heads * n + head * a.vdim + v] : 0.0f);
+    for (int i0 = tid; i0 < kChunkT * w.v_pad; i0 += 128 * 8) {  // (v_pad is a multiple of 64: whole turns of 1024)
+        float v[8];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+            const int i = i0 + 128 * j, t = chunk * kChunkT + i / w.v_pad, e = i % w.v_pad;
+            v[j] = t < a.tokens && e < a.vdim ? a.p[size_t(t) * a.ld + 2 * a.heads * n + head * a.vdim + e] : 0.0f;
+        }
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+            const int i = i0 + 128 * j, t = chunk * kChunkT + i / w.v_pad, e = i % w.v_pad;
+            w.xs[(size_t(t) * a.heads + head) * w.v_pad + e] = __float2bfloat16_rn(v[j]);
+        }
     }
     __syncthreads();
     const size_t at = size_t(head) * chunks + chunk;
@@ -229,20 +271,25 @@ __global__ void __launch_bounds__(128) chunk_scan_kernel(const __grid_constant__
             const float* tail = mat + 256;  // mamba2: dt, running sums; hgrn2: F_16
             uint32_t xv[4];                 // x as a B operand: columns 0..7 (0, 1) and 8..15 (2, 3); transposed it is the A operand {0, 2, 1, 3}
             load_frag_b(xv, xs + warp * 16, kVPitch);
-            float O[2][4] = {};
+            float O[2][4] = {}, P[3][2][4] = {};  // independent sums: a product waits for the one before it in the same registers
 #pragma unroll
             for (int ks = 0; ks < ROWS / 16; ++ks) {
                 uint32_t q[4], ql[4], h[4], l[4];
                 load_frag_a(q, ops + ks * 16, kPitch);
                 split_bf16(S[2 * ks][0], S[2 * ks][1], &h[0], &l[0]), split_bf16(S[2 * ks + 1][0], S[2 * ks + 1][1], &h[1], &l[1]);
                 split_bf16(S[2 * ks][2], S[2 * ks][3], &h[2], &l[2]), split_bf16(S[2 * ks + 1][2], S[2 * ks + 1][3], &h[3], &l[3]);
-                mma_16816(O[0], q, h[0], h[1]), mma_16816(O[1], q, h[2], h[3]);
-                mma_16816(O[0], q, l[0], l[1]), mma_16816(O[1], q, l[2], l[3]);
+                if (ks & 1) mma_16816(P[0][0], q, h[0], h[1]), mma_16816(P[0][1], q, h[2], h[3]);
+                else mma_16816(O[0], q, h[0], h[1]), mma_16816(O[1], q, h[2], h[3]);
+                mma_16816(P[1][0], q, l[0], l[1]), mma_16816(P[1][1], q, l[2], l[3]);
                 if (KIND == kScanHgrn2) {
                     load_frag_a(ql, ops + kChunkT * kPitch + ks * 16, kPitch);
-                    mma_16816(O[0], ql, h[0], h[1]), mma_16816(O[1], ql, h[2], h[3]);
+                    mma_16816(P[2][0], ql, h[0], h[1]), mma_16816(P[2][1], ql, h[2], h[3]);
                 }
             }
+#pragma unroll
+            for (int i = 0; i < 2; ++i)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) O[i][e] += P[0][i][e] + (P[1][i][e] + P[2][i][e]);
             // the sums inside the chunk
             float A[8];  // A rows t = g, g + 8 at s = 2c, 2c + 1 | 2c + 8, 2c + 9, in operand order
 #pragma unroll

@@ -171,7 +171,7 @@ struct NormProjectArgs {
 constexpr int kProjectThreads = 256;
 
 template <typename T>
-__global__ void __launch_bounds__(kProjectThreads) norm_project_kernel(NormProjectArgs a) {
+__global__ void __launch_bounds__(kProjectThreads, 4) norm_project_kernel(NormProjectArgs a) {
     extern __shared__ float act_smem[];
     __shared__ float red[kProjectThreads / 32];
     const int tid = threadIdx.x, token = blockIdx.y, pitch = a.stack[0].pitch;
@@ -192,27 +192,14 @@ __global__ void __launch_bounds__(kProjectThreads) norm_project_kernel(NormProje
     bool first = true;
     pdl_wait();
     float ss = 0.0f;
-    for (int i = tid; i < pitch; i += kProjectThreads) {
-        const float v = i < a.width ? x[i] : 0.0f;
-        act_smem[i] = v;  // (a thread keeps its own elements here until the sum is known)
-        ss += v * v;
-    }
+#pragma unroll 4
+    for (int i = tid; i < a.width; i += kProjectThreads) ss += x[i] * x[i];
     ss = block_sum(ss, red);
     const float inv = 1.0f / sqrtf(ss / static_cast<float>(a.width) + a.eps);
-    constexpr int kKeep = 16;
-    float keep[kKeep];
-#pragma unroll
-    for (int j = 0; j < kKeep; ++j) keep[j] = tid + j * kProjectThreads < pitch ? act_smem[tid + j * kProjectThreads] : 0.0f;
-    __syncthreads();
-    for (int s = 0; s < a.n_stack; ++s) {
-#pragma unroll
-        for (int j = 0; j < kKeep; ++j) {
-            const int i = tid + j * kProjectThreads;
-            if (i < pitch) act_smem[s * pitch + act_index<T>(i, pitch)] = i < a.width ? round_to<T>(keep[j] * inv * a.norm_w[s][i]) : 0.0f;
-        }
-        for (int i = tid + kKeep * kProjectThreads; i < pitch; i += kProjectThreads)
+    for (int s = 0; s < a.n_stack; ++s)
+#pragma unroll 4
+        for (int i = tid; i < pitch; i += kProjectThreads)
             act_smem[s * pitch + act_index<T>(i, pitch)] = i < a.width ? round_to<T>(x[i] * inv * a.norm_w[s][i]) : 0.0f;
-    }
     __syncthreads();
     for (int s = 0; s < a.n_stack; ++s)
         for (int k = 0; k < a.stack[s].n_seg; ++k) {
@@ -292,7 +279,7 @@ struct FinishProjectArgs {
 };
 
 template <typename T>
-__global__ void __launch_bounds__(kProjectThreads) finish_project_kernel(FinishProjectArgs a) {
+__global__ void __launch_bounds__(kProjectThreads, 4) finish_project_kernel(FinishProjectArgs a) {
     extern __shared__ float act_smem[];
     __shared__ float red[kProjectThreads / 32];
     const int tid = threadIdx.x, lane = tid & 31, token = blockIdx.y;

@@ -257,15 +257,14 @@ class LayeredLoader {
     }
 };
 
-inline int load_layered_model(const std::string& dir, int device, bool f32, std::shared_ptr<LayeredModel>* out) {
+inline int load_layered_model(const LayeredFolder& folder, int device, bool f32, std::shared_ptr<LayeredModel>* out) {
     auto m = std::make_shared<LayeredModel>();
-    SafetensorsFile file;
-    int rc = read_model_folder(dir, &m->spec, &file);
-    if (rc != QUINTRIT_OK) return rc;
+    m->spec = folder.spec;
+    int rc = QUINTRIT_OK;
     m->device = device, m->f32 = f32;
     QTB_CUDA(cudaSetDevice(device));
     QTB_CUDA(cudaDeviceGetAttribute(&m->sm_count, cudaDevAttrMultiProcessorCount, device));
-    if ((rc = LayeredLoader(m.get(), file).run()) != QUINTRIT_OK) return rc;
+    if ((rc = LayeredLoader(m.get(), folder.file).run()) != QUINTRIT_OK) return rc;
     *out = std::move(m);
     return QUINTRIT_OK;
 }
@@ -439,7 +438,9 @@ inline int layered_chunk_scan(quintrit_b200_decoder* d, const LayerSpec& l, cons
     chunk_work(d->lay->work, mamba, l.heads, l.vdim, a.n, l.groups, a.tokens, &w);
     const int chunks = chunk_count(a.tokens), rows = w.rows;
     if (mamba) {
-        ssd_conv_kernel<<<dim3((l.heads * w.v_pad + 2 * l.groups * rows + 127) / 128, chunks), 128, 0, s>>>(a, w);
+        const dim3 cgrid((l.heads * w.v_pad + 2 * l.groups * rows + 127) / 128, chunks);
+        auto conv = [&](auto kernel) { kernel<<<cgrid, 128, 0, s>>>(a, w); };
+        l.conv == 4 ? conv(ssd_conv_kernel<4>) : l.conv == 3 ? conv(ssd_conv_kernel<3>) : l.conv == 2 ? conv(ssd_conv_kernel<2>) : conv(ssd_conv_kernel<0>);
         QTB_LAUNCH_CHECK();
         ssd_gram_kernel<<<dim3(l.groups + 1, chunks), 256, size_t(2 * kChunkT) * (rows + 1) * sizeof(float), s>>>(a, w);
         QTB_LAUNCH_CHECK();

@@ -3,6 +3,7 @@
 // and constants; a design is an entry of kLayeredDesigns: it names its config keys and tensors and fills the description.
 #pragma once
 #include <cstdint>
+#include <cstdio>
 #include <fstream>
 #include <functional>
 #include <sstream>
@@ -168,7 +169,6 @@ inline std::string check_layered(const LayeredSpec& s) {
         if (l.kind == MixerKind::kMamba2) {
             if (l.heads % l.groups != 0) return at + "heads is not a multiple of groups";
             if (l.inner() % l.norm_groups != 0) return at + "norm_groups does not divide heads * vdim";
-            if (l.conv > 16) return at + "more than 16 convolution taps";
         }
         if (l.kind != MixerKind::kAttention && l.key_dim() > 256) return at + "more than 256 state rows per head";
         if (l.kind == MixerKind::kAttention) {
@@ -202,6 +202,39 @@ inline int read_model_folder(const std::string& dir, LayeredSpec* spec, Safetens
     if (rc == 1) return fail(QUINTRIT_ERR_IO, "%s", why.c_str());
     if (rc != 0) return fail(QUINTRIT_ERR_FORMAT, "%s", why.c_str());
     return QUINTRIT_OK;
+}
+
+struct LayeredFolder {
+    LayeredSpec spec;
+    SafetensorsFile file;
+};
+
+// The folder's directory as text: hyperparameters one per line, layers, tensors by name.
+inline std::string describe_layered(const LayeredSpec& s, const SafetensorsFile& f) {
+    char num[96];
+    std::string t = "architecture " + s.design + "\nvocab_size " + std::to_string(s.vocab) + "\nhidden_size " + std::to_string(s.width) + "\nnum_layers " + std::to_string(s.layers.size()) +
+                    "\ncontext_length " + std::to_string(s.max_positions) + "\ntied " + (s.head == s.embed ? "1" : "0") + "\n";
+    std::snprintf(num, sizeof num, "rms_norm_eps %.9g\nembed_scale %.9g\n", static_cast<double>(s.eps), static_cast<double>(s.embed_scale));
+    t += num;
+    for (size_t i = 0; i < s.layers.size(); ++i) {
+        const LayerSpec& l = s.layers[i];
+        t += "layer_" + std::to_string(i) + " " + mixer_name(l.kind) + " heads=" + std::to_string(l.heads) + " vdim=" + std::to_string(l.vdim);
+        if (l.kind == MixerKind::kMamba2)
+            t += " state=" + std::to_string(l.state) + " groups=" + std::to_string(l.groups) + " conv=" + std::to_string(l.conv) + " norm_groups=" + std::to_string(l.norm_groups);
+        else
+            t += " dim=" + std::to_string(l.dim);
+        if (l.kind == MixerKind::kAttention) {
+            std::snprintf(num, sizeof num, " kv_heads=%d window=%d pool=%d scale=%.9g", l.kv_heads, l.window, l.pool, static_cast<double>(l.scale));
+            t += num;
+        }
+        t += " ff=" + std::to_string(l.ff) + "\n";
+    }
+    for (const auto& e : f.tensors) {
+        t += "tensor " + e.first + " type=" + e.second.dtype + " shape=";
+        for (size_t i = 0; i < e.second.shape.size(); ++i) t += (i ? "x" : "") + std::to_string(e.second.shape[i]);
+        t += " bytes=" + std::to_string(e.second.bytes) + "\n";
+    }
+    return t;
 }
 
 }  // namespace qtb

@@ -1007,7 +1007,7 @@ int rt_begin_sampling(quintrit_session* s, const quintrit_generate_params_t& prm
     if (!*on_device) return QUINTRIT_OK;
     DeviceGuard dg(s->dec->device);
     if (s->dec->d_rng == nullptr) {
-        int rc = dev_alloc(s->dec, &s->dec->d_rng, 1);
+        int rc = dev_alloc(s->dec, &s->dec->d_rng, 1, false);  // (clearing it would run beside the copy below, which is in the decoder's own stream)
         if (rc != QUINTRIT_OK) return rc;
     }
     QTB_CUDA(cudaMemcpyAsync(s->dec->d_rng, &sampler.state, sizeof sampler.state, cudaMemcpyHostToDevice, s->dec->stream));

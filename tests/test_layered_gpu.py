@@ -276,12 +276,12 @@ def test_greedy_and_sampled_generation_through_sessions(tmp_path):
     # the sampling loop: top-k 1 and temperature 0 are greedy; equal seeds give equal tokens; the draw follows the device sampler's
     assert s.sample_tokens(prompt, 30, temperature=0.0).tolist() == want
     assert s.sample_tokens(prompt, 30, temperature=1.0, top_k=1).tolist() == want
-    one, two = s.sample_tokens(prompt, 20, temperature=1.5, top_k=20, top_p=0.95, seed=7), s.sample_tokens(prompt, 20, temperature=1.5, top_k=20, top_p=0.95, seed=7)
-    assert one.tolist() == two.tolist() and one.tolist() != s.sample_tokens(prompt, 20, temperature=1.5, top_k=20, top_p=0.95, seed=0x9E3779B97F4A7C15).tolist()
+    one, two = s.sample_tokens(prompt, 20, temperature=20.0, top_k=20, top_p=0.95, seed=7), s.sample_tokens(prompt, 20, temperature=20.0, top_k=20, top_p=0.95, seed=7)
+    assert one.tolist() == two.tolist() and one.tolist() != s.sample_tokens(prompt, 20, temperature=20.0, top_k=20, top_p=0.95, seed=0x9E3779B97F4A7C15).tolist()
     fresh = model.new_session()
     row, state = fresh.feed(prompt, [len(prompt) - 1])[0], 7
     for t in one:
-        tok, state = q.sample_logits(row, 1.5, 20, 0.95, state)
+        tok, state = q.sample_logits(row, 20.0, 20, 0.95, state)
         assert tok == t
         row = fresh.feed([tok], [0])[0]
     with pytest.raises(q.QuintritError) as e:
