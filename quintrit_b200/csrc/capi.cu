@@ -1578,7 +1578,8 @@ int decoder_from_model(const GgufModel& md, uint32_t ctx, quintrit_b200_decoder*
     if (md.layered) {
         DeviceGuard g(static_cast<int>(md.device));
         quintrit_b200_decoder* d = nullptr;
-        const int rc = layered_decoder_create(md.layered, ctx, &d);
+        int rc = upload_exp2_table();  // the sampler's exponential
+        if (rc == QUINTRIT_OK) rc = layered_decoder_create(md.layered, ctx, &d);
         if (rc != QUINTRIT_OK) {
             destroy_decoder(d);
             return rc;

@@ -15,6 +15,7 @@
 namespace qtb {
 
 constexpr int kChunkT = 16, kChunkV = 64;  // tokens of a chunk; state columns of a block (16 per warp)
+constexpr int kChunkStages = 4;             // chunks whose inputs are in shared memory or on the way
 
 // Row count of the state the scan is compiled for, 0 if it is too large for it.
 inline int chunk_scan_rows(int n) { return n <= 32 ? 32 : n <= 64 ? 64 : n <= 128 ? 128 : 0; }
@@ -132,10 +133,12 @@ __global__ void __launch_bounds__(256) ssd_gram_kernel(const __grid_constant__ S
     w.gram[(size_t(chunk) * a.groups + g) * 256 + tid] = s;
 }
 
-// hgrn2: gates, A, scaled operands. grid: (heads, chunks), 128 threads; n <= 128
+// hgrn2: gates, A, scaled operands. grid: (heads, chunks), 128 threads; n <= ROWS
+template <int ROWS>
 __global__ void __launch_bounds__(128) hgrn_prep_kernel(const __grid_constant__ ScanArgs a, const __grid_constant__ ChunkWork w) {
     extern __shared__ float prep_sm[];
-    const int head = blockIdx.x, chunk = blockIdx.y, chunks = gridDim.y, tid = threadIdx.x, n = a.n, rows = w.rows;
+    const int head = blockIdx.x, chunk = blockIdx.y, chunks = gridDim.y, tid = threadIdx.x, n = a.n;
+    constexpr int rows = ROWS;
     float *q = prep_sm, *k = q + kChunkT * rows, *f = k + kChunkT * rows;
     for (int i0 = tid; i0 < kChunkT * rows; i0 += 128 * 4) {  // four elements' loads in flight (kChunkT * rows is a multiple of 512)
         float qr[4], fr[4], low[4];
@@ -150,21 +153,22 @@ __global__ void __launch_bounds__(128) hgrn_prep_kernel(const __grid_constant__ 
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int i = i0 + 128 * j;
+            const float e = expf(-fabsf(fr[j])), r = 1.0f / (1.0f + e), up = fr[j] >= 0.0f ? r : e * r, down = fr[j] >= 0.0f ? e * r : r;  // sigmoids of z and -z
             q[i] = there[j] ? silu_f(qr[j]) : 0.0f;
-            f[i] = there[j] ? low[j] + (1.0f - low[j]) * sigmoid_f(fr[j]) : 1.0f;
-            k[i] = there[j] ? (1.0f - low[j]) * sigmoid_f(-fr[j]) : 0.0f;
+            f[i] = there[j] ? low[j] + (1.0f - low[j]) * up : 1.0f;
+            k[i] = there[j] ? (1.0f - low[j]) * down : 0.0f;
         }
     }
     for (int i0 = tid; i0 < kChunkT * w.v_pad; i0 += 128 * 8) {  // (v_pad is a multiple of 64: whole turns of 1024)
         float v[8];
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
-            const int i = i0 + 128 * j, t = chunk * kChunkT + i / w.v_pad, e = i % w.v_pad;
+            const int i = i0 + 128 * j, t = chunk * kChunkT + i / w.v_pad, e = i - (t - chunk * kChunkT) * w.v_pad;
             v[j] = t < a.tokens && e < a.vdim ? a.p[size_t(t) * a.ld + 2 * a.heads * n + head * a.vdim + e] : 0.0f;
         }
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
-            const int i = i0 + 128 * j, t = chunk * kChunkT + i / w.v_pad, e = i % w.v_pad;
+            const int i = i0 + 128 * j, t = chunk * kChunkT + i / w.v_pad, e = i - (t - chunk * kChunkT) * w.v_pad;
             w.xs[(size_t(t) * a.heads + head) * w.v_pad + e] = __float2bfloat16_rn(v[j]);
         }
     }
@@ -211,7 +215,7 @@ __global__ void __launch_bounds__(128) hgrn_prep_kernel(const __grid_constant__ 
 
 template <int KIND> inline size_t chunk_scan_smem(int rows) {
     const size_t stage = size_t(KIND == kScanMamba2 ? 2 : 4) * kChunkT * (rows + 8) * 2 + size_t(kChunkT) * (kChunkV + 8) * 2 + 256 * 4 + (KIND == kScanMamba2 ? 32 : rows) * 4;
-    return 2 * stage;
+    return kChunkStages * stage;
 }
 
 // grid: (heads, ceil(vdim / 64)); warp w owns the state columns 16 w .. 16 w + 15 of the block's 64. y: without mamba2's silu(z), which the
@@ -234,7 +238,12 @@ __global__ void __launch_bounds__(128) chunk_scan_kernel(const __grid_constant__
             const int v = vw + g + (e >> 1) * 8, d = 8 * j + 2 * c + (e & 1);
             S[j][e] = pos0 > 0 && v < a.vdim && d < a.n ? state[size_t(v) * a.n + d] : 0.0f;
         }
-    auto fetch = [&](int chunk, unsigned char* st) {
+    auto fetch = [&](int chunk) {
+        if (chunk >= chunks) {
+            cp_async_commit_group();  // (an empty group keeps the count of groups in step with the chunks)
+            return;
+        }
+        unsigned char* st = cs_sm + (chunk % kChunkStages) * kStage;
         bf16* ops = reinterpret_cast<bf16*>(st);
         bf16* xs = ops + kOps * kChunkT * kPitch;
         float* mat = reinterpret_cast<float*>(xs + kChunkT * kVPitch);
@@ -254,16 +263,12 @@ __global__ void __launch_bounds__(128) chunk_scan_kernel(const __grid_constant__
         for (int i = tid; i < 64 + kTail / 4; i += 128) cp_async16(mat + i * 4, i < 64 ? m + i * 4 : tail + (i - 64) * 4, true);
         cp_async_commit_group();
     };
-    fetch(0, cs_sm);
+    for (int i = 0; i < kChunkStages - 1; ++i) fetch(i);
     for (int chunk = 0; chunk < chunks; ++chunk) {
-        unsigned char* st = cs_sm + (chunk & 1) * kStage;
-        if (chunk + 1 < chunks) {
-            fetch(chunk + 1, cs_sm + ((chunk + 1) & 1) * kStage);
-            cp_async_wait_group<1>();
-        } else {
-            cp_async_wait_group<0>();
-        }
+        unsigned char* st = cs_sm + (chunk % kChunkStages) * kStage;
+        cp_async_wait_group<kChunkStages - 2>();
         __syncthreads();
+        fetch(chunk + kChunkStages - 1);  // into the stage of the chunk before this one, which every warp has left
         if (vw < a.vdim) {
             const bf16* ops = reinterpret_cast<const bf16*>(st);
             const bf16* xs = ops + kOps * kChunkT * kPitch;
@@ -358,7 +363,6 @@ __global__ void __launch_bounds__(128) chunk_scan_kernel(const __grid_constant__
                 }
             }
         }
-        __syncthreads();
     }
 #pragma unroll
     for (int j = 0; j < ROWS / 8; ++j)

@@ -445,7 +445,8 @@ inline int layered_chunk_scan(quintrit_b200_decoder* d, const LayerSpec& l, cons
         ssd_gram_kernel<<<dim3(l.groups + 1, chunks), 256, size_t(2 * kChunkT) * (rows + 1) * sizeof(float), s>>>(a, w);
         QTB_LAUNCH_CHECK();
     } else {
-        hgrn_prep_kernel<<<dim3(l.heads, chunks), 128, size_t(3 * kChunkT) * rows * sizeof(float), s>>>(a, w);
+        auto prep = [&](auto kernel) { kernel<<<dim3(l.heads, chunks), 128, size_t(3 * kChunkT) * rows * sizeof(float), s>>>(a, w); };
+        rows == 32 ? prep(hgrn_prep_kernel<32>) : rows == 64 ? prep(hgrn_prep_kernel<64>) : prep(hgrn_prep_kernel<128>);
         QTB_LAUNCH_CHECK();
     }
     const dim3 grid(l.heads, w.v_pad / kChunkV);

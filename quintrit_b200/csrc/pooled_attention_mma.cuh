@@ -16,6 +16,12 @@ inline int pooled_mma_dims(int dim, int vdim) {
 }
 inline size_t pooled_mma_smem(int dims) { return size_t(kPmRows + 4 * kPmKeys) * (dims + 8) * 2; }
 
+__device__ __forceinline__ float fast_exp2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+
 // grid: (query tiles, heads). The launch's keys and values are in the cache (pooled_append_kernel).
 template <int D>
 __global__ void __launch_bounds__(kPmThreads) pooled_attention_mma_kernel(const __grid_constant__ PooledAttnArgs a) {
@@ -65,6 +71,7 @@ __global__ void __launch_bounds__(kPmThreads) pooled_attention_mma_kernel(const 
     int row_pos[2], row_nb[2];
 #pragma unroll
     for (int h = 0; h < 2; ++h) row_pos[h] = first + warp * 16 + g + 8 * h, row_nb[h] = pooled_blocks_seen(row_pos[h], a.window, a.pool);
+    const int first_nb = pooled_blocks_seen(first, a.window, a.pool);
     const float to_exp2 = a.scale * 1.4426950408889634f;  // log2(e)
     for (int tile = 0; tile < tiles; ++tile) {
         if (tile + 1 < tiles) {
@@ -92,22 +99,31 @@ __global__ void __launch_bounds__(kPmThreads) pooled_attention_mma_kernel(const 
         const bool pooled = tile < pool_tiles;
         const int k0 = pooled ? tile * kPmKeys : lo + (tile - pool_tiles) * kPmKeys;
         float mx[2] = {m[0], m[1]};
+        const bool open = pooled ? k0 + kPmKeys <= first_nb : k0 + kPmKeys - 1 <= first && k0 > first + kPmRows - 1 - a.window;  // every row sees the whole tile
+        if (open) {
 #pragma unroll
-        for (int j = 0; j < kPmKeys / 8; ++j)
+            for (int j = 0; j < kPmKeys / 8; ++j)
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const int h = e >> 1, key = k0 + j * 8 + 2 * c + (e & 1);
-                const bool seen = pooled ? key < row_nb[h] : key <= row_pos[h] && key > row_pos[h] - a.window;
-                s[j][e] = seen ? s[j][e] * to_exp2 : -INFINITY;
-                mx[h] = fmaxf(mx[h], s[j][e]);
-            }
-        float fac[2];
+                for (int e = 0; e < 4; ++e) s[j][e] *= to_exp2, mx[e >> 1] = fmaxf(mx[e >> 1], s[j][e]);
+        } else {
+#pragma unroll
+            for (int j = 0; j < kPmKeys / 8; ++j)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const int h = e >> 1, key = k0 + j * 8 + 2 * c + (e & 1);
+                    const bool seen = pooled ? key < row_nb[h] : key <= row_pos[h] && key > row_pos[h] - a.window;
+                    s[j][e] = seen ? s[j][e] * to_exp2 : -INFINITY;
+                    mx[h] = fmaxf(mx[h], s[j][e]);
+                }
+        }
+        float fac[2], m_safe[2];
 #pragma unroll
         for (int h = 0; h < 2; ++h) {
             mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 1));
             mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 2));
             fac[h] = mx[h] == -INFINITY ? 1.0f : exp2f(m[h] - mx[h]);  // nothing seen so far: nothing to rescale
             m[h] = mx[h];
+            m_safe[h] = mx[h] == -INFINITY ? 0.0f : mx[h];
             l[h] *= fac[h];
         }
 #pragma unroll
@@ -117,7 +133,7 @@ __global__ void __launch_bounds__(kPmThreads) pooled_attention_mma_kernel(const 
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 const int h = e >> 1;
-                s[j][e] = s[j][e] == -INFINITY ? 0.0f : exp2f(s[j][e] - m[h]);
+                s[j][e] = fast_exp2(s[j][e] - m_safe[h]);  // 0 for a key that is not seen
                 l[h] += s[j][e];
             }
 #pragma unroll

@@ -93,7 +93,7 @@ MIXED = [M(4, 24, 20, groups=2, conv=4, norm_groups=2, ff=88), A(6, 2, 24, 16, 1
 
 
 def mixed(vocab=71, positions=700):
-    return mf.lasosun_config(MIXED, 56, vocab, positions, eps=1e-5, embed_scale=3.0)
+    return mf.lasosun_config(MIXED, 56, vocab, positions, eps=1e-5, embed_scale=0.3)
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
@@ -265,7 +265,7 @@ def greedy(config, w, prompt, n):
 
 def test_greedy_and_sampled_generation_through_sessions(tmp_path):
     config = mixed(positions=120)
-    model, w = build(tmp_path, config, 14, "float32")
+    model, w = build(tmp_path, config, 16, "float32")
     prompt = ids_for(9, 21, 71)
     want, margin = greedy(config, w, prompt, 30)
     assert margin > 1e-3
@@ -276,12 +276,12 @@ def test_greedy_and_sampled_generation_through_sessions(tmp_path):
     # the sampling loop: top-k 1 and temperature 0 are greedy; equal seeds give equal tokens; the draw follows the device sampler's
     assert s.sample_tokens(prompt, 30, temperature=0.0).tolist() == want
     assert s.sample_tokens(prompt, 30, temperature=1.0, top_k=1).tolist() == want
-    one, two = s.sample_tokens(prompt, 20, temperature=20.0, top_k=20, top_p=0.95, seed=7), s.sample_tokens(prompt, 20, temperature=20.0, top_k=20, top_p=0.95, seed=7)
-    assert one.tolist() == two.tolist() and one.tolist() != s.sample_tokens(prompt, 20, temperature=20.0, top_k=20, top_p=0.95, seed=0x9E3779B97F4A7C15).tolist()
+    one, two = s.sample_tokens(prompt, 20, temperature=1.5, top_k=20, top_p=0.95, seed=7), s.sample_tokens(prompt, 20, temperature=1.5, top_k=20, top_p=0.95, seed=7)
+    assert one.tolist() == two.tolist() and one.tolist() != s.sample_tokens(prompt, 20, temperature=1.5, top_k=20, top_p=0.95, seed=0x9E3779B97F4A7C15).tolist()
     fresh = model.new_session()
     row, state = fresh.feed(prompt, [len(prompt) - 1])[0], 7
     for t in one:
-        tok, state = q.sample_logits(row, 20.0, 20, 0.95, state)
+        tok, state = q.sample_logits(row, 1.5, 20, 0.95, state)
         assert tok == t
         row = fresh.feed([tok], [0])[0]
     with pytest.raises(q.QuintritError) as e:
