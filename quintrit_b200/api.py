@@ -673,7 +673,7 @@ def gguf_describe(path: str) -> dict:
             for f in fields:
                 if "=" in f:
                     k, v = f.split("=")
-                    t[k] = tuple(int(x) for x in v.split("x")) if k == "shape" else int(v) if v.isdigit() else v
+                    t[k] = tuple(int(x) for x in v.split("x") if x) if k == "shape" else int(v) if v.isdigit() else v
             tensors.append(t)
         else:
             out[key] = rest

@@ -1453,8 +1453,9 @@ struct GgufModel {
     }
     // Largest context a decoder of this model may have: the model's maximum, at most `limit` (0: 4096) and 7936, rounded down to
     // a multiple of 256 when it reaches 256 (gpu.rs:141-146).
-    // A layered model keeps windows and states instead of a cache of the whole context: any length up to its position table.
+    // A layered model takes any length up to its position table, if it has one; without one the caller says how much (0: kLayeredContext).
     uint32_t context_for(uint32_t limit) const {
+        if (layered && shape.ctx_train == 0) return limit != 0 ? limit : kLayeredContext;
         if (layered) return static_cast<uint32_t>(std::min<uint64_t>(shape.ctx_train, limit != 0 ? limit : shape.ctx_train));
         uint64_t want = std::min<uint64_t>(shape.ctx_train, limit != 0 ? limit : 4096);
         want = std::min<uint64_t>(want, 7936);
@@ -1479,7 +1480,8 @@ int load_model_folder(const char* path, uint32_t device, bool f32, GgufModel* ou
     m.vocab = s.vocab, m.hidden = s.width, m.layers = s.layers.size(), m.ctx_train = s.max_positions, m.eps = s.eps, m.tied = s.head == s.embed;
     for (const LayerSpec& l : s.layers) {
         m.inter = std::max<uint64_t>(m.inter, l.ff);
-        if (l.kind == MixerKind::kAttention && m.heads == 0) m.heads = l.heads, m.kv_heads = l.kv_heads, m.head_dim = l.dim;
+        for (const MixerSpec& x : l.mixers)
+            if (x.cached() && m.heads == 0) m.heads = x.heads, m.kv_heads = x.kv_heads, m.head_dim = x.dim;
     }
     return QUINTRIT_OK;
 }

@@ -8,6 +8,8 @@
 // that are at work together share weight rows.
 //
 // The dual form makes two products of one tile, W_o y and W_down m, in two accumulators and ends with both gates and the residual sum.
+// The grouped form multiplies runs of consecutive activation rows, each with its own range of weight rows (the experts of a mixture); which
+// runs there are is read from device memory.
 // Every wait is bounded, as in gemm_tc.cuh, whose mbarrier, descriptor and status conventions are used here.
 //
 // 32-bit weights: a plain tiled kernel in 32-bit arithmetic with the same endings.
@@ -26,16 +28,24 @@ __host__ __device__ constexpr int dense_stages(int n) { return n > 128 ? 4 : 6; 
 __host__ __device__ constexpr int dense_stage_bytes(int n) { return (kDenseM + n) * kDenseK * 2; }
 __host__ __device__ constexpr int dense_smem(int n) { return dense_stages(n) * dense_stage_bytes(n) + 1024 + 256; }
 
+enum DenseForm : int { kDensePlain = 0, kDenseDual = 1, kDenseGrouped = 2 };
+// Grouped form: activation rows token0 .. token0 + tokens - 1 (at most a tile's N) times the weight rows from row0 on.
+struct DenseRun { int row0, token0, tokens, pad; };
+
 struct DenseGemmArgs {
     int tokens;
     int n_prob;              // plain form: 1 or 2 stacks, each over its own activations
     int k_steps[2];          // 64-column slices
-    int row_tiles[2];
-    DenseStack stack[2];     // plain form: the endings
+    int row_tiles[2];        // grouped form: of one range of weight rows
+    DenseStack stack[2];     // plain and grouped form: the endings
     // dual form
     float* x;
     int width;
     const float *gate1, *gate2;
+    const float* token_gate;      // factor of the first product, one per token; nullptr: 1
+    // grouped form
+    const DenseRun* runs;
+    const int* n_runs;
     unsigned int* status;
     unsigned int spin_limit;
 };
@@ -46,8 +56,10 @@ __device__ __forceinline__ void dense_end(const DenseSeg& g, int row, int token,
     if (row >= g.rows) return;
     if (g.kind == kSegSwiGlu) {
         if ((row & 1) == 0) static_cast<T*>(g.t)[size_t(token) * g.ld + (row >> 1)] = to_storage<T>(silu_f(v) * pair);
+    } else if (g.kind == kSegStore) {
+        static_cast<T*>(g.t)[size_t(token) * g.ld + row] = to_storage<T>(v);
     } else {
-        g.f[size_t(token) * g.ld + row] = g.kind == kSegSigmoid ? sigmoid_f(v + g.bias[row]) : v;
+        g.f[size_t(token) * g.ld + row] = g.kind == kSegSigmoid ? sigmoid_f(v + (g.bias != nullptr ? g.bias[row] : 0.0f)) : v;
     }
 }
 
@@ -75,11 +87,12 @@ __device__ __forceinline__ void tmem_load16(uint32_t taddr, uint32_t (&v)[16]) {
 }
 }  // namespace dense_detail
 
-template <int N, bool DUAL>
+template <int N, int FORM>
 __global__ void __launch_bounds__(kDenseThreads, 1) dense_gemm_tc_kernel(const __grid_constant__ CUtensorMap w0, const __grid_constant__ CUtensorMap h0, const __grid_constant__ CUtensorMap w1,
                                                                          const __grid_constant__ CUtensorMap h1, const __grid_constant__ DenseGemmArgs a) {
     using namespace gemm_detail;
     using namespace dense_detail;
+    constexpr bool DUAL = FORM == kDenseDual, GROUPED = FORM == kDenseGrouped;
     extern __shared__ unsigned char dense_smem_raw[];
     unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(dense_smem_raw) + 1023) & ~uintptr_t(1023));
     constexpr int S = dense_stages(N), kStage = dense_stage_bytes(N), kAcc = DUAL ? 2 * N : N;  // kAcc: tensor-memory columns of a tile
@@ -95,9 +108,14 @@ __global__ void __launch_bounds__(kDenseThreads, 1) dense_gemm_tc_kernel(const _
 
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int token_tiles = (a.tokens + N - 1) / N;
-    const int items = token_tiles * (a.row_tiles[0] + (!DUAL && a.n_prob > 1 ? a.row_tiles[1] : 0));
+    const int items = GROUPED ? *a.n_runs * a.row_tiles[0] : token_tiles * (a.row_tiles[0] + (!DUAL && a.n_prob > 1 ? a.row_tiles[1] : 0));
     // tile `item`: its problem, first row and first token
     auto locate = [&](int item, int* prob, int* row0, int* token0) {
+        if constexpr (GROUPED) {
+            const DenseRun run = a.runs[item / a.row_tiles[0]];
+            *prob = 0, *row0 = run.row0 + item % a.row_tiles[0] * kDenseM, *token0 = run.token0;
+            return;
+        }
         const int tile = item / token_tiles;
         *prob = !DUAL && tile >= a.row_tiles[0] ? 1 : 0;
         *row0 = (tile - (*prob ? a.row_tiles[0] : 0)) * kDenseM;
@@ -194,7 +212,7 @@ __global__ void __launch_bounds__(kDenseThreads, 1) dense_gemm_tc_kernel(const _
             if (!okay) break;
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
             const uint32_t acc = tmem_base + (uint32_t((warp & 3) * 32) << 16) + set * kAcc;
-            const int n_here = min(N, a.tokens - token0);
+            const int n_here = GROUPED ? a.runs[item / a.row_tiles[0]].tokens : min(N, a.tokens - token0);
             if constexpr (DUAL) {
                 const int row = row0 + r;
                 const bool has2 = a.k_steps[1] > 0;
@@ -208,7 +226,7 @@ __global__ void __launch_bounds__(kDenseThreads, 1) dense_gemm_tc_kernel(const _
 #pragma unroll
                         for (int i = 0; i < 16; ++i) {
                             const size_t at = size_t(token0 + min(c0 + i, n_here - 1)) * a.width + row;
-                            add[i] = __uint_as_float(v1[i]) * (a.gate1 != nullptr ? a.gate1[at] : 1.0f);
+                            add[i] = __uint_as_float(v1[i]) * (a.gate1 != nullptr ? a.gate1[at] : a.token_gate != nullptr ? a.token_gate[token0 + min(c0 + i, n_here - 1)] : 1.0f);
                             if (has2) add[i] += __uint_as_float(v2[i]) * (a.gate2 != nullptr ? a.gate2[at] : 1.0f);
                             x[i] = a.x[at];
                         }
@@ -219,7 +237,8 @@ __global__ void __launch_bounds__(kDenseThreads, 1) dense_gemm_tc_kernel(const _
                 }
             } else {
                 const DenseStack& st = a.stack[prob];
-                const DenseSeg& g = st.seg[st.n_seg > 1 && row0 >= st.seg[1].row0 ? 1 : 0];
+                const int stack_row0 = GROUPED ? row0 - a.runs[item / a.row_tiles[0]].row0 : row0;
+                const DenseSeg& g = dense_seg_of(st, stack_row0);
                 for (int c0 = turn * 16; c0 < n_here; c0 += 32) {
                     uint32_t v[16];
                     tmem_load16(acc + c0, v);
@@ -227,7 +246,7 @@ __global__ void __launch_bounds__(kDenseThreads, 1) dense_gemm_tc_kernel(const _
 #pragma unroll
                     for (int i = 0; i < 16; ++i) {
                         const float val = __uint_as_float(v[i]), pair = __shfl_xor_sync(0xffffffffu, val, 1);
-                        if (c0 + i < n_here) dense_end<bf16>(g, row0 + r - g.row0, token0 + c0 + i, val, pair);
+                        if (c0 + i < n_here) dense_end<bf16>(g, stack_row0 + r - g.row0, token0 + c0 + i, val, pair);
                     }
                 }
             }
@@ -248,13 +267,16 @@ __global__ void __launch_bounds__(kDenseThreads, 1) dense_gemm_tc_kernel(const _
 // ---- 32-bit products ------------------------------------------------------------------------------------------------------------------
 constexpr int kF32Tile = 64, kF32K = 16;
 
-template <bool DUAL>
+template <int FORM>
 __global__ void __launch_bounds__(256) dense_gemm_f32_kernel(const float* w0, const float* h0, int pitch0, const float* w1, const float* h1, int pitch1, const __grid_constant__ DenseGemmArgs a) {
+    constexpr bool DUAL = FORM == kDenseDual, GROUPED = FORM == kDenseGrouped;
     __shared__ float ws[kF32K][kF32Tile + 4], hs[kF32K][kF32Tile + 4];
     const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
     const int per = kDenseM / kF32Tile;  // row tiles are counted in units of kDenseM
-    const int token0 = blockIdx.x * kF32Tile;
-    const int prob = !DUAL && static_cast<int>(blockIdx.y) >= a.row_tiles[0] * per ? 1 : 0;
+    if (GROUPED && static_cast<int>(blockIdx.x) >= *a.n_runs) return;
+    const DenseRun run = GROUPED ? a.runs[blockIdx.x] : DenseRun{0, static_cast<int>(blockIdx.x) * kF32Tile, 0, 0};
+    const int token0 = run.token0, end = GROUPED ? token0 + run.tokens : a.tokens;
+    const int prob = !DUAL && !GROUPED && static_cast<int>(blockIdx.y) >= a.row_tiles[0] * per ? 1 : 0;
     const int row0 = (static_cast<int>(blockIdx.y) - (prob ? a.row_tiles[0] * per : 0)) * kF32Tile;
     float acc[2][4][4] = {};
     for (int half = 0; half < (DUAL ? 2 : 1); ++half) {
@@ -265,8 +287,8 @@ __global__ void __launch_bounds__(256) dense_gemm_f32_kernel(const float* w0, co
             __syncthreads();
             for (int i = tid; i < kF32Tile * kF32K; i += 256) {
                 const int r = i / kF32K, k = i % kF32K;
-                ws[k][r] = w[size_t(row0 + r) * pitch + k0 + k];
-                hs[k][r] = token0 + r < a.tokens ? h[size_t(token0 + r) * pitch + k0 + k] : 0.0f;
+                ws[k][r] = w[size_t(run.row0 + row0 + r) * pitch + k0 + k];
+                hs[k][r] = token0 + r < end ? h[size_t(token0 + r) * pitch + k0 + k] : 0.0f;
             }
             __syncthreads();
 #pragma unroll
@@ -283,7 +305,7 @@ __global__ void __launch_bounds__(256) dense_gemm_f32_kernel(const float* w0, co
     }
     for (int j = 0; j < 4; ++j) {
         const int token = token0 + ty * 4 + j;
-        if (token >= a.tokens) continue;
+        if (token >= end) continue;
         for (int i = 0; i < 4; ++i) {
             const int row = row0 + tx * 4 + i;
             if constexpr (DUAL) {
@@ -291,11 +313,12 @@ __global__ void __launch_bounds__(256) dense_gemm_f32_kernel(const float* w0, co
                 const size_t at = size_t(token) * a.width + row;
                 float add = acc[0][i][j];
                 if (a.gate1 != nullptr) add *= a.gate1[at];
+                else if (a.token_gate != nullptr) add *= a.token_gate[token];
                 if (a.k_steps[1] > 0) add += acc[1][i][j] * (a.gate2 != nullptr ? a.gate2[at] : 1.0f);
                 a.x[at] += add;
             } else {
                 const DenseStack& st = a.stack[prob];
-                const DenseSeg& g = st.seg[st.n_seg > 1 && row0 >= st.seg[1].row0 ? 1 : 0];
+                const DenseSeg& g = dense_seg_of(st, row0);
                 dense_end<float>(g, row - g.row0, token, acc[0][i][j], acc[0][i ^ 1][j]);
             }
         }

@@ -2,9 +2,11 @@
 // (layered.cuh) takes a decode step with. Activations and sums are 32-bit; an activation is rounded to the storage type where the
 // batched path (dense_gemm_tc.cuh) stores it, so both paths round in the same places.
 //
-//   norm_project_kernel    RMS norms of the residual stream, then up to two stacked projections of them, each row range with its own
-//                          ending (plain, sigmoid of a gate, SwiGLU of interleaved gate | up rows)
+//   norm_project_kernel    norms of the residual stream (to which the normed results of two mixers may still have to be added), then up to
+//                          two stacked projections of them, each row range with its own ending (plain, sigmoid of a gate, SwiGLU of
+//                          interleaved gate | up rows)
 //   finish_project_kernel  the mixer's output norm, then output and down projection, both gates and the residual sum
+//   out_project_kernel     output norm and gate of one mixer or two side by side, then their output projections
 //
 // The kernels of a decode step follow one another with programmatic dependent launch: a kernel may start while the one before it still runs,
 // brings what does not depend on it (weights, states, cached keys) on the way, and only then waits for its results.
@@ -52,20 +54,40 @@ __device__ __forceinline__ void l2_prefetch(const void* p, size_t bytes) {
 }
 
 // What becomes of the rows of one range of a stacked projection.
-enum SegKind : int { kSegPlain = 0, kSegSigmoid = 1, kSegSwiGlu = 2 };
+enum SegKind : int { kSegPlain = 0, kSegSigmoid = 1, kSegSwiGlu = 2, kSegStore = 3 };
 struct DenseSeg {
     int row0, rows;      // rows of the stack (row0 a multiple of kRowPad)
     int kind;
     int ld;              // elements between the results of consecutive tokens
     float* f;            // kSegPlain, kSegSigmoid: 32-bit results
-    void* t;             // kSegSwiGlu: silu(row 2 i) * row 2 i + 1, in the storage type
-    const float* bias;   // kSegSigmoid: added before the sigmoid
+    void* t;             // kSegSwiGlu: silu(row 2 i) * row 2 i + 1, in the storage type; kSegStore: results in the storage type
+    const float* bias;   // kSegSigmoid: added before the sigmoid, may be nullptr
 };
 struct DenseStack {
     const void* w;       // [rows padded][pitch], storage type
     int pitch, cols;     // pitch: columns padded to kColPad
     int n_seg;
-    DenseSeg seg[2];
+    DenseSeg seg[4];
+};
+// The range that row `row` of a stack belongs to.
+__device__ __forceinline__ const DenseSeg& dense_seg_of(const DenseStack& st, int row) {
+    int k = 0;
+    while (k + 1 < st.n_seg && row >= st.seg[k + 1].row0) ++k;
+    return st.seg[k];
+}
+
+// A norm over the model width: RMS (x / rms(x)) w, or, element by element, tanh(alpha x) w + b.
+struct NormParams {
+    const float* w;
+    const float* b;      // not nullptr: the tanh form
+    float alpha;
+};
+__device__ __forceinline__ float norm_value(const NormParams& n, float x, float inv, int i) { return n.b != nullptr ? tanhf(n.alpha * x) * n.w[i] + n.b[i] : x * inv * n.w[i]; }
+
+// Two vectors whose RMS norms, each with its weight, are averaged and added to the residual stream.
+struct PairSum {
+    const float* r[2];   // [tokens][width]; nullptr: nothing is added
+    const float* w[2];
 };
 
 // ---- reductions ---------------------------------------------------------------------------------------------------------------------
@@ -162,10 +184,13 @@ __device__ __forceinline__ void dot_rows(const T* w, int pitch, const float* h, 
 // ---- norms and the projections of their results ----------------------------------------------------------------------------------------
 struct NormProjectArgs {
     const float* x;             // residual stream, [tokens][width]
-    const float* norm_w[2];     // weights of the two norms
+    NormParams norm[2];
     float eps;
     int width, n_stack;         // projections: 1 or 2, each over its own norm of x
     DenseStack stack[2];
+    PairSum pair;               // added to x first; the first block writes the sum to x_out (not x itself)
+    float* x_out;
+    void* h_out;                // the first norm's result in the storage type, [tokens][pitch]; may be nullptr
 };
 
 constexpr int kProjectThreads = 256;
@@ -191,15 +216,36 @@ __global__ void __launch_bounds__(kProjectThreads, 4) norm_project_kernel(NormPr
     }
     bool first = true;
     pdl_wait();
-    float ss = 0.0f;
+    if (a.pair.r[0] != nullptr) {
+        float* sum = act_smem + a.n_stack * pitch;
+        const float *l = a.pair.r[0] + size_t(token) * a.width, *r = a.pair.r[1] + size_t(token) * a.width;
+        float sl = 0.0f, sr = 0.0f;
 #pragma unroll 4
-    for (int i = tid; i < a.width; i += kProjectThreads) ss += x[i] * x[i];
-    ss = block_sum(ss, red);
-    const float inv = 1.0f / sqrtf(ss / static_cast<float>(a.width) + a.eps);
+        for (int i = tid; i < a.width; i += kProjectThreads) sl += l[i] * l[i], sr += r[i] * r[i];
+        sl = block_sum(sl, red), sr = block_sum(sr, red);
+        const float il = 0.5f / sqrtf(sl / static_cast<float>(a.width) + a.eps), ir = 0.5f / sqrtf(sr / static_cast<float>(a.width) + a.eps);
+#pragma unroll 4
+        for (int i = tid; i < a.width; i += kProjectThreads) {
+            const float v = x[i] + (l[i] * il * a.pair.w[0][i] + r[i] * ir * a.pair.w[1][i]);
+            sum[i] = v;
+            if (blockIdx.x == 0) a.x_out[size_t(token) * a.width + i] = v;
+        }
+        x = sum;  // (each thread reads back what it wrote)
+    }
+    float inv = 1.0f;
+    if (a.norm[0].b == nullptr) {
+        float ss = 0.0f;
+#pragma unroll 4
+        for (int i = tid; i < a.width; i += kProjectThreads) ss += x[i] * x[i];
+        inv = 1.0f / sqrtf(block_sum(ss, red) / static_cast<float>(a.width) + a.eps);
+    }
     for (int s = 0; s < a.n_stack; ++s)
 #pragma unroll 4
-        for (int i = tid; i < pitch; i += kProjectThreads)
-            act_smem[s * pitch + act_index<T>(i, pitch)] = i < a.width ? round_to<T>(x[i] * inv * a.norm_w[s][i]) : 0.0f;
+        for (int i = tid; i < pitch; i += kProjectThreads) {
+            const float v = i < a.width ? round_to<T>(norm_value(a.norm[s], x[i], inv, i)) : 0.0f;
+            act_smem[s * pitch + act_index<T>(i, pitch)] = v;
+            if (a.h_out != nullptr && s == 0 && blockIdx.x == 0) static_cast<T*>(a.h_out)[size_t(token) * pitch + i] = to_storage<T>(v);
+        }
     __syncthreads();
     for (int s = 0; s < a.n_stack; ++s)
         for (int k = 0; k < a.stack[s].n_seg; ++k) {
@@ -217,7 +263,7 @@ __global__ void __launch_bounds__(kProjectThreads, 4) norm_project_kernel(NormPr
                     static_cast<T*>(g.t)[size_t(token) * g.ld + unit] = to_storage<T>(silu_f(v[0]) * v[1]);
                 } else {
                     float* f = g.f + size_t(token) * g.ld + r;
-                    for (int j = 0; j < 2 && r + j < g.rows; ++j) f[j] = g.kind == kSegSigmoid ? sigmoid_f(v[j] + g.bias[r + j]) : v[j];
+                    for (int j = 0; j < 2 && r + j < g.rows; ++j) f[j] = g.kind == kSegSigmoid ? sigmoid_f(v[j] + (g.bias != nullptr ? g.bias[r + j] : 0.0f)) : v[j];
                 }
             }
             unit -= units;
@@ -225,10 +271,14 @@ __global__ void __launch_bounds__(kProjectThreads, 4) norm_project_kernel(NormPr
 }
 
 // ---- output norm of a mixer -----------------------------------------------------------------------------------------------------------
-// y of one token in `parts` equal parts, each divided by its own root mean square, times w[i % w_len]; in place in shared memory, in the
-// order act_index<T>. red: one float per warp.
+// y of one token in `parts` equal parts, each divided by its own root mean square, times w[i % w_len] (w may be nullptr) and times
+// silu(gate[i]) (gate may be nullptr); in place in shared memory, in the order act_index<T>. red: one float per warp.
 template <typename T>
-__device__ __forceinline__ void parts_norm(float* y, int n, int pitch, int parts, float eps, const float* w, int w_len, float* red) {
+__device__ __forceinline__ void parts_norm(float* y, int n, int pitch, int parts, float eps, const float* w, int w_len, const float* gate, float* red) {
+    const auto ending = [&](float v, int e) {
+        if (w != nullptr) v *= w[e % w_len];
+        return round_to<T>(gate != nullptr ? v * silu_f(gate[e]) : v);
+    };
     const int len = n / parts, warps = blockDim.x >> 5, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     if (parts >= warps) {  // a warp per part
         for (int p = warp; p < parts; p += warps) {
@@ -240,7 +290,7 @@ __device__ __forceinline__ void parts_norm(float* y, int n, int pitch, int parts
             const float inv = 1.0f / sqrtf(warp_sum(ss) / static_cast<float>(len) + eps);
             for (int i = lane; i < len; i += 32) {
                 const int e = p * len + i, at = act_index<T>(e, pitch);
-                y[at] = round_to<T>(y[at] * inv * w[e % w_len]);
+                y[at] = ending(y[at] * inv, e);
             }
         }
         __syncthreads();
@@ -255,7 +305,7 @@ __device__ __forceinline__ void parts_norm(float* y, int n, int pitch, int parts
         const float inv = 1.0f / sqrtf(block_sum(ss, red) / static_cast<float>(len) + eps);
         for (int i = threadIdx.x; i < len; i += blockDim.x) {
             const int e = p * len + i, at = act_index<T>(e, pitch);
-            y[at] = round_to<T>(y[at] * inv * w[e % w_len]);
+            y[at] = ending(y[at] * inv, e);
         }
     }
     __syncthreads();
@@ -317,7 +367,7 @@ __global__ void __launch_bounds__(kProjectThreads, 4) finish_project_kernel(Fini
         for (int i = tid; i < a.down_pitch / kPer; i += kProjectThreads) act_put_storage(m, i, a.down_pitch, static_cast<const T*>(a.m) + size_t(token) * a.down_pitch);
     }
     __syncthreads();
-    if (norm) parts_norm<T>(y, a.inner, a.o_pitch, a.norm_parts, a.eps, a.norm_w, a.norm_len, red);
+    if (norm) parts_norm<T>(y, a.inner, a.o_pitch, a.norm_parts, a.eps, a.norm_w, a.norm_len, nullptr, red);
     for (int row = blockIdx.x * (kProjectThreads / 32) + (tid >> 5); row < a.width; row += warps) {
         float so[1], sd[1] = {0.0f};
         const T *o_row = static_cast<const T*>(a.o) + size_t(row) * a.o_pitch, *d_row = static_cast<const T*>(a.down) + size_t(row) * a.down_pitch;
@@ -336,6 +386,66 @@ __global__ void __launch_bounds__(kProjectThreads, 4) finish_project_kernel(Fini
     }
 }
 
+// ---- output projections of one mixer, or of two side by side ------------------------------------------------------------------------------
+struct OutProjectArgs {
+    int width, n;               // n: mixers
+    float eps;
+    struct Mixer {
+        const float* y;         // 32-bit output of the mixer, [tokens][inner]
+        int inner, parts;       // parts > 0: each divided by its root mean square
+        const float* gate;      // times silu(gate[token * gate_ld + i]); may be nullptr
+        int gate_ld;
+        const void* w;          // [width][pitch]
+        int pitch;
+        float* out;             // [tokens][width]
+        bool add;               // out += W y instead of out = W y
+    } mix[2];
+};
+
+template <typename T>
+__global__ void __launch_bounds__(kProjectThreads, 4) out_project_kernel(const __grid_constant__ OutProjectArgs a) {
+    extern __shared__ float act_smem[];
+    __shared__ float red[kProjectThreads / 32];
+    const int tid = threadIdx.x, lane = tid & 31, token = blockIdx.y, warps = gridDim.x * (kProjectThreads / 32), units = a.n * a.width;
+    const int unit0 = blockIdx.x * (kProjectThreads / 32) + (tid >> 5);
+    pdl_trigger();
+    RowHead<1> head;
+    bool first = true;
+    if (unit0 < units) {
+        const OutProjectArgs::Mixer& m = a.mix[unit0 >= a.width ? 1 : 0];
+        load_pieces<T, 1>(head, static_cast<const T*>(m.w) + size_t(unit0 % a.width) * m.pitch, m.pitch, lane);
+    }
+    pdl_wait();
+    for (int k = 0; k < a.n; ++k) {
+        const OutProjectArgs::Mixer& m = a.mix[k];
+        // a block all of whose rows belong to the other mixer leaves this one's vector out
+        const int lo = blockIdx.x * (kProjectThreads / 32), hi = lo + kProjectThreads / 32 - 1;
+        if (warps >= units && (k == 0 ? lo >= a.width : hi < a.width)) continue;
+        float* y = act_smem + (k > 0 ? a.mix[0].pitch : 0);
+        const float* src = m.y + size_t(token) * m.inner;
+#pragma unroll 4
+        for (int i = tid; i < m.pitch; i += kProjectThreads) {
+            const float v = i < m.inner ? src[i] : 0.0f;
+            y[act_index<T>(i, m.pitch)] = m.parts > 0 ? v : round_to<T>(v);
+        }
+        __syncthreads();
+        if (m.parts > 0) parts_norm<T>(y, m.inner, m.pitch, m.parts, a.eps, nullptr, 1, m.gate != nullptr ? m.gate + size_t(token) * m.gate_ld : nullptr, red);
+    }
+    for (int unit = unit0; unit < units; unit += warps) {
+        const int k = unit >= a.width ? 1 : 0, row = unit - k * a.width;
+        const OutProjectArgs::Mixer& m = a.mix[k];
+        const T* w = static_cast<const T*>(m.w) + size_t(row) * m.pitch;
+        float v[1];
+        if (!first) load_pieces<T, 1>(head, w, m.pitch, lane);
+        first = false;
+        dot_rows<T, 1>(w, m.pitch, act_smem + (k > 0 ? a.mix[0].pitch : 0), head, v);
+        if (lane == 0) {
+            float* out = m.out + size_t(token) * a.width + row;
+            *out = m.add ? *out + v[0] : v[0];
+        }
+    }
+}
+
 // ---- batched counterparts of the steps around the projections ------------------------------------------------------------------------------
 // x = embed[token] * scale + pos[position] (pos may be nullptr)
 template <typename T>
@@ -347,26 +457,122 @@ __global__ void embed_scaled_kernel(const T* embed, int pitch, const T* pos_tabl
     x[size_t(t) * width + i] = v;
 }
 
-// h_s = RMS norm of x with the weights w_s, in the storage type; rows (optional) picks tokens
+// h_s = norm s of x, in the storage type; rows (optional) picks tokens
 template <typename T>
-__global__ void __launch_bounds__(256) norm_rows_kernel(const float* x, int width, float eps, const float* w0, T* h0, const float* w1, T* h1, int pitch, const uint32_t* rows) {
+__global__ void __launch_bounds__(256) norm_rows_kernel(const float* x, int width, float eps, NormParams n0, T* h0, NormParams n1, T* h1, int pitch, const uint32_t* rows) {
     __shared__ float red[8];
     const int t = blockIdx.x;
     const float* xr = x + size_t(rows != nullptr ? rows[t] : t) * width;
-    float ss = 0.0f;
-    for (int i = threadIdx.x; i < width; i += blockDim.x) ss += xr[i] * xr[i];
-    const float inv = 1.0f / sqrtf(block_sum(ss, red) / static_cast<float>(width) + eps);
+    float inv = 1.0f;
+    if (n0.b == nullptr) {
+        float ss = 0.0f;
+        for (int i = threadIdx.x; i < width; i += blockDim.x) ss += xr[i] * xr[i];
+        inv = 1.0f / sqrtf(block_sum(ss, red) / static_cast<float>(width) + eps);
+    }
     for (int i = threadIdx.x; i < width; i += blockDim.x) {
-        const float v = xr[i] * inv;
-        h0[size_t(t) * pitch + i] = to_storage<T>(v * w0[i]);
-        if (h1 != nullptr) h1[size_t(t) * pitch + i] = to_storage<T>(v * w1[i]);
+        h0[size_t(t) * pitch + i] = to_storage<T>(norm_value(n0, xr[i], inv, i));
+        if (h1 != nullptr) h1[size_t(t) * pitch + i] = to_storage<T>(norm_value(n1, xr[i], inv, i));
     }
 }
 
-// The mixer's output norm of many tokens (parts_norm), into the storage type; without a norm a plain conversion. gate (may be nullptr):
-// y is first multiplied by silu(gate[token * gate_ld + i]).
+// x = norm(embed[token]), also written to `first` (the first of the vectors that depth averages run over; may be nullptr), and h = next(x)
 template <typename T>
-__global__ void __launch_bounds__(256) finish_rows_kernel(const float* y, const float* gate, int gate_ld, int inner, int parts, float eps, const float* w, int w_len, T* out, int pitch) {
+__global__ void __launch_bounds__(256) embed_norm_kernel(const T* embed, int pitch, const uint32_t* tokens, int width, float eps, NormParams norm, float* x, float* first, NormParams next, T* h) {
+    extern __shared__ float act_smem[];
+    __shared__ float red[8];
+    const int t = blockIdx.x;
+    const T* row = embed + size_t(tokens[t]) * pitch;
+    float ss = 0.0f;
+    for (int i = threadIdx.x; i < width; i += blockDim.x) {
+        const float v = from_storage(row[i]);
+        act_smem[i] = v, ss += v * v;
+    }
+    float inv = norm.b == nullptr ? 1.0f / sqrtf(block_sum(ss, red) / static_cast<float>(width) + eps) : 1.0f;
+    ss = 0.0f;
+    for (int i = threadIdx.x; i < width; i += blockDim.x) {
+        const float v = norm_value(norm, act_smem[i], inv, i);
+        act_smem[i] = v, ss += v * v;
+        x[size_t(t) * width + i] = v;
+        if (first != nullptr) first[size_t(t) * width + i] = v;
+    }
+    if (h == nullptr) return;
+    inv = next.b == nullptr ? 1.0f / sqrtf(block_sum(ss, red) / static_cast<float>(width) + eps) : 1.0f;
+    for (int i = threadIdx.x; i < width; i += blockDim.x) h[size_t(t) * pitch + i] = to_storage<T>(norm_value(next, act_smem[i], inv, i));
+}
+
+// What a layer passes on: x = sum over j < n - 1 of w[j] X_j + w[n - 1] v, where v is the layer's result, stored as X_(n - 1).
+struct DepthMix {
+    float* x;            // X_j at x + j * stride, each [tokens][width]
+    size_t stride;
+    const float* w;
+    int n;               // 0: the layer's result itself goes on
+};
+
+// Rows of the residual stream between the products: v = x + the averaged norms of a pair (PairSum) + the weighted results of the chosen
+// experts, then the depth average, then a norm for the next product.
+struct RowsArgs {
+    const float* x;
+    float* x_out;               // may be x
+    int width, pitch;
+    float eps;
+    PairSum pair;
+    const void* pick;           // results of the experts [pair rows][width], storage type; nullptr: none
+    const uint32_t* pick_row;   // [tokens][top]: their rows
+    const float* pick_weight;   // [tokens][top]
+    int top;
+    DepthMix depth;
+    NormParams norm;
+    void* h;                    // storage type, [tokens][pitch]; nullptr: no norm
+};
+
+template <typename T>
+__global__ void __launch_bounds__(256) rows_kernel(const __grid_constant__ RowsArgs a) {
+    extern __shared__ float act_smem[];
+    __shared__ float red[8];
+    const size_t t = blockIdx.x, row = t * a.width;
+    const int tid = threadIdx.x;
+    float il = 0.0f, ir = 0.0f;
+    const bool pair = a.pair.r[0] != nullptr;
+    if (pair) {
+        float sl = 0.0f, sr = 0.0f;
+#pragma unroll 4
+        for (int i = tid; i < a.width; i += 256) {
+            const float l = a.pair.r[0][row + i], r = a.pair.r[1][row + i];
+            sl += l * l, sr += r * r;
+        }
+        sl = block_sum(sl, red), sr = block_sum(sr, red);
+        il = 0.5f / sqrtf(sl / static_cast<float>(a.width) + a.eps), ir = 0.5f / sqrtf(sr / static_cast<float>(a.width) + a.eps);
+    }
+    float ss = 0.0f;
+    for (int i = tid; i < a.width; i += 256) {
+        float v = a.x[row + i];
+        if (pair) v += a.pair.r[0][row + i] * il * a.pair.w[0][i] + a.pair.r[1][row + i] * ir * a.pair.w[1][i];
+        if (a.pick != nullptr) {
+            float s = 0.0f;
+#pragma unroll 4
+            for (int k = 0; k < a.top; ++k) s = fmaf(a.pick_weight[t * a.top + k], from_storage(static_cast<const T*>(a.pick)[size_t(a.pick_row[t * a.top + k]) * a.width + i]), s);
+            v += s;
+        }
+        if (a.depth.n > 0) {
+            a.depth.x[(a.depth.n - 1) * a.depth.stride + row + i] = v;
+            float s = 0.0f;
+#pragma unroll 4
+            for (int j = 0; j < a.depth.n - 1; ++j) s = fmaf(a.depth.w[j], a.depth.x[j * a.depth.stride + row + i], s);
+            v = fmaf(a.depth.w[a.depth.n - 1], v, s);
+        }
+        a.x_out[row + i] = v;
+        act_smem[i] = v, ss += v * v;
+    }
+    if (a.h == nullptr) return;
+    const float inv = a.norm.b == nullptr ? 1.0f / sqrtf(block_sum(ss, red) / static_cast<float>(a.width) + a.eps) : 1.0f;
+    for (int i = tid; i < a.width; i += 256) static_cast<T*>(a.h)[t * a.pitch + i] = to_storage<T>(norm_value(a.norm, act_smem[i], inv, i));
+}
+
+// The mixer's output norm of many tokens (parts_norm), into the storage type; without a norm a plain conversion. gate (may be nullptr):
+// y is first multiplied by silu(gate[token * gate_ld + i]); gate_after: the normed y is.
+template <typename T>
+__global__ void __launch_bounds__(256) finish_rows_kernel(const float* y, const float* gate, const float* gate_after, int gate_ld, int inner, int parts, float eps, const float* w, int w_len, T* out,
+                                                          int pitch) {
     extern __shared__ float act_smem[];
     __shared__ float red[8];
     const int t = blockIdx.x;
@@ -375,7 +581,7 @@ __global__ void __launch_bounds__(256) finish_rows_kernel(const float* y, const 
         act_smem[i] = gate != nullptr ? v * silu_f(gate[size_t(t) * gate_ld + i]) : v;
     }
     __syncthreads();
-    if (parts > 0) parts_norm<float>(act_smem, inner, inner, parts, eps, w, w_len, red);
+    if (parts > 0) parts_norm<float>(act_smem, inner, inner, parts, eps, w, w_len, gate_after != nullptr ? gate_after + size_t(t) * gate_ld : nullptr, red);
     for (int i = threadIdx.x; i < inner; i += blockDim.x) out[size_t(t) * pitch + i] = to_storage<T>(act_smem[i]);
 }
 

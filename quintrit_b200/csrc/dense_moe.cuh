@@ -1,0 +1,256 @@
+// Mixture of experts over dense (16- or 32-bit) weights, the feed-forward of a layered model's layer. A token's router logits become softmax scores
+// over all experts; experts form equal groups of neighbours, only those of the groups with the largest scores can be chosen (a group counts by its
+// largest score), and of these the `top` largest are. Their weights are the scores times a factor, not renormalized. A shared expert, which every
+// token uses, is multiplied by a number per token; it is projected together with the router (dense_gemv.cuh, dense_gemm_tc.cuh).
+//
+// One token: moe_up_step_kernel chooses (every block for itself) and makes the chosen experts' activations, moe_down_step_kernel makes their
+// results, the residual sum and what follows it. Many tokens: the chosen (token, expert) pairs are sorted by expert, the activations copied in
+// that order, and two grouped products run over the experts' runs of rows.
+#pragma once
+#include "dense_gemm_tc.cuh"
+
+namespace qtb {
+
+struct RouterArgs {
+    int experts, groups, keep, top;
+    float scale;
+};
+
+// One warp: the chosen experts of a token, best first, and their weights, from its logits. score: `experts` floats of shared memory (this warp's).
+// Equal scores: the lower index first.
+__device__ __forceinline__ void choose_experts(const RouterArgs& r, const float* logits, float* score, int* chosen, float* weight) {
+    const int lane = threadIdx.x & 31;
+    float mx = -INFINITY, sum = 0.0f;
+    for (int i = lane; i < r.experts; i += 32) mx = fmaxf(mx, logits[i]);
+    for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+    for (int i = lane; i < r.experts; i += 32) {
+        const float e = expf(logits[i] - mx);
+        score[i] = e, sum += e;
+    }
+    sum = warp_sum(sum);
+    __syncwarp();
+    const int size = r.experts / r.groups;
+    auto best_of = [&](float v, int i) {  // the warp's largest value, the lower index of equal ones
+        for (int o = 16; o > 0; o >>= 1) {
+            const float v2 = __shfl_xor_sync(0xffffffffu, v, o);
+            const int i2 = __shfl_xor_sync(0xffffffffu, i, o);
+            if (v2 > v || (v2 == v && i2 < i)) v = v2, i = i2;
+        }
+        return make_float2(v, __int_as_float(i));
+    };
+    if (r.keep < r.groups) {
+        // a group is dropped when `keep` others are better; its scores then no longer count (exponentials are not negative)
+        for (int g0 = 0; g0 < r.groups; g0 += 32) {
+            const int g = g0 + lane;
+            float mine = -1.0f;
+            int better = 0;
+            if (g < r.groups)
+                for (int i = 0; i < size; ++i) mine = fmaxf(mine, score[g * size + i]);
+            for (int o = 0; o < r.groups; ++o) {
+                float other = -1.0f;
+                if (r.groups <= 32) {
+                    other = __shfl_sync(0xffffffffu, mine, o);
+                } else {
+                    for (int i = 0; i < size; ++i) other = fmaxf(other, fabsf(score[o * size + i]));
+                }
+                better += (other > mine || (other == mine && o < g)) ? 1 : 0;
+            }
+            __syncwarp();
+            // (a dropped score changes its sign, so that a group looked at later still sees its size; -0.0 stands for a dropped zero)
+            if (g < r.groups && better >= r.keep)
+                for (int i = 0; i < size; ++i) score[g * size + i] = -score[g * size + i] - 1e-30f;
+            __syncwarp();
+        }
+    }
+    for (int k = 0; k < r.top; ++k) {
+        float v = -INFINITY;
+        int at = r.experts;
+        for (int i = lane; i < r.experts; i += 32)
+            if (score[i] > v) v = score[i], at = i;
+        const float2 b = best_of(v, at);
+        at = min(__float_as_int(b.y), r.experts - 1);  // (stays in range whatever the logits are)
+        if (lane == 0) chosen[k] = at, weight[k] = b.x / sum * r.scale;
+        if (lane == (at & 31)) score[at] = -INFINITY;
+        __syncwarp();
+    }
+}
+
+// ---- one token -----------------------------------------------------------------------------------------------------------------------------
+struct MoeUpStepArgs {
+    RouterArgs router;
+    const float* logits;
+    const void* h;          // normed input, storage type, [pitch]
+    const void* w;          // [experts][rows_pad][pitch]: gate and up rows in turn
+    int pitch, rows_pad, ff;
+    void* m;                // [top][m_pitch]: silu(gate) * up, storage type
+    int m_pitch;
+    int* chosen;            // [top]
+    float* weight;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(kProjectThreads, 4) moe_up_step_kernel(const __grid_constant__ MoeUpStepArgs a) {
+    extern __shared__ float act_smem[];  // the input, then the router's scores
+    __shared__ int chosen[32];
+    __shared__ float weight[32];
+    const int tid = threadIdx.x, warps = gridDim.x * (kProjectThreads / 32), units = a.router.top * a.ff;
+    pdl_trigger();
+    pdl_wait();
+    if (tid < 32) {
+        choose_experts(a.router, a.logits, act_smem + a.pitch, chosen, weight);
+        if (blockIdx.x == 0 && tid < a.router.top) a.chosen[tid] = chosen[tid], a.weight[tid] = weight[tid];
+    }
+    constexpr int kPer = 16 / sizeof(T);
+    for (int i = tid; i < a.pitch / kPer; i += kProjectThreads) act_put_storage(act_smem, i, a.pitch, static_cast<const T*>(a.h));
+    __syncthreads();
+    for (int unit = blockIdx.x * (kProjectThreads / 32) + (tid >> 5); unit < units; unit += warps) {
+        const int k = unit / a.ff, i = unit % a.ff;
+        const T* rows = static_cast<const T*>(a.w) + (size_t(chosen[k]) * a.rows_pad + 2 * i) * a.pitch;
+        RowHead<2> head;
+        float v[2];
+        load_pieces<T, 2>(head, rows, a.pitch, tid & 31);
+        dot_rows<T, 2>(rows, a.pitch, act_smem, head, v);
+        if ((tid & 31) == 0) static_cast<T*>(a.m)[size_t(k) * a.m_pitch + i] = to_storage<T>(silu_f(v[0]) * v[1]);
+    }
+}
+
+struct MoeDownStepArgs {
+    const float* x;         // residual stream before the feed-forward
+    float* x_out;
+    int width, top;
+    const void* m;          // [top][pitch]
+    const void* w;          // [experts][rows_pad][pitch]
+    int pitch, rows_pad;
+    const int* chosen;
+    const float* weight;
+    const void* shared_m;   // [shared_pitch]
+    const void* shared_w;   // [width][shared_pitch]
+    int shared_pitch;
+    const float* shared_scale;
+    DepthMix depth;
+    int rows;               // rows of the result per block
+};
+
+constexpr int kMoeDownRows = 16;  // at most
+
+// A block takes a few rows of the result; its warps share the products of these rows with the activations of every chosen expert.
+template <typename T>
+__global__ void __launch_bounds__(kProjectThreads) moe_down_step_kernel(const __grid_constant__ MoeDownStepArgs a) {
+    extern __shared__ float act_smem[];  // activations of the experts, of the shared expert
+    __shared__ float part[kMoeDownRows * 33];
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, row0 = blockIdx.x * a.rows, rows = min(a.rows, a.width - row0), per = a.top + 1, units = rows * per;
+    float* shared_act = act_smem + a.top * a.pitch;
+    pdl_trigger();
+    if (lane == 0 && warp < rows) l2_prefetch(static_cast<const T*>(a.shared_w) + size_t(row0 + warp) * a.shared_pitch, a.shared_pitch * sizeof(T));
+    pdl_wait();
+    auto row_of = [&](int unit) {
+        const int r = row0 + unit / per, k = unit % per;
+        return k < a.top ? static_cast<const T*>(a.w) + (size_t(a.chosen[k]) * a.rows_pad + r) * a.pitch : static_cast<const T*>(a.shared_w) + size_t(r) * a.shared_pitch;
+    };
+    auto pitch_of = [&](int unit) { return unit % per < a.top ? a.pitch : a.shared_pitch; };
+    RowHead<1> head, next;
+    if (warp < units) load_pieces<T, 1>(head, row_of(warp), pitch_of(warp), lane);
+    constexpr int kPer = 16 / sizeof(T);
+    for (int i = tid; i < a.top * (a.pitch / kPer); i += kProjectThreads) {
+        const int k = i / (a.pitch / kPer), p = i % (a.pitch / kPer);
+        act_put_storage(act_smem + k * a.pitch, p, a.pitch, static_cast<const T*>(a.m) + size_t(k) * a.pitch);
+    }
+    for (int i = tid; i < a.shared_pitch / kPer; i += kProjectThreads) act_put_storage(shared_act, i, a.shared_pitch, static_cast<const T*>(a.shared_m));
+    __syncthreads();
+    for (int unit = warp; unit < units; unit += kProjectThreads / 32) {
+        const int after = unit + kProjectThreads / 32, k = unit % per;
+        if (after < units) load_pieces<T, 1>(next, row_of(after), pitch_of(after), lane);
+        float v[1];
+        dot_rows<T, 1>(row_of(unit), pitch_of(unit), k < a.top ? act_smem + k * a.pitch : shared_act, head, v);
+        if (lane == 0) part[unit / per * 33 + k] = v[0];
+        head = next;
+    }
+    __syncthreads();
+    for (int r = warp; r < rows; r += kProjectThreads / 32) {
+        const int row = row0 + r;
+        float s = lane < a.top ? part[r * 33 + lane] * a.weight[lane] : 0.0f;
+        s = warp_sum(s);
+        const float v = a.x[row] + s + part[r * 33 + a.top] * *a.shared_scale;
+        if (a.depth.n == 0) {
+            if (lane == 0) a.x_out[row] = v;
+            continue;
+        }
+        float d = 0.0f;
+        for (int j = lane; j < a.depth.n - 1; j += 32) d = fmaf(a.depth.w[j], a.depth.x[j * a.depth.stride + row], d);
+        d = warp_sum(d);
+        if (lane == 0) {
+            a.depth.x[(a.depth.n - 1) * a.depth.stride + row] = v;
+            a.x_out[row] = fmaf(a.depth.w[a.depth.n - 1], v, d);
+        }
+    }
+}
+
+// ---- many tokens ---------------------------------------------------------------------------------------------------------------------------
+struct MoeRouteArgs {
+    RouterArgs router;
+    int tokens;
+    const float* logits;    // [tokens][experts]
+    int* chosen;            // [tokens][top]
+    float* weight;          // [tokens][top]
+    int* count;             // [experts], zero between launches: tokens of an expert
+    int* rank;              // [tokens][top]: a pair's place among those of its expert
+    int* first;             // [experts]: first pair row of an expert
+    uint32_t* row;          // [tokens][top]: row of a pair
+    DenseRun *up_runs, *down_runs;
+    int *n_runs;
+    int up_rows, down_rows, tile;  // weight rows of an expert in the two stacks; activation rows of a run
+};
+
+// A warp per token. dynamic shared memory: 4 * experts floats
+__global__ void __launch_bounds__(128) moe_route_kernel(const __grid_constant__ MoeRouteArgs a) {
+    extern __shared__ float route_sm[];
+    __shared__ int chosen[4][32];
+    __shared__ float weight[4][32];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, t = blockIdx.x * 4 + warp, top = a.router.top;
+    if (t >= a.tokens) return;
+    choose_experts(a.router, a.logits + size_t(t) * a.router.experts, route_sm + warp * a.router.experts, chosen[warp], weight[warp]);
+    __syncwarp();
+    if (lane < top) {
+        const int e = chosen[warp][lane];
+        a.chosen[t * top + lane] = e, a.weight[t * top + lane] = weight[warp][lane];
+        a.rank[t * top + lane] = atomicAdd(a.count + e, 1);
+    }
+}
+
+// One block of 1024 threads, a thread per expert: where the experts' rows begin, and the runs of both products. Leaves the counts at zero.
+__global__ void __launch_bounds__(1024) moe_plan_kernel(const __grid_constant__ MoeRouteArgs a) {
+    __shared__ int rows_sum[32], runs_sum[32];
+    const int e = threadIdx.x, warp = e >> 5, lane = e & 31;
+    const int n = e < a.router.experts ? a.count[e] : 0, r = (n + a.tile - 1) / a.tile;
+    int rows = n, runs = r;  // running sums
+    for (int o = 1; o < 32; o <<= 1) {
+        const int x = __shfl_up_sync(0xffffffffu, rows, o), y = __shfl_up_sync(0xffffffffu, runs, o);
+        if (lane >= o) rows += x, runs += y;
+    }
+    if (lane == 31) rows_sum[warp] = rows, runs_sum[warp] = runs;
+    __syncthreads();
+    int rows0 = 0, runs0 = 0, all = 0;
+    for (int w = 0; w < 32; ++w) {
+        if (w < warp) rows0 += rows_sum[w], runs0 += runs_sum[w];
+        all += runs_sum[w];
+    }
+    rows0 += rows - n, runs0 += runs - r;
+    if (e == 0) *a.n_runs = all;
+    if (e >= a.router.experts) return;
+    a.first[e] = rows0, a.count[e] = 0;
+    for (int k = 0; k < r; ++k) {
+        const int from = k * a.tile, here = min(a.tile, n - from);
+        a.up_runs[runs0 + k] = DenseRun{e * a.up_rows, rows0 + from, here, 0};
+        a.down_runs[runs0 + k] = DenseRun{e * a.down_rows, rows0 + from, here, 0};
+    }
+}
+
+// Copies each pair's activations to its row. grid: (top, tokens); pitch in 16-byte pieces
+__global__ void __launch_bounds__(128) moe_gather_kernel(const __grid_constant__ MoeRouteArgs a, const uint4* h, uint4* out, int pieces) {
+    const int pair = blockIdx.y * a.router.top + blockIdx.x;
+    const uint32_t row = a.first[a.chosen[pair]] + a.rank[pair];
+    if (threadIdx.x == 0) a.row[pair] = row;
+    for (int i = threadIdx.x; i < pieces; i += 128) out[size_t(row) * pieces + i] = h[size_t(blockIdx.y) * pieces + i];
+}
+
+}  // namespace qtb

@@ -2,9 +2,10 @@
 //
 //   S_t = a_t (.) S_(t-1) + k_t x_t^T      y_t = S_t^T q_t       (S: N rows x vdim columns; a_t: a number or one per row)
 //
-// Two ways to make a, k, q and x from a layer's projections (ScanKind):
+// Three ways to make a, k, q and x from a layer's projections (ScanKind):
 //   mamba2  a = exp(-exp(A_log) dt), k = dt B, q = C, with dt = softplus(dt_raw + dt_bias); x, B and C come out of a causal convolution
 //           per channel and silu; the result is y + D x, times silu(z)
+//   retention  a: a constant per head, q and k rotated by their position, k times N^(-1/2), x = v
 //   hgrn2   a = l + (1 - l) sigmoid(f_raw + f_bias), k = 1 - a, q = silu(q_raw), x = v
 // All of it in 32-bit arithmetic. The output norm follows in the kernel that consumes y (dense_gemv.cuh).
 //
@@ -13,22 +14,26 @@
 // inputs before the start as zero, so a slot needs no clearing when it is used again.
 #pragma once
 #include "dense_gemv.cuh"
+#include "rotation.cuh"
 
 namespace qtb {
 
-enum ScanKind : int { kScanMamba2 = 0, kScanHgrn2 = 1 };
+enum ScanKind : int { kScanMamba2 = 0, kScanHgrn2 = 1, kScanRetention = 2 };
 
 struct ScanArgs {
     int tokens;               // consecutive tokens of a sequence in this launch (1: a decode step, sequences in gridDim.z)
     const uint32_t* pos;      // positions as SeqIndex describes them
     SeqIndex seq;
-    const float* p;           // projections [token][ld]; mamba2: z | x | B | C | dt, hgrn2: q | f | v
+    const float* p;           // projections [token][ld]; mamba2: z | x | B | C | dt, hgrn2: q | f | v, retention: q | k | v | g
     int ld;
     int heads, vdim, n;       // n: rows of the state
     int groups;               // mamba2: B and C are shared by heads / groups heads
     int taps;
     const float *conv_w, *conv_b, *dt_bias, *a_log, *d_skip;  // mamba2
     const float *f_bias, *lower;                              // hgrn2, heads * n each
+    const float* decay;       // retention, one per head
+    const double* turns;      // retention: turns of a rotated pair per position, rot_dims / 2 of them (rotation.cuh)
+    int rot_dims;
     float* state;             // [slot][heads][vdim][n]
     float* conv;              // [slot][taps][conv channels]
     float* y;                 // [token][heads * vdim]
@@ -100,6 +105,26 @@ __global__ void __launch_bounds__(kScanThreads) gated_scan_kernel(const __grid_c
                 const int t = i / kScanRows, v = v0 + i % kScanRows;
                 xs[i] = v < a.vdim ? conv_silu(a, ring, row0 + t0 + t, t0 + t, pos0 + t0 + t, head * a.vdim + v, channels, inner) : 0.0f;
             }
+        } else if (KIND == kScanRetention) {
+            const float scale = 1.0f / sqrtf(static_cast<float>(n));
+            const int half = a.rot_dims / 2, items = n - half;  // an item is a rotated pair, or an element that stays as it is
+            for (int i = tid; i < nt * items; i += kScanThreads) {
+                const int t = i / items, j = i % items;
+                const float* p = a.p + size_t(row0 + t0 + t) * a.ld + head * n;
+                const float* pk = p + a.heads * n;
+                if (j < half) {
+                    const float2 cs = rotation(a.turns[j], pos0 + t0 + t);
+                    const float2 q = rotate_pair(p[j], p[j + half], cs), k = rotate_pair(pk[j], pk[j + half], cs);
+                    qs[t * n + j] = q.x, qs[t * n + j + half] = q.y;
+                    ks[t * n + j] = k.x * scale, ks[t * n + j + half] = k.y * scale;
+                } else {
+                    qs[t * n + j + half] = p[j + half], ks[t * n + j + half] = pk[j + half] * scale;
+                }
+            }
+            for (int i = tid; i < nt * kScanRows; i += kScanThreads) {
+                const int t = i / kScanRows, v = v0 + i % kScanRows;
+                xs[i] = v < a.vdim ? a.p[size_t(row0 + t0 + t) * a.ld + 2 * a.heads * n + head * a.vdim + v] : 0.0f;
+            }
         } else {
             for (int i = tid; i < nt * n; i += kScanThreads) {
                 const int t = i / n, c = head * n + i % n;
@@ -119,12 +144,12 @@ __global__ void __launch_bounds__(kScanThreads) gated_scan_kernel(const __grid_c
             float x[4], acc[4] = {};
 #pragma unroll
             for (int j = 0; j < 4; ++j) x[j] = xs[t * kScanRows + warp * 4 + j];
-            const float decay = KIND == kScanMamba2 ? one[kScanStage + t] : 0.0f, step = KIND == kScanMamba2 ? one[t] : 1.0f;
+            const float decay = KIND == kScanMamba2 ? one[kScanStage + t] : KIND == kScanRetention ? a.decay[head] : 0.0f, step = KIND == kScanMamba2 ? one[t] : 1.0f;
 #pragma unroll
             for (int e = 0; e < kScanMaxPer; ++e) {
                 const int i = lane + 32 * e;
                 if (i < n) {
-                    const float k = ks[t * n + i] * step, q = qs[t * n + i], d = KIND == kScanMamba2 ? decay : as[t * n + i];
+                    const float k = ks[t * n + i] * step, q = qs[t * n + i], d = KIND != kScanHgrn2 ? decay : as[t * n + i];
 #pragma unroll
                     for (int j = 0; j < 4; ++j) {
                         s[j][e] = d * s[j][e] + k * x[j];
