@@ -15,12 +15,12 @@ ROW_LIMIT = 1 << 20  # values drawn per tensor; larger tensors repeat them from 
 
 def bf16_bits(a) -> np.ndarray:
     """float32 -> bfloat16 bit patterns, round to nearest even."""
-    u = np.ascontiguousarray(a, np.float32).view(np.uint32)
-    return ((u + 0x7FFF + ((u >> 16) & 1)) >> 16).astype(np.uint16)
+    u = np.ascontiguousarray(a, np.float32).view(np.uint32).reshape(np.shape(a))
+    return np.asarray((u + 0x7FFF + ((u >> 16) & 1)) >> 16).astype(np.uint16)
 
 
 def bf16_floats(bits: np.ndarray) -> np.ndarray:
-    return (bits.astype(np.uint32) << 16).view(np.float32)
+    return np.asarray(bits.astype(np.uint32) << 16).view(np.float32)
 
 
 def write_safetensors(path: str, tensors: dict) -> None:
@@ -128,4 +128,91 @@ def random_lasosun(config: dict, seed: int) -> dict:
         if bits.size < n:
             bits = np.resize(bits, n)
         out[name] = bits.reshape(shape)
+    return out
+
+
+# ---- Tosevik -----------------------------------------------------------------------------------------------------------------------------
+def retention(heads, dim, vdim, decay=None, rot=None, base=10000.0) -> dict:
+    """decay: one number per head (default: memories of 32 tokens and up); rot: rotated dimensions (default: all)."""
+    decay = [1.0 - 2.0 ** -(5 + 5 * h / max(heads - 1, 1)) for h in range(heads)] if decay is None else list(decay)
+    return {"heads": heads, "dim": dim, "vdim": vdim, "decay": decay, "rot": {"dims": dim if rot is None else rot, "base": base}}
+
+
+def logistic(heads, kv_heads, dim, vdim, coef=0.3, every=64, scale=None) -> dict:
+    return {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": dim ** -0.5 if scale is None else scale, "q_temp": {"coef": coef, "every": every}}
+
+
+def experts(count, top, ff, shared_ff, groups=1, keep=1, scale=1.0) -> dict:
+    return {"kind": "moe", "expert": {"ff": ff}, "shared": {"ff": shared_ff}, "router": {"experts": count, "top": top, "scale": scale, "groups": {"count": groups, "keep": keep}}}
+
+
+def retention_layer(mixer: dict, mlp: dict | None = None) -> dict:
+    return {"type": "retention", "mixer": mixer, "mlp": mlp}
+
+
+def parallel_layer(left: dict, right: dict, mlp: dict | None = None) -> dict:
+    return {"type": "parallel", "mixer": {"left": left, "right": right}, "mlp": mlp}
+
+
+def tosevik_config(layers, width, vocab, eps=1e-6) -> dict:
+    return {"architecture": "Tosevik", "width": width, "vocab": vocab, "norm": {"eps": eps}, "layers": layers}
+
+
+def tosevik_shapes(config: dict) -> dict:
+    """Tensor name -> shape, in file order."""
+    W = config["width"]
+    norm = lambda name: {name: (W,), name + ".b": (W,), name + ".alpha": ()}
+
+    def ret(m, p):
+        qk, v = m["heads"] * m["dim"], m["heads"] * m["vdim"]
+        return {p + "q": (qk, W), p + "k": (qk, W), p + "v": (v, W), p + "g": (v, W), p + "o": (W, v)}
+
+    def swiglu(p, ff):
+        return {p + "gate": (ff, W), p + "up": (ff, W), p + "down": (W, ff)}
+
+    out = {"embed": (config["vocab"], W)} | norm("embed.norm")
+    for i, l in enumerate(config["layers"]):
+        p, m, mlp = f"l{i}.", l["mixer"], l["mlp"]
+        out |= norm(p + "norm1") | (norm(p + "norm2") if mlp else {})
+        if l["type"] == "retention":
+            out |= ret(m, p + "mix.")
+        else:
+            a = m["left"]
+            q, k, v = a["heads"] * a["dim"], a["kv_heads"] * a["dim"], a["kv_heads"] * a["vdim"]
+            x = p + "mix.left."
+            out |= {x + "q": (q, W), x + "k": (k, W), x + "v": (v, W), x + "q.norm": (q,), x + "k.norm": (k,), x + "pb": (a["heads"],), x + "o": (W, a["heads"] * a["vdim"])}
+            out |= ret(m["right"], p + "mix.right.") | {x + "out": (W,), p + "mix.right.out": (W,)}
+        if mlp:
+            for e in range(mlp["router"]["experts"]):
+                out |= swiglu(p + f"mlp.e{e}.", mlp["expert"]["ff"])
+            out |= {p + "mlp.router": (mlp["router"]["experts"], W)} | swiglu(p + "mlp.shared.", mlp["shared"]["ff"]) | {p + "mlp.shared.sg": (1, W)}
+        out[p + "dwa"] = (i + 2,)
+    return out | norm("final.norm") | {"head": (config["vocab"], W)}
+
+
+def random_tosevik(config: dict, seed: int) -> dict:
+    """Seeded bfloat16 weights (bit patterns): matrices with unit output variance for unit inputs; averages over depth that add up to one."""
+    rng = np.random.default_rng(seed)
+    out = {}
+    for name, shape in tosevik_shapes(config).items():
+        leaf, n = name.rsplit(".", 1)[-1], int(np.prod(shape))
+        if leaf == "alpha":
+            a = rng.uniform(0.4, 0.9, n)
+        elif leaf == "b":
+            a = rng.normal(0, 0.1, n)
+        elif leaf in ("norm", "norm1", "norm2", "out"):
+            a = rng.uniform(0.7, 1.3, n)
+        elif leaf == "pb":
+            a = rng.normal(-3.0, 0.5, n)
+        elif leaf == "dwa":
+            a = rng.normal(0, 0.3, n)
+            a[-1] = 1.0 - a[:-1].sum()
+        elif leaf == "embed":
+            a = rng.normal(0, 1.0, min(n, ROW_LIMIT))
+        elif leaf == "router":
+            a = rng.normal(0, 2.0 * shape[1] ** -0.5, min(n, ROW_LIMIT))
+        else:
+            a = rng.normal(0, shape[1] ** -0.5, min(n, ROW_LIMIT))
+        bits = bf16_bits(a)
+        out[name] = (np.resize(bits, n) if bits.size < n else bits).reshape(shape)
     return out
