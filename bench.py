@@ -469,9 +469,22 @@ def layered_config(size: str, layers=None, positions: int = 8192):
     return mf.lasosun_config([kinds[i % 3]() for i in range(layers or L)], W, 32768, positions)
 
 
+def tosevik_bench_config(size: str, layers=None):
+    """The same widths, layer counts and multiply-adds of the feed-forward: 32 experts, of which a token uses 7 and the shared one, each an eighth of
+    the dense width. Two layers of retention (heads of 128 x 256), then one of attention (heads of 128, four query heads per KV head) beside
+    retention (heads of 128 x 128)."""
+    from quintrit_b200 import model_folder as mf
+
+    W, ff, L = LAYERED_SIZES[size]
+    moe = mf.experts(32, 7, ff // 8, ff // 8, groups=4, keep=2, scale=1.5)
+    kinds = [lambda: mf.retention_layer(mf.retention(W // 128, 128, 256), moe), lambda: mf.retention_layer(mf.retention(W // 128, 128, 256), moe),
+             lambda: mf.parallel_layer(mf.logistic(W // 128, W // 512, 128, 128), mf.retention(W // 256, 128, 128), moe)]
+    return mf.tosevik_config([kinds[i % 3]() for i in range(layers or L)], W, 32768)
+
+
 def run_layered(args, local_rank: int):
-    """Prompt ingestion and decoding of layered models (Lasosun) beside a ternary LLaMA-form model of the same width, feed-forward, layer count and
-    vocabulary: tokens/s of a 4096-token prompt (wall clock around the call that ends with the logits on the host, best of three), and device
+    """Prompt ingestion and decoding of layered models (Lasosun, Tosevik) beside a ternary LLaMA-form model of the same width, feed-forward, layer
+    count and vocabulary: tokens/s of a 4096-token prompt (wall clock around the call that ends with the logits on the host, best of three), and device
     time of a decode step at that context. Fractions are of the measured HBM rate (bytes of the weights a step reads) and of the measured dense
     bf16 rate (multiply-adds of the projections)."""
     import shutil
@@ -491,15 +504,7 @@ def run_layered(args, local_rank: int):
     for size in args.layered_sizes.split(","):
         cfg = layered_config(size, args.decode_layers)
         W, ff = cfg["width"], cfg["layers"][0]["mlp"]["ff"]
-        shapes = mf.lasosun_shapes(cfg)
-        matrix = sum(int(np.prod(s)) for n, s in shapes.items() if len(s) == 2 and n not in ("embed", "pos") and not n.endswith("conv"))
         head = cfg["vocab"] * W
-        tmp = tempfile.mkdtemp()
-        try:
-            mf.write_folder(tmp, cfg, mf.random_lasosun(cfg, 5))
-            dec = q.Decoder.open(tmp, device=local_rank)
-        finally:
-            shutil.rmtree(tmp)
         prompt = synth.prompt_tokens(6, args.layered_prompt, cfg["vocab"])
 
         def ingest(dec):
@@ -516,8 +521,23 @@ def run_layered(args, local_rank: int):
             return {"prefill_tokens_per_s": round(len(prompt) / t), "prefill_ms": round(t * 1e3, 2), "prefill_frac_of_bf16": round(2 * macs * len(prompt) / t / tensor / 1e12, 3),
                     "decode_ms": round(ms, 4), "decode_tokens_per_s": round(1e3 / ms, 1), "weight_bytes": int(weight_bytes), "decode_frac_of_hbm": round(weight_bytes / (ms * 1e-3) / hbm / 1e9, 3)}
 
-        r = {"size": size, "width": W, "ff": ff, "layers": len(cfg["layers"]), "prompt": len(prompt), "lasosun_bf16": row(dec, 2 * (matrix + head), matrix)}
-        dec.free()
+        r = {"size": size, "width": W, "ff": ff, "layers": len(cfg["layers"]), "prompt": len(prompt)}
+        for design in args.layered_designs.split(","):
+            c, shapes, make = (cfg, mf.lasosun_shapes(cfg), mf.random_lasosun) if design == "lasosun" else (t := tosevik_bench_config(size, args.decode_layers), mf.tosevik_shapes(t), mf.random_tosevik)
+            matrix = 0  # multiply-adds of a token's projections = weights that it reads
+            for n, s in shapes.items():
+                if len(s) != 2 or n in ("embed", "pos", "head") or n.endswith("conv"):
+                    continue
+                expert = n.split(".")[2][1:] if ".mlp.e" in n else ""
+                matrix += int(np.prod(s)) * (not expert.isdigit() or int(expert) < c["layers"][int(n[1:n.index(".")])]["mlp"]["router"]["top"])
+            tmp = tempfile.mkdtemp()
+            try:
+                mf.write_folder(tmp, c, make(c, 5))
+                dec = q.Decoder.open(tmp, device=local_rank, context=max(8192, len(prompt) + 64))
+            finally:
+                shutil.rmtree(tmp)
+            r[design + "_bf16"] = row(dec, 2 * (matrix + head), matrix)
+            dec.free()
         if not args.no_decode:  # the ternary model
             dims = dict(hidden=W, inter=ff, layers=len(cfg["layers"]), q_heads=W // 128, kv_heads=W // 512, head_dim=128, vocab=cfg["vocab"])
             spec = synth.torch_model(dims, torch.device("cuda", local_rank), min(8192, len(prompt) + 256))
@@ -1031,7 +1051,8 @@ def main():
     ap.add_argument("--block-scaled-decode", action="store_true", help="run only a whole-token decode of a block-scaled (Q2_0) model of the decode shape (profiling aid)")
     ap.add_argument("--decode-shape", default="falcon3_10b", choices=["falcon3_10b", "bitnet_2b"])
     ap.add_argument("--decode-layers", type=int, default=None, help="fewer layers than the shape has (experiments)")
-    ap.add_argument("--layered-model", action="store_true", help="run only prompt ingestion and decoding of layered models (Lasosun) beside a ternary model of equal size")
+    ap.add_argument("--layered-model", action="store_true", help="run only prompt ingestion and decoding of layered models beside a ternary model of equal size")
+    ap.add_argument("--layered-designs", default="lasosun,tosevik", help="with --layered-model: which designs")
     ap.add_argument("--layered-sizes", default="1k,2k,4k", help="with --layered-model: which of %s" % ", ".join(LAYERED_SIZES))
     ap.add_argument("--layered-prompt", type=int, default=4096, help="with --layered-model: prompt tokens")
     ap.add_argument("--moe-only", action="store_true", help="run only the mixture-of-experts block leg and print its object")

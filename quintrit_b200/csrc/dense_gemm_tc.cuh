@@ -63,6 +63,63 @@ __device__ __forceinline__ void dense_end(const DenseSeg& g, int row, int token,
     }
 }
 
+// Sixteen results of a weight row, tokens `token` .. token + n - 1 (n <= 16), of a plain- or grouped-form tile in 16-bit storage. Lanes 2 i and
+// 2 i + 1 hold rows 2 i and 2 i + 1: where both rows end up beside one another, each of the two lanes takes eight tokens for both.
+__device__ __forceinline__ void dense_end16(const DenseSeg& g, int row, int token, int n, const uint32_t (&v)[16]) {
+    const int kind = g.kind, lane = threadIdx.x & 31;
+    const size_t ld = g.ld;
+    if (kind == kSegPlain || kind == kSegSigmoid) {
+        if (row >= g.rows) return;
+        float* f = g.f + size_t(token) * ld + row;
+        if (kind == kSegPlain) {
+            if (n >= 16) {
+#pragma unroll
+                for (int i = 0; i < 16; ++i) f[i * ld] = __uint_as_float(v[i]);
+            } else {
+#pragma unroll
+                for (int i = 0; i < 16; ++i)
+                    if (i < n) f[i * ld] = __uint_as_float(v[i]);
+            }
+            return;
+        }
+        const float bias = g.bias != nullptr ? g.bias[row] : 0.0f;
+#pragma unroll
+        for (int i = 0; i < 16; ++i)
+            if (i < n) f[i * ld] = sigmoid_f(__uint_as_float(v[i]) + bias);
+        return;
+    }
+    const bool odd = lane & 1;
+    float a[8], b[8];  // of rows 2 i and 2 i + 1, the first or the last eight tokens
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+        const uint32_t other = __shfl_xor_sync(0xffffffffu, odd ? v[i] : v[i + 8], 1);
+        a[i] = __uint_as_float(odd ? other : v[i]), b[i] = __uint_as_float(odd ? v[i + 8] : other);
+    }
+    const int mine = odd ? 8 : 0, even = row & ~1;
+    if (even >= g.rows) return;
+    bf16* t = static_cast<bf16*>(g.t) + size_t(token + mine) * ld;
+    if (kind == kSegSwiGlu) {
+        t += even >> 1;
+#pragma unroll
+        for (int i = 0; i < 8; ++i)
+            if (mine + i < n) t[i * ld] = __float2bfloat16_rn(__fdividef(a[i], 1.0f + __expf(-a[i])) * b[i]);
+        return;
+    }
+    t += even;
+    if (ld % 2 == 0 && even + 1 < g.rows) {
+#pragma unroll
+        for (int i = 0; i < 8; ++i)
+            if (mine + i < n) *reinterpret_cast<__nv_bfloat162*>(t + i * ld) = __floats2bfloat162_rn(a[i], b[i]);
+        return;
+    }
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+        if (mine + i < n) {
+            t[i * ld] = __float2bfloat16_rn(a[i]);
+            if (even + 1 < g.rows) t[i * ld + 1] = __float2bfloat16_rn(b[i]);
+        }
+}
+
 namespace dense_detail {
 __device__ __forceinline__ void tma_load_2d(uint32_t dst, const CUtensorMap* map, int x, int y, uint32_t bar) {
     asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];" ::"r"(dst), "l"(map), "r"(x), "r"(y), "r"(bar) : "memory");
@@ -222,32 +279,46 @@ __global__ void __launch_bounds__(kDenseThreads, 1) dense_gemm_tc_kernel(const _
                     if (has2) tmem_load16(acc + N + c0, v2);
                     asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
                     if (row < a.width) {
+                        const size_t at = size_t(token0 + c0) * a.width + row;
+                        const int n16 = min(16, n_here - c0);
                         float add[16], x[16];
 #pragma unroll
                         for (int i = 0; i < 16; ++i) {
-                            const size_t at = size_t(token0 + min(c0 + i, n_here - 1)) * a.width + row;
-                            add[i] = __uint_as_float(v1[i]) * (a.gate1 != nullptr ? a.gate1[at] : a.token_gate != nullptr ? a.token_gate[token0 + min(c0 + i, n_here - 1)] : 1.0f);
-                            if (has2) add[i] += __uint_as_float(v2[i]) * (a.gate2 != nullptr ? a.gate2[at] : 1.0f);
-                            x[i] = a.x[at];
+                            x[i] = i < n16 ? a.x[at + i * size_t(a.width)] : 0.0f;
+                            add[i] = __uint_as_float(v1[i]);
+                        }
+                        if (a.gate1 != nullptr) {
+#pragma unroll
+                            for (int i = 0; i < 16; ++i) add[i] *= i < n16 ? a.gate1[at + i * size_t(a.width)] : 0.0f;
+                        } else if (a.token_gate != nullptr) {
+#pragma unroll
+                            for (int i = 0; i < 16; ++i) add[i] *= i < n16 ? a.token_gate[token0 + c0 + i] : 0.0f;
+                        }
+                        if (has2) {
+                            if (a.gate2 != nullptr) {
+#pragma unroll
+                                for (int i = 0; i < 16; ++i) add[i] = fmaf(__uint_as_float(v2[i]), i < n16 ? a.gate2[at + i * size_t(a.width)] : 0.0f, add[i]);
+                            } else {
+#pragma unroll
+                                for (int i = 0; i < 16; ++i) add[i] += __uint_as_float(v2[i]);
+                            }
                         }
 #pragma unroll
                         for (int i = 0; i < 16; ++i)
-                            if (c0 + i < n_here) a.x[size_t(token0 + c0 + i) * a.width + row] = x[i] + add[i];
+                            if (i < n16) a.x[at + i * size_t(a.width)] = x[i] + add[i];
                     }
                 }
             } else {
                 const DenseStack& st = a.stack[prob];
                 const int stack_row0 = GROUPED ? row0 - a.runs[item / a.row_tiles[0]].row0 : row0;
                 const DenseSeg& g = dense_seg_of(st, stack_row0);
-                for (int c0 = turn * 16; c0 < n_here; c0 += 32) {
-                    uint32_t v[16];
-                    tmem_load16(acc + c0, v);
+                for (int c0 = turn * 32; c0 < n_here; c0 += 64) {  // (the columns behind n_here exist: N is a multiple of 64)
+                    uint32_t v[2][16];
+                    tmem_load16(acc + c0, v[0]);
+                    tmem_load16(acc + c0 + 16, v[1]);
                     asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
-#pragma unroll
-                    for (int i = 0; i < 16; ++i) {
-                        const float val = __uint_as_float(v[i]), pair = __shfl_xor_sync(0xffffffffu, val, 1);
-                        if (c0 + i < n_here) dense_end<bf16>(g, stack_row0 + r - g.row0, token0 + c0 + i, val, pair);
-                    }
+                    dense_end16(g, stack_row0 + r - g.row0, token0 + c0, n_here - c0, v[0]);
+                    if (c0 + 16 < n_here) dense_end16(g, stack_row0 + r - g.row0, token0 + c0 + 16, n_here - c0 - 16, v[1]);
                 }
             }
             asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");

@@ -530,6 +530,7 @@ inline int layered_decoder_setup(quintrit_b200_decoder* d, const std::shared_ptr
                              reinterpret_cast<const void*>(pooled_attention_kernel<float, true>), reinterpret_cast<const void*>(pooled_attention_kernel<float, false>),
                              reinterpret_cast<const void*>(dense_gemm_tc_kernel<128, kDenseDual>), reinterpret_cast<const void*>(dense_gemm_tc_kernel<128, kDensePlain>),
                              reinterpret_cast<const void*>(dense_gemm_tc_kernel<256, kDensePlain>), reinterpret_cast<const void*>(dense_gemm_tc_kernel<128, kDenseGrouped>),
+                             reinterpret_cast<const void*>(dense_gemm_tc_kernel<256, kDenseGrouped>),
                              reinterpret_cast<const void*>(chunk_scan_kernel<kScanMamba2, 32>), reinterpret_cast<const void*>(chunk_scan_kernel<kScanMamba2, 64>),
                              reinterpret_cast<const void*>(chunk_scan_kernel<kScanMamba2, 128>), reinterpret_cast<const void*>(chunk_scan_kernel<kScanHgrn2, 32>),
                              reinterpret_cast<const void*>(chunk_scan_kernel<kScanHgrn2, 64>), reinterpret_cast<const void*>(chunk_scan_kernel<kScanHgrn2, 128>),
@@ -916,7 +917,7 @@ int layered_experts(quintrit_b200_decoder* d, size_t li, int n) {
     cudaStream_t s = d->stream;
     MoeRouteArgs r{};
     r.router = layered_router(sp), r.tokens = n, r.logits = x.logits, r.chosen = x.chosen, r.weight = x.weight, r.count = x.count, r.rank = x.rank, r.first = x.first, r.row = x.row;
-    r.up_runs = x.up_runs, r.down_runs = x.down_runs, r.n_runs = x.n_runs, r.up_rows = l.expert_rows(), r.down_rows = l.expert_down_rows(), r.tile = sizeof(T) == 2 ? 128 : kF32Tile;
+    r.up_runs = x.up_runs, r.down_runs = x.down_runs, r.n_runs = x.n_runs, r.up_rows = l.expert_rows(), r.down_rows = l.expert_down_rows(), r.tile = sizeof(T) != 2 ? kF32Tile : n * sp.top >= 160 * sp.experts ? 256 : 128;  // (the wider tile where an expert's share fills most of it)
     moe_route_kernel<<<(n + 3) / 4, 128, size_t(4) * sp.experts * sizeof(float), s>>>(r);
     QTB_LAUNCH_CHECK();
     moe_plan_kernel<<<1, 1024, 0, s>>>(r);
@@ -928,8 +929,10 @@ int layered_experts(quintrit_b200_decoder* d, size_t li, int n) {
         a.tokens = n * sp.top, a.n_prob = 1, a.k_steps[0] = w.pitch / kDenseK, a.row_tiles[0] = rows / kDenseM, a.runs = runs, a.n_runs = x.n_runs;
         a.stack[0] = layered_stack(w), a.stack[0].n_seg = 1, a.stack[0].seg[0] = seg, a.status = d->d_counters + 2, a.spin_limit = kDenseSpinLimit;
         const int most = n * sp.top / r.tile + std::min(sp.experts, n * sp.top);  // runs there can be
+        const int blocks = std::min(d->sm_count, most * a.row_tiles[0]);
         if constexpr (sizeof(T) == 2)
-            dense_gemm_tc_kernel<128, kDenseGrouped><<<std::min(d->sm_count, most * a.row_tiles[0]), kDenseThreads, dense_smem(128), s>>>(w.map, map, w.map, map, a);
+            r.tile == 256 ? dense_gemm_tc_kernel<256, kDenseGrouped><<<blocks, kDenseThreads, dense_smem(256), s>>>(w.map, map, w.map, map, a)
+                          : dense_gemm_tc_kernel<128, kDenseGrouped><<<blocks, kDenseThreads, dense_smem(128), s>>>(w.map, map, w.map, map, a);
         else
             dense_gemm_f32_kernel<kDenseGrouped><<<dim3(most, a.row_tiles[0] * (kDenseM / kF32Tile)), 256, 0, s>>>(
                 static_cast<const float*>(w.w), static_cast<const float*>(act), w.pitch, static_cast<const float*>(w.w), static_cast<const float*>(act), w.pitch, a);
