@@ -413,23 +413,28 @@ __global__ void __launch_bounds__(kProjectThreads, 4) out_project_kernel(const _
     bool first = true;
     if (unit0 < units) {
         const OutProjectArgs::Mixer& m = a.mix[unit0 >= a.width ? 1 : 0];
-        load_pieces<T, 1>(head, static_cast<const T*>(m.w) + size_t(unit0 % a.width) * m.pitch, m.pitch, lane);
+        const T* w = static_cast<const T*>(m.w) + size_t(unit0 % a.width) * m.pitch;
+        load_pieces<T, 1>(head, w, m.pitch, lane);
+        if (lane == 0) l2_prefetch(w, m.pitch * sizeof(T));
     }
     pdl_wait();
+    float* gates = act_smem + a.mix[0].pitch + (a.n > 1 ? a.mix[1].pitch : 0);
     for (int k = 0; k < a.n; ++k) {
         const OutProjectArgs::Mixer& m = a.mix[k];
         // a block all of whose rows belong to the other mixer leaves this one's vector out
         const int lo = blockIdx.x * (kProjectThreads / 32), hi = lo + kProjectThreads / 32 - 1;
         if (warps >= units && (k == 0 ? lo >= a.width : hi < a.width)) continue;
         float* y = act_smem + (k > 0 ? a.mix[0].pitch : 0);
-        const float* src = m.y + size_t(token) * m.inner;
-#pragma unroll 4
+        const float *src = m.y + size_t(token) * m.inner, *gate = m.gate != nullptr ? m.gate + size_t(token) * m.gate_ld : nullptr;
+#pragma unroll 8
         for (int i = tid; i < m.pitch; i += kProjectThreads) {
-            const float v = i < m.inner ? src[i] : 0.0f;
+            const float v = i < m.inner ? src[i] : 0.0f, z = gate != nullptr && i < m.inner ? gate[i] : 0.0f;
             y[act_index<T>(i, m.pitch)] = m.parts > 0 ? v : round_to<T>(v);
+            if (gate != nullptr && i < m.inner) gates[i] = z;
         }
         __syncthreads();
-        if (m.parts > 0) parts_norm<T>(y, m.inner, m.pitch, m.parts, a.eps, nullptr, 1, m.gate != nullptr ? m.gate + size_t(token) * m.gate_ld : nullptr, red);
+        if (m.parts > 0) parts_norm<T>(y, m.inner, m.pitch, m.parts, a.eps, nullptr, 1, gate != nullptr ? gates : nullptr, red);
+        else __syncthreads();
     }
     for (int unit = unit0; unit < units; unit += warps) {
         const int k = unit >= a.width ? 1 : 0, row = unit - k * a.width;
@@ -544,7 +549,44 @@ __global__ void __launch_bounds__(256) rows_kernel(const __grid_constant__ RowsA
         il = 0.5f / sqrtf(sl / static_cast<float>(a.width) + a.eps), ir = 0.5f / sqrtf(sr / static_cast<float>(a.width) + a.eps);
     }
     float ss = 0.0f;
-    for (int i = tid; i < a.width; i += 256) {
+    if (a.width % 4 == 0) {  // four elements at a time, every vector's loads together
+        const auto at4 = [](const float* p) { return *reinterpret_cast<const float4*>(p); };
+        const auto fma4 = [](float f, const float4& x, float4& s) { s.x = fmaf(f, x.x, s.x), s.y = fmaf(f, x.y, s.y), s.z = fmaf(f, x.z, s.z), s.w = fmaf(f, x.w, s.w); };
+        for (int i = tid * 4; i < a.width; i += 256 * 4) {
+            float4 v = at4(a.x + row + i);
+            if (pair) {
+                const float4 l = at4(a.pair.r[0] + row + i), r = at4(a.pair.r[1] + row + i), wl = at4(a.pair.w[0] + i), wr = at4(a.pair.w[1] + i);
+                v.x += l.x * il * wl.x + r.x * ir * wr.x, v.y += l.y * il * wl.y + r.y * ir * wr.y, v.z += l.z * il * wl.z + r.z * ir * wr.z, v.w += l.w * il * wl.w + r.w * ir * wr.w;
+            }
+            if (a.pick != nullptr) {
+                float4 s = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll 8
+                for (int k = 0; k < a.top; ++k) {
+                    const T* p = static_cast<const T*>(a.pick) + size_t(a.pick_row[t * a.top + k]) * a.width + i;
+                    float4 f;
+                    if constexpr (sizeof(T) == 2) {
+                        const uint2 u = *reinterpret_cast<const uint2*>(p);
+                        f = make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xffff0000u), __uint_as_float(u.y << 16), __uint_as_float(u.y & 0xffff0000u));
+                    } else {
+                        f = at4(p);
+                    }
+                    fma4(a.pick_weight[t * a.top + k], f, s);
+                }
+                v.x += s.x, v.y += s.y, v.z += s.z, v.w += s.w;
+            }
+            if (a.depth.n > 0) {
+                *reinterpret_cast<float4*>(a.depth.x + (a.depth.n - 1) * a.depth.stride + row + i) = v;
+                float4 s = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll 8
+                for (int j = 0; j < a.depth.n - 1; ++j) fma4(a.depth.w[j], at4(a.depth.x + j * a.depth.stride + row + i), s);
+                fma4(a.depth.w[a.depth.n - 1], v, s);
+                v = s;
+            }
+            if (a.x_out != a.x || pair || a.pick != nullptr || a.depth.n > 0) *reinterpret_cast<float4*>(a.x_out + row + i) = v;
+            *reinterpret_cast<float4*>(act_smem + i) = v;
+            ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+        }
+    } else for (int i = tid; i < a.width; i += 256) {
         float v = a.x[row + i];
         if (pair) v += a.pair.r[0][row + i] * il * a.pair.w[0][i] + a.pair.r[1][row + i] * ir * a.pair.w[1][i];
         if (a.pick != nullptr) {
@@ -565,6 +607,7 @@ __global__ void __launch_bounds__(256) rows_kernel(const __grid_constant__ RowsA
     }
     if (a.h == nullptr) return;
     const float inv = a.norm.b == nullptr ? 1.0f / sqrtf(block_sum(ss, red) / static_cast<float>(a.width) + a.eps) : 1.0f;
+    __syncthreads();  // (the sums lie in other threads' places)
     for (int i = tid; i < a.width; i += 256) static_cast<T*>(a.h)[t * a.pitch + i] = to_storage<T>(norm_value(a.norm, act_smem[i], inv, i));
 }
 

@@ -100,17 +100,20 @@ __global__ void __launch_bounds__(kProjectThreads, 4) moe_up_step_kernel(const _
         choose_experts(a.router, a.logits, act_smem + a.pitch, chosen, weight);
         if (blockIdx.x == 0 && tid < a.router.top) a.chosen[tid] = chosen[tid], a.weight[tid] = weight[tid];
     }
-    constexpr int kPer = 16 / sizeof(T);
-    for (int i = tid; i < a.pitch / kPer; i += kProjectThreads) act_put_storage(act_smem, i, a.pitch, static_cast<const T*>(a.h));
+    else {
+        constexpr int kPer = 16 / sizeof(T);
+        for (int i = tid - 32; i < a.pitch / kPer; i += kProjectThreads - 32) act_put_storage(act_smem, i, a.pitch, static_cast<const T*>(a.h));
+    }
     __syncthreads();
-    for (int unit = blockIdx.x * (kProjectThreads / 32) + (tid >> 5); unit < units; unit += warps) {
-        const int k = unit / a.ff, i = unit % a.ff;
-        const T* rows = static_cast<const T*>(a.w) + (size_t(chosen[k]) * a.rows_pad + 2 * i) * a.pitch;
-        RowHead<2> head;
+    auto rows_of = [&](int unit) { return static_cast<const T*>(a.w) + (size_t(chosen[unit / a.ff]) * a.rows_pad + 2 * (unit % a.ff)) * a.pitch; };
+    RowHead<2> head;
+    int unit = blockIdx.x * (kProjectThreads / 32) + (tid >> 5);
+    if (unit < units) load_pieces<T, 2>(head, rows_of(unit), a.pitch, tid & 31);
+    for (; unit < units; unit += warps) {
         float v[2];
-        load_pieces<T, 2>(head, rows, a.pitch, tid & 31);
-        dot_rows<T, 2>(rows, a.pitch, act_smem, head, v);
-        if ((tid & 31) == 0) static_cast<T*>(a.m)[size_t(k) * a.m_pitch + i] = to_storage<T>(silu_f(v[0]) * v[1]);
+        dot_rows<T, 2>(rows_of(unit), a.pitch, act_smem, head, v);
+        if (unit + warps < units) load_pieces<T, 2>(head, rows_of(unit + warps), a.pitch, tid & 31);
+        if ((tid & 31) == 0) static_cast<T*>(a.m)[size_t(unit / a.ff) * a.m_pitch + unit % a.ff] = to_storage<T>(silu_f(v[0]) * v[1]);
     }
 }
 
@@ -131,7 +134,7 @@ struct MoeDownStepArgs {
     int rows;               // rows of the result per block
 };
 
-constexpr int kMoeDownRows = 16;  // at most
+constexpr int kMoeDownRows = kProjectThreads / 32;  // at most: a warp ends a row
 
 // A block takes a few rows of the result; its warps share the products of these rows with the activations of every chosen expert.
 template <typename T>
@@ -148,39 +151,68 @@ __global__ void __launch_bounds__(kProjectThreads) moe_down_step_kernel(const __
         return k < a.top ? static_cast<const T*>(a.w) + (size_t(a.chosen[k]) * a.rows_pad + r) * a.pitch : static_cast<const T*>(a.shared_w) + size_t(r) * a.shared_pitch;
     };
     auto pitch_of = [&](int unit) { return unit % per < a.top ? a.pitch : a.shared_pitch; };
-    RowHead<1> head, next;
-    if (warp < units) load_pieces<T, 1>(head, row_of(warp), pitch_of(warp), lane);
-    constexpr int kPer = 16 / sizeof(T);
+    // what the ending needs, on its way with the first weights
+    const int end_row = row0 + warp;
+    float x = 0.0f, w = 0.0f, shared_scale = 0.0f, past = 0.0f;
+    if (warp < rows) {
+        x = a.x[end_row], shared_scale = *a.shared_scale;
+        if (lane < a.top) w = a.weight[lane];
+        for (int j = lane; j < a.depth.n - 1; j += 32) past = fmaf(a.depth.w[j], a.depth.x[j * a.depth.stride + end_row], past);
+    }
+    constexpr int kPer = 16 / sizeof(T), kWarps = kProjectThreads / 32;
+    // a warp takes two (row, expert) products at a time, the next two on their way
+    struct Two { uint4 v[2][4]; };
+    auto load = [&](int unit, int p0, Two& b) {
+#pragma unroll
+        for (int k = 0; k < 2; ++k) {
+            const int u = unit + k * kWarps;
+            const T* row = u < units ? row_of(u) : nullptr;
+            const int pieces = u < units ? pitch_of(u) / kPer : 0;
+#pragma unroll
+            for (int i = 0; i < 4; ++i) b.v[k][i] = p0 + 32 * i < pieces ? load_stream(row + size_t(p0 + 32 * i) * kPer) : make_uint4(0, 0, 0, 0);
+        }
+    };
+    Two now, next;
+    load(warp, lane, now);
     for (int i = tid; i < a.top * (a.pitch / kPer); i += kProjectThreads) {
         const int k = i / (a.pitch / kPer), p = i % (a.pitch / kPer);
         act_put_storage(act_smem + k * a.pitch, p, a.pitch, static_cast<const T*>(a.m) + size_t(k) * a.pitch);
     }
     for (int i = tid; i < a.shared_pitch / kPer; i += kProjectThreads) act_put_storage(shared_act, i, a.shared_pitch, static_cast<const T*>(a.shared_m));
     __syncthreads();
-    for (int unit = warp; unit < units; unit += kProjectThreads / 32) {
-        const int after = unit + kProjectThreads / 32, k = unit % per;
-        if (after < units) load_pieces<T, 1>(next, row_of(after), pitch_of(after), lane);
-        float v[1];
-        dot_rows<T, 1>(row_of(unit), pitch_of(unit), k < a.top ? act_smem + k * a.pitch : shared_act, head, v);
-        if (lane == 0) part[unit / per * 33 + k] = v[0];
-        head = next;
+    const int longest = max(a.pitch, a.shared_pitch) / kPer;
+    for (int unit = warp; unit < units; unit += 2 * kWarps) {
+        float sum[2] = {0.0f, 0.0f};
+        for (int p0 = lane; p0 - lane < longest; p0 += 128) {
+            if (p0 != lane) load(unit, p0, now);
+            if (p0 == lane && unit + 2 * kWarps < units) load(unit + 2 * kWarps, lane, next);
+#pragma unroll
+            for (int k = 0; k < 2; ++k) {
+                const int u = unit + k * kWarps;
+                if (u >= units) continue;
+                const int e = u % per, pitch = e < a.top ? a.pitch : a.shared_pitch;
+                const float* act = e < a.top ? act_smem + e * a.pitch : shared_act;
+#pragma unroll
+                for (int i = 0; i < 4; ++i)
+                    if (p0 + 32 * i < pitch / kPer) sum[k] += dot_piece(now.v[k][i], act, p0 + 32 * i, pitch, T());
+            }
+        }
+#pragma unroll
+        for (int k = 0; k < 2; ++k) {
+            const int u = unit + k * kWarps;
+            sum[k] = warp_sum(sum[k]);
+            if (lane == 0 && u < units) part[u / per * 33 + u % per] = sum[k];
+        }
+        now = next;
     }
     __syncthreads();
-    for (int r = warp; r < rows; r += kProjectThreads / 32) {
-        const int row = row0 + r;
-        float s = lane < a.top ? part[r * 33 + lane] * a.weight[lane] : 0.0f;
-        s = warp_sum(s);
-        const float v = a.x[row] + s + part[r * 33 + a.top] * *a.shared_scale;
-        if (a.depth.n == 0) {
-            if (lane == 0) a.x_out[row] = v;
-            continue;
-        }
-        float d = 0.0f;
-        for (int j = lane; j < a.depth.n - 1; j += 32) d = fmaf(a.depth.w[j], a.depth.x[j * a.depth.stride + row], d);
-        d = warp_sum(d);
+    if (warp < rows) {
+        float s = lane < a.top ? part[warp * 33 + lane] * w : 0.0f;
+        s = warp_sum(s), past = warp_sum(past);
         if (lane == 0) {
-            a.depth.x[(a.depth.n - 1) * a.depth.stride + row] = v;
-            a.x_out[row] = fmaf(a.depth.w[a.depth.n - 1], v, d);
+            const float v = x + s + part[warp * 33 + a.top] * shared_scale;
+            if (a.depth.n > 0) a.depth.x[(a.depth.n - 1) * a.depth.stride + end_row] = v;
+            a.x_out[end_row] = a.depth.n > 0 ? fmaf(a.depth.w[a.depth.n - 1], v, past) : v;
         }
     }
 }

@@ -410,7 +410,7 @@ inline void layered_store_view(const LayeredModel& m, const LayeredStore& st, si
 // Shares a decode step's attention is cut into: enough blocks for the device, none below one tile of keys.
 inline int attention_splits(const MixerSpec& l, int ctx, int n, int sm_count) {
     if (l.kind == MixerKind::kLogistic) {
-        const int groups = l.kv_heads * ((l.heads / l.kv_heads + kLaHeads - 1) / kLaHeads) * n;
+        const int gqa = l.heads / l.kv_heads, per = logistic_heads(gqa), groups = l.kv_heads * ((gqa + per - 1) / per) * n;
         return std::max(1, std::min({(ctx + kLaKeys - 1) / kLaKeys, 4 * sm_count / groups, 64}));
     }
     const int groups = l.kv_heads * ((l.heads / l.kv_heads + kPaHeads - 1) / kPaHeads) * n;
@@ -422,6 +422,10 @@ typedef void (*LogisticKernel)(LogisticArgs);
 inline LogisticKernel logistic_kernel_for(int dims) {
     static const LogisticKernel k[] = {logistic_mma_kernel<32>, logistic_mma_kernel<64>, logistic_mma_kernel<96>, logistic_mma_kernel<128>, logistic_mma_kernel<192>, logistic_mma_kernel<256>};
     return k[logistic_dims_slot(dims)];
+}
+typedef void (*LogisticStep)(LogisticArgs, int, int);
+template <typename T, bool OWN> LogisticStep logistic_step_for(int heads) {
+    return heads == 1 ? logistic_step_kernel<T, OWN, 1> : heads == 4 ? logistic_step_kernel<T, OWN, 4> : logistic_step_kernel<T, OWN, 8>;
 }
 // The two kernels of retention over many tokens that are compiled for the head's sizes.
 struct RetentionKernels {
@@ -470,7 +474,7 @@ inline int layered_decoder_setup(quintrit_b200_decoder* d, const std::shared_ptr
                 continue;
             }
             if (l.kind == MixerKind::kLogistic) queries = std::max(queries, size_t(l.heads) * round_up(l.dim, 8));
-            const int per = l.kind == MixerKind::kLogistic ? kLaHeads : kPaHeads;
+            const int per = l.kind == MixerKind::kLogistic ? logistic_heads(l.heads / l.kv_heads) : kPaHeads;
             groups = std::max<size_t>(groups, size_t(l.kv_heads) * ((l.heads / l.kv_heads + per - 1) / per));
             for (int n = 1; n <= kLayeredMaxBatch; ++n) {
                 const size_t sp = attention_splits(l, d->ctx, n, m.sm_count);
@@ -523,7 +527,6 @@ inline int layered_decoder_setup(quintrit_b200_decoder* d, const std::shared_ptr
                              reinterpret_cast<const void*>(embed_norm_kernel<bf16>), reinterpret_cast<const void*>(embed_norm_kernel<float>),
                              reinterpret_cast<const void*>(moe_up_step_kernel<bf16>), reinterpret_cast<const void*>(moe_up_step_kernel<float>),
                              reinterpret_cast<const void*>(moe_down_step_kernel<bf16>), reinterpret_cast<const void*>(moe_down_step_kernel<float>),
-                             reinterpret_cast<const void*>(logistic_step_kernel<bf16>), reinterpret_cast<const void*>(logistic_step_kernel<float>),
                              reinterpret_cast<const void*>(gated_scan_kernel<kScanMamba2>), reinterpret_cast<const void*>(gated_scan_kernel<kScanHgrn2>),
                              reinterpret_cast<const void*>(gated_scan_kernel<kScanRetention>),
                              reinterpret_cast<const void*>(pooled_attention_kernel<bf16, true>), reinterpret_cast<const void*>(pooled_attention_kernel<bf16, false>),
@@ -536,6 +539,8 @@ inline int layered_decoder_setup(quintrit_b200_decoder* d, const std::shared_ptr
                              reinterpret_cast<const void*>(chunk_scan_kernel<kScanHgrn2, 64>), reinterpret_cast<const void*>(chunk_scan_kernel<kScanHgrn2, 128>),
                              reinterpret_cast<const void*>(pooled_attention_mma_kernel<32>), reinterpret_cast<const void*>(pooled_attention_mma_kernel<64>),
                              reinterpret_cast<const void*>(pooled_attention_mma_kernel<128>)};
+    for (int heads : {1, 4, 8})
+        for (LogisticStep k : {logistic_step_for<bf16, true>(heads), logistic_step_for<float, true>(heads), logistic_step_for<float, false>(heads)}) kernels.push_back(reinterpret_cast<const void*>(k));
     for (int dims : {32, 64, 96, 128, 192, 256}) kernels.push_back(reinterpret_cast<const void*>(logistic_kernel_for(dims)));
     for (int rows : {32, 64, 128, 256}) {
         kernels.push_back(reinterpret_cast<const void*>(retention_kernels(rows, 64).state));
@@ -547,12 +552,13 @@ inline int layered_decoder_setup(quintrit_b200_decoder* d, const std::shared_ptr
     const size_t limit = static_cast<size_t>(optin) - 4608;  // (a kernel's own shared variables count too)
     for (const LayeredLayer& ly : m.layers) {
         size_t need = std::max<size_t>({3 * wp * 4, (size_t(ly.mix[0].o.pitch) + (ly.mix.size() > 1 ? ly.mix[1].o.pitch : ly.down.pitch)) * 4});
+        if (!ly.spec.parallel) need = std::max(need, (size_t(ly.mix[0].o.pitch) + 2 * (ly.mix.size() > 1 ? ly.mix[1].o.pitch : ly.mix[0].o.pitch)) * 4);
         if (ly.spec.ff_kind == FfKind::kExperts) need = std::max({need, (size_t(ly.spec.top) * ly.experts_down.pitch + ly.down.pitch) * 4, (wp + 4 * ly.spec.experts) * 4});
         for (const LayeredMixer& x : ly.mix) {
             const MixerSpec& l = x.spec;
             need = std::max(need, size_t(l.inner()) * 4);
             if (l.kind == MixerKind::kAttention) need = std::max(need, pooled_attn_smem(round_up(l.dim, 8), round_up(l.vdim, 8), static_cast<int>(e)));
-            else if (l.kind == MixerKind::kLogistic) need = std::max(need, logistic_step_smem(round_up(l.dim, 8), l.vdim, round_up(l.vdim, 8), static_cast<int>(e)));
+            else if (l.kind == MixerKind::kLogistic) need = std::max(need, logistic_step_smem(logistic_heads(l.heads / l.kv_heads), round_up(l.dim, 8), l.vdim, round_up(l.vdim, 8), static_cast<int>(e)));
             else need = std::max(need, scan_smem(l.key_dim()));
         }
         if (need > limit) return fail(QUINTRIT_ERR_UNSUPPORTED, "a vector of the model does not fit the shared memory of one block (%zu bytes, %zu are available)", need, limit);
@@ -602,6 +608,10 @@ inline int layered_retention_chunks(quintrit_b200_decoder* d, const MixerSpec& l
     retention_work(d->lay->work, l.heads, l.dim, l.vdim, a.tokens, &r.work);
     const RetentionKernels f = retention_kernels(r.work.rows, r.work.v_pad);
     const int chunks = retention_chunks(a.tokens);
+    const bool even = l.dim % 2 == 0 && l.vdim % 2 == 0 && l.rot_dims % 4 == 0 && a.ld % 2 == 0 && (a.p - d->lay->p1) % 2 == 0;
+    const dim3 grid(l.heads, r.work.tokens / kRetPrep);
+    even ? retention_prepare_kernel<true><<<grid, 128, 0, d->stream>>>(r) : retention_prepare_kernel<false><<<grid, 128, 0, d->stream>>>(r);
+    QTB_LAUNCH_CHECK();
     f.state<<<dim3(l.heads, chunks, r.work.v_pad / kRetV), 128, f.state_smem, d->stream>>>(r);
     QTB_LAUNCH_CHECK();
     retention_carry_kernel<<<dim3(r.work.v_pad * r.work.rows / 512, l.heads), 128, 0, d->stream>>>(r);
@@ -696,19 +706,25 @@ int layered_mixer(quintrit_b200_decoder* d, size_t li, int k, int n, const Layer
         a.scale = l.scale, a.eps = d->eps, a.q_norm = w.q_norm, a.k_norm = w.k_norm, a.temp_coef = l.temp_coef, a.temp_every = l.temp_every, a.value_norm = l.value_norm;
         a.slope = w.slope, a.bias = w.logit_bias, a.q = y.q, a.k = st.cache.k, a.v = st.cache.v, a.capacity = st.cache.ring;
         a.out = y.y_t[k], a.out_pitch = w.o.pitch, a.y = y.y[k], a.part = y.part_acc, a.done = y.done;
-        launch_dependent(logistic_prepare_kernel<T>, dim3(n), 256, 0, s, a);
-        QTB_LAUNCH_CHECK();
-        if (sizeof(T) == 2 && tokens > 1) {
-            const int dims = logistic_mma_dims(l.dim, l.vdim);
-            logistic_kernel_for(dims)<<<dim3((tokens + kPmRows - 1) / kPmRows, l.heads), kPmThreads, pooled_mma_smem(dims), s>>>(a);
+        const int gqa = l.heads / l.kv_heads, per = logistic_heads(gqa), hg = l.kv_heads * ((gqa + per - 1) / per), elem = sizeof(T);
+        const size_t smem = logistic_step_smem(per, a.dim_pad, a.vdim, a.vdim_pad, elem);
+        const int key_lanes = std::min(logistic_lanes(a.dim_pad * elem / 16), 32), value_lanes = logistic_lanes(a.vdim_pad * elem / 16);
+        if (tokens == 1) {
+            a.splits = attention_splits(l, d->ctx, n, y.model->sm_count);
+            launch_dependent(logistic_step_for<T, true>(per), dim3(hg, a.splits, n), kLaThreads, smem, s, a, key_lanes, value_lanes);
             QTB_LAUNCH_CHECK();
-            *ready = true;
             return QUINTRIT_OK;
         }
-        a.splits = tokens == 1 ? attention_splits(l, d->ctx, n, y.model->sm_count) : 1;
-        const int hg = l.kv_heads * ((l.heads / l.kv_heads + kLaHeads - 1) / kLaHeads), elem = sizeof(T);
-        launch_dependent(logistic_step_kernel<T>, dim3(hg, a.splits, n), kLaThreads, logistic_step_smem(a.dim_pad, a.vdim, a.vdim_pad, elem), s, a,
-                         std::min(logistic_lanes(a.dim_pad * elem / 16), 32), logistic_lanes(a.vdim_pad * elem / 16));
+        logistic_prepare_kernel<T><<<n, 256, 0, s>>>(a);
+        QTB_LAUNCH_CHECK();
+        if constexpr (sizeof(T) == 2) {
+            const int dims = logistic_mma_dims(l.dim, l.vdim);
+            logistic_kernel_for(dims)<<<dim3((tokens + kPmRows - 1) / kPmRows, l.heads), kPmThreads, pooled_mma_smem(dims), s>>>(a);
+            *ready = true;
+        } else {
+            a.splits = 1;
+            logistic_step_for<T, false>(per)<<<dim3(hg, 1, n), kLaThreads, smem, s>>>(a, key_lanes, value_lanes);
+        }
         QTB_LAUNCH_CHECK();
         return QUINTRIT_OK;
     }
@@ -868,7 +884,7 @@ int layered_sequential_step(quintrit_b200_decoder* d, size_t li, const LayeredTa
     if ((rc = project(a)) != QUINTRIT_OK) return rc;
     OutProjectArgs o{};
     o.width = W, o.n = sets, o.eps = m.spec.eps;
-    size_t smem = 0;
+    size_t smem = 0, gates = 0;
     for (int k = 0; k < sets; ++k) {
         const LayeredMixer& x = l.mix[k];
         bool ready;
@@ -877,8 +893,9 @@ int layered_sequential_step(quintrit_b200_decoder* d, size_t li, const LayeredTa
         t.y = y.y[k], t.inner = x.spec.inner(), t.parts = layered_norm_parts(x.spec), t.w = x.o.w, t.pitch = x.o.pitch;
         if (x.spec.kind == MixerKind::kRetention) t.gate = y.p1 + x.col + x.spec.gate_col(), t.gate_ld = l.spec.in_rows();
         t.out = sets > 1 ? (k > 0 ? y.g2 : y.g1) : y.x, t.add = sets == 1;
-        smem += size_t(x.o.pitch) * sizeof(float);
+        smem += size_t(x.o.pitch) * sizeof(float), gates = std::max(gates, t.gate != nullptr ? size_t(x.o.pitch) * sizeof(float) : 0);
     }
+    smem += gates;
     launch_dependent(out_project_kernel<T>, dim3(std::min((sets * W + warps - 1) / warps, 4 * m.sm_count)), kProjectThreads, smem, s, o);
     QTB_LAUNCH_CHECK();
     PairSum pair{};

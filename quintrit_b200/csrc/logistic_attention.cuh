@@ -38,7 +38,9 @@ struct LogisticArgs {
 
 // Norms of one token's queries, keys and values; the queries' temperature; keys and values go to the cache. One block per token.
 template <typename T>
-__device__ void logistic_prepare(const LogisticArgs& a, int z, float* red) {
+__global__ void __launch_bounds__(256) logistic_prepare_kernel(const __grid_constant__ LogisticArgs a) {
+    __shared__ float red[8];
+    const int z = blockIdx.x;
     const uint32_t slot = a.seq.pos_stride != 0 ? seq_of(a.seq, z) : 0, pos = seq_position(a.seq, a.pos, z);
     const float *q = a.p + size_t(z) * a.ld, *k = q + a.heads * a.dim, *v = k + a.kv_heads * a.dim;
     const int tid = threadIdx.x, nt = blockDim.x, nq = a.heads * a.dim, nk = a.kv_heads * a.dim;
@@ -77,24 +79,19 @@ __device__ void logistic_prepare(const LogisticArgs& a, int z, float* red) {
     }
 }
 
-template <typename T>
-__global__ void __launch_bounds__(256) logistic_prepare_kernel(const __grid_constant__ LogisticArgs a) {
-    __shared__ float red[8];
-    pdl_trigger();
-    pdl_wait();
-    logistic_prepare<T>(a, blockIdx.x, red);
-}
-
 // ---- one query position per block ----------------------------------------------------------------------------------------------------------
-// Up to eight query heads of one kv head over a share of the keys; the last block of a position and head group to finish adds the shares up.
-// 128 keys at a time: a few lanes per key make the weights, then a few lanes per key group add the values up, whose first rows are already on
-// their way. grid: (kv heads * head groups, splits, tokens or sequences)
-constexpr int kLaThreads = 256, kLaKeys = 128, kLaHeads = 8;
+// Up to H query heads of one kv head over a share of the keys; the last block of a position and head group to finish adds the shares up.
+// 128 keys at a time: a few lanes per key make the weights, then a few lanes per key group add the values up. A decode step (OWN) makes the norms
+// itself, takes its own key and value from the projections and appends them to the cache; the first cached keys and values are on their way
+// before it waits for the projections. grid: (kv heads * head groups, splits, tokens or sequences)
+constexpr int kLaThreads = 256, kLaKeys = 128;
+
+inline int logistic_heads(int gqa) { return gqa <= 1 ? 1 : gqa <= 4 ? 4 : 8; }  // H the kernel is compiled for
 
 inline int logistic_lanes(int pieces) { return pieces <= 1 ? 1 : pieces <= 2 ? 2 : pieces <= 4 ? 4 : pieces <= 8 ? 8 : pieces <= 16 ? 16 : pieces <= 32 ? 32 : 64; }
-inline size_t logistic_step_smem(int dim_pad, int vdim, int vdim_pad, int elem) {
+inline size_t logistic_step_smem(int heads, int dim_pad, int vdim, int vdim_pad, int elem) {
     const int lanes = logistic_lanes(vdim_pad * elem / 16), groups = lanes < 32 ? kLaThreads / 32 : kLaThreads / lanes;
-    return size_t(kLaHeads) * (dim_pad + kLaKeys + groups * vdim) * 4;
+    return (size_t(heads) * (dim_pad + kLaKeys + groups * vdim) + dim_pad + vdim_pad + kLaThreads) * 4;
 }
 
 template <typename T> struct Piece;  // 16 bytes of the storage type as floats
@@ -110,88 +107,139 @@ template <> struct Piece<float> {
     static __device__ __forceinline__ void get(const uint4& w, float (&f)[4]) { f[0] = __uint_as_float(w.x), f[1] = __uint_as_float(w.y), f[2] = __uint_as_float(w.z), f[3] = __uint_as_float(w.w); }
 };
 
-template <typename T>
-__global__ void __launch_bounds__(kLaThreads) logistic_step_kernel(const __grid_constant__ LogisticArgs a, int key_lanes, int value_lanes) {
+template <typename T, bool OWN, int H>
+__global__ void __launch_bounds__(kLaThreads, H > 4 ? 1 : 2) logistic_step_kernel(const __grid_constant__ LogisticArgs a, int key_lanes, int value_lanes) {
     extern __shared__ __align__(16) float la_sm[];
     __shared__ bool last_block;
+    __shared__ float sums[2][kLaThreads / 32], own_weight[H];
     constexpr int P = Piece<T>::kN;
     pdl_trigger();
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const int gqa = a.heads / a.kv_heads, groups = (gqa + kLaHeads - 1) / kLaHeads;
-    const int kvh = blockIdx.x / groups, h0 = kvh * gqa + (blockIdx.x % groups) * kLaHeads, nh = min(kLaHeads, (kvh + 1) * gqa - h0);
+    const int gqa = a.heads / a.kv_heads, groups = (gqa + H - 1) / H;
+    const int kvh = blockIdx.x / groups, h0 = kvh * gqa + (blockIdx.x % groups) * H, nh = min(H, (kvh + 1) * gqa - h0);
     const int z = blockIdx.z, split = blockIdx.y;
     const uint32_t slot = a.seq.pos_stride != 0 ? seq_of(a.seq, z) : 0;
-    const int pos = static_cast<int>(seq_position(a.seq, a.pos, z)), total = pos + 1;
+    const int pos = static_cast<int>(seq_position(a.seq, a.pos, z)), total = OWN ? pos : pos + 1;  // keys to be read from the cache
     const int per = (total + a.splits - 1) / a.splits, begin = min(split * per, total), end = min(begin + per, total);
-    float *qs = la_sm, *ws = qs + kLaHeads * a.dim_pad, *red = ws + kLaHeads * kLaKeys;
+    float *qs = la_sm, *ws = qs + H * a.dim_pad, *own_k = ws + H * kLaKeys, *own_v = own_k + a.dim_pad, *red = own_v + a.vdim_pad;
     const size_t krow = size_t(a.kv_heads) * a.dim_pad, vrow = size_t(a.kv_heads) * a.vdim_pad;
-    const T* ks = static_cast<const T*>(a.k) + size_t(slot) * a.capacity * krow + kvh * a.dim_pad;
-    const T* vs = static_cast<const T*>(a.v) + size_t(slot) * a.capacity * vrow + kvh * a.vdim_pad;
+    T* ks = static_cast<T*>(a.k) + size_t(slot) * a.capacity * krow + kvh * a.dim_pad;
+    T* vs = static_cast<T*>(a.v) + size_t(slot) * a.capacity * vrow + kvh * a.vdim_pad;
     const int kpieces = a.dim_pad / P, vpieces = a.vdim_pad / P;
     const int kl = lane & (key_lanes - 1), kg = (tid / key_lanes), kgroups = kLaThreads / key_lanes;        // key_lanes <= 32
     const int vl = tid & (value_lanes - 1), vg = tid / value_lanes, vgroups = kLaThreads / value_lanes;     // value_lanes <= 64
-    pdl_wait();  // (the newest key, and the queries)
-    for (int i = tid; i < kLaHeads * a.dim_pad; i += kLaThreads) qs[i] = i < nh * a.dim_pad ? from_storage(static_cast<const T*>(a.q)[(size_t(z) * a.heads + h0) * a.dim_pad + i]) : 0.0f;
-    float acc[kLaHeads][P];
+    uint4 kr[4], vr[8];
+    auto fetch_keys = [&](int t0, int nt, int r0, int p) {
 #pragma unroll
-    for (int h = 0; h < kLaHeads; ++h)
+        for (int u = 0; u < 4; ++u) {
+            const int r = r0 + u * kgroups;
+            kr[u] = r < nt && p < kpieces ? *reinterpret_cast<const uint4*>(ks + size_t(t0 + r) * krow + p * P) : make_uint4(0, 0, 0, 0);
+        }
+    };
+    auto fetch_values = [&](int t0, int nt, int r0) {  // eight rows of this key group
+#pragma unroll
+        for (int u = 0; u < 8; ++u) {
+            const int r = r0 + u * vgroups;
+            vr[u] = r < nt && vl < vpieces ? *reinterpret_cast<const uint4*>(vs + size_t(t0 + r) * vrow + vl * P) : make_uint4(0, 0, 0, 0);
+        }
+    };
+    if (OWN) fetch_keys(begin, min(kLaKeys, end - begin), kg, kl), fetch_values(begin, min(kLaKeys, end - begin), vg);  // (written by earlier steps)
+    pdl_wait();
+    if (OWN) {
+        const float *q = a.p + size_t(z) * a.ld, *k = q + a.heads * a.dim, *v = k + a.kv_heads * a.dim + kvh * a.vdim;
+        const int nq = a.heads * a.dim, nk = a.kv_heads * a.dim;
+        float sq = 0.0f, sk = 0.0f;
+        if (a.q_norm != nullptr) {
+#pragma unroll 8
+            for (int i = tid; i < nq; i += kLaThreads) sq += q[i] * q[i];
+        }
+        if (a.k_norm != nullptr) {
+#pragma unroll 4
+            for (int i = tid; i < nk; i += kLaThreads) sk += k[i] * k[i];
+        }
+        sq = warp_sum(sq), sk = warp_sum(sk);
+        if (lane == 0) sums[0][warp] = sq, sums[1][warp] = sk;
+        __syncthreads();
+        sq = sk = 0.0f;
+#pragma unroll
+        for (int w = 0; w < kLaThreads / 32; ++w) sq += sums[0][w], sk += sums[1][w];
+        const float iq = a.q_norm != nullptr ? 1.0f / sqrtf(sq / static_cast<float>(nq) + a.eps) : 1.0f, ik = a.k_norm != nullptr ? 1.0f / sqrtf(sk / static_cast<float>(nk) + a.eps) : 1.0f;
+        const float temp = a.temp_coef != 0.0f ? 1.0f + a.temp_coef * logf(floorf(static_cast<float>(pos + 1) / a.temp_every) + 1.0f) : 1.0f;
+        for (int i = tid; i < nh * a.dim_pad; i += kLaThreads) {
+            const int e = i % a.dim_pad, at = (h0 + i / a.dim_pad) * a.dim + e;
+            qs[i] = e < a.dim ? round_to<T>(q[at] * iq * (a.q_norm != nullptr ? a.q_norm[at] : 1.0f) * temp) : 0.0f;
+        }
+        if (split == 0) {
+            for (int e = tid; e < a.dim_pad; e += kLaThreads) own_k[e] = e < a.dim ? round_to<T>(k[kvh * a.dim + e] * ik * (a.k_norm != nullptr ? a.k_norm[kvh * a.dim + e] : 1.0f)) : 0.0f;
+            if (warp == 7) {
+                float sv = 0.0f;
+                for (int e = lane; e < a.vdim; e += 32) sv += v[e] * v[e];
+                const float iv = a.value_norm ? 1.0f / sqrtf(warp_sum(sv) / static_cast<float>(a.vdim) + a.eps) : 1.0f;
+                for (int e = lane; e < a.vdim_pad; e += 32) own_v[e] = e < a.vdim ? round_to<T>(v[e] * iv) : 0.0f;
+            }
+            __syncthreads();
+            if (warp < nh) {
+                float s = 0.0f;
+                for (int e = lane; e < a.dim_pad; e += 32) s = fmaf(qs[warp * a.dim_pad + e], own_k[e], s);
+                s = warp_sum(s);
+                if (lane == 0) own_weight[warp] = sigmoid_f(s * a.scale + a.bias[h0 + warp]);
+            }
+            if (blockIdx.x % groups == 0) {  // (no block of this launch reads this row of the cache)
+                for (int e = tid; e < a.dim_pad; e += kLaThreads) ks[size_t(pos) * krow + e] = to_storage<T>(own_k[e]);
+                for (int e = tid; e < a.vdim_pad; e += kLaThreads) vs[size_t(pos) * vrow + e] = to_storage<T>(own_v[e]);
+            }
+        }
+    } else {
+        for (int i = tid; i < nh * a.dim_pad; i += kLaThreads) qs[i] = from_storage(static_cast<const T*>(a.q)[(size_t(z) * a.heads + h0) * a.dim_pad + i]);
+    }
+    float acc[H][P];
+#pragma unroll
+    for (int h = 0; h < H; ++h)
 #pragma unroll
         for (int e = 0; e < P; ++e) acc[h][e] = 0.0f;
     for (int t0 = begin; t0 < end; t0 += kLaKeys) {
         const int nt = min(kLaKeys, end - t0);
-        uint4 vr[8];
-        auto fetch_values = [&](int r0) {  // eight rows of this key group
-#pragma unroll
-            for (int u = 0; u < 8; ++u) {
-                const int r = r0 + u * vgroups;
-                vr[u] = r < nt && vl < vpieces ? *reinterpret_cast<const uint4*>(vs + size_t(t0 + r) * vrow + vl * P) : make_uint4(0, 0, 0, 0);
-            }
-        };
-        fetch_values(vg);
+        const bool fetched = OWN && t0 == begin;
+        if (!fetched) fetch_values(t0, nt, vg);
         __syncthreads();  // queries are there; weights of the tile before have been used
-        for (int r0 = kg; r0 < kLaKeys; r0 += 4 * kgroups) {
-            float s[4][kLaHeads];
+        for (int r0 = kg; r0 - kg < nt; r0 += 4 * kgroups) {
+            float s[4][H];
 #pragma unroll
             for (int u = 0; u < 4; ++u)
 #pragma unroll
-                for (int h = 0; h < kLaHeads; ++h) s[u][h] = 0.0f;
+                for (int h = 0; h < H; ++h) s[u][h] = 0.0f;
             for (int p = kl; p < kpieces; p += key_lanes) {
-                uint4 kr[4];
-#pragma unroll
-                for (int u = 0; u < 4; ++u) {
-                    const int r = r0 + u * kgroups;
-                    kr[u] = r < nt ? *reinterpret_cast<const uint4*>(ks + size_t(t0 + r) * krow + p * P) : make_uint4(0, 0, 0, 0);
-                }
+                if (!(fetched && r0 == kg && p == kl)) fetch_keys(t0, nt, r0, p);
                 float kf[4][P];
 #pragma unroll
                 for (int u = 0; u < 4; ++u) Piece<T>::get(kr[u], kf[u]);
 #pragma unroll
-                for (int h = 0; h < kLaHeads; ++h)
+                for (int h = 0; h < H; ++h)
                     if (h < nh) {
+                        float q[P];
 #pragma unroll
-                        for (int e = 0; e < P; ++e) {
-                            const float q = qs[h * a.dim_pad + p * P + e];
+                        for (int e = 0; e < P; e += 4) *reinterpret_cast<float4*>(q + e) = *reinterpret_cast<const float4*>(qs + h * a.dim_pad + p * P + e);
 #pragma unroll
-                            for (int u = 0; u < 4; ++u) s[u][h] = fmaf(q, kf[u][e], s[u][h]);
-                        }
+                        for (int e = 0; e < P; ++e)
+#pragma unroll
+                            for (int u = 0; u < 4; ++u) s[u][h] = fmaf(q[e], kf[u][e], s[u][h]);
                     }
             }
 #pragma unroll
-            for (int h = 0; h < kLaHeads; ++h)
+            for (int h = 0; h < H; ++h)
                 if (h < nh) {
 #pragma unroll
                     for (int u = 0; u < 4; ++u) {
                         float v = s[u][h];
                         for (int o = key_lanes >> 1; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
                         const int r = r0 + u * kgroups;
-                        if (kl == 0 && r < kLaKeys)
-                            ws[h * kLaKeys + r] = r < nt ? sigmoid_f(v * a.scale - a.slope[h0 + h] * static_cast<float>(pos - t0 - r) + a.bias[h0 + h]) : 0.0f;
+                        if (kl == 0 && r < nt) ws[h * kLaKeys + r] = sigmoid_f(v * a.scale - a.slope[h0 + h] * static_cast<float>(pos - t0 - r) + a.bias[h0 + h]);
                     }
                 }
         }
         __syncthreads();
         for (int r0 = vg; r0 < nt; r0 += 8 * vgroups) {
-            if (r0 != vg) fetch_values(r0);
+            if (r0 != vg) fetch_values(t0, nt, r0);
 #pragma unroll
             for (int u = 0; u < 8; ++u) {
                 const int r = r0 + u * vgroups;
@@ -199,7 +247,7 @@ __global__ void __launch_bounds__(kLaThreads) logistic_step_kernel(const __grid_
                 float vf[P];
                 Piece<T>::get(vr[u], vf);
 #pragma unroll
-                for (int h = 0; h < kLaHeads; ++h)
+                for (int h = 0; h < H; ++h)
                     if (h < nh) {
                         const float w = ws[h * kLaKeys + r];
 #pragma unroll
@@ -211,21 +259,21 @@ __global__ void __launch_bounds__(kLaThreads) logistic_step_kernel(const __grid_
     // sums of the key groups: those of a warp by shuffles, then through shared memory
     const int rows = value_lanes < 32 ? kLaThreads / 32 : vgroups, mine = value_lanes < 32 ? warp : vg;
 #pragma unroll
-    for (int h = 0; h < kLaHeads; ++h)
+    for (int h = 0; h < H; ++h)
         if (h < nh) {
 #pragma unroll
             for (int e = 0; e < P; ++e) {
                 float v = acc[h][e];
                 for (int o = 16; o >= value_lanes; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
                 const int c = vl * P + e;
-                if ((value_lanes >= 32 || lane < value_lanes) && c < a.vdim) red[(mine * kLaHeads + h) * a.vdim + c] = v;
+                if ((value_lanes >= 32 || lane < value_lanes) && c < a.vdim) red[(mine * H + h) * a.vdim + c] = v;
             }
         }
     __syncthreads();
     for (int i = tid; i < nh * a.vdim; i += kLaThreads) {
         const int h = i / a.vdim, c = i % a.vdim;
-        float s = 0.0f;
-        for (int k = 0; k < rows; ++k) s += red[(k * kLaHeads + h) * a.vdim + c];
+        float s = OWN && split == 0 ? own_weight[h] * own_v[c] : 0.0f;
+        for (int k = 0; k < rows; ++k) s += red[(k * H + h) * a.vdim + c];
         if (a.splits == 1) a.y[(size_t(z) * a.heads + h0 + h) * a.vdim + c] = s;
         else a.part[((size_t(z) * a.heads + h0 + h) * a.splits + split) * a.vdim + c] = s;
     }
@@ -238,14 +286,31 @@ __global__ void __launch_bounds__(kLaThreads) logistic_step_kernel(const __grid_
     if (!last_block) return;
     if (tid == 0) *counter = 0;
     __threadfence();
-    for (int i = tid; i < nh * a.vdim; i += kLaThreads) {
-        const int h = i / a.vdim, c = i % a.vdim;
-        const float* part = a.part + ((size_t(z) * a.heads + h0 + h) * a.splits) * a.vdim + c;
-        float s = 0.0f;
-#pragma unroll 8
-        for (int k = 0; k < a.splits; ++k) s += __ldcg(part + size_t(k) * a.vdim);
-        a.y[(size_t(z) * a.heads + h0 + h) * a.vdim + c] = s;
+    // the shares that had keys, their sums by parts of the block: as many threads per result as there are for it
+    const int live = per > 0 ? max(1, (total + per - 1) / per) : 1, results = nh * a.vdim, teams = max(1, min(kLaThreads / max(results, 1), 8));
+    if (teams == 1) {
+        for (int i = tid; i < results; i += kLaThreads) {
+            const int h = i / a.vdim, c = i % a.vdim;
+            const float* part = a.part + ((size_t(z) * a.heads + h0 + h) * a.splits) * a.vdim + c;
+            float s = 0.0f;
+#pragma unroll 16
+            for (int k = 0; k < live; ++k) s += __ldcg(part + size_t(k) * a.vdim);
+            a.y[(size_t(z) * a.heads + h0 + h) * a.vdim + c] = s;
+        }
+        return;
     }
+    const int team = tid / results, i = tid % results, h = i / a.vdim, c = i % a.vdim;
+    float s = 0.0f;
+    if (team < teams) {
+        const float* part = a.part + ((size_t(z) * a.heads + h0 + h) * a.splits) * a.vdim + c;
+#pragma unroll 16
+        for (int k = team; k < live; k += teams) s += __ldcg(part + size_t(k) * a.vdim);
+        red[tid] = s;
+    }
+    __syncthreads();
+    if (team != 0) return;
+    for (int t = 1; t < teams; ++t) s += red[t * results + i];
+    a.y[(size_t(z) * a.heads + h0 + h) * a.vdim + c] = s;
 }
 
 // ---- many query positions on the tensor cores of a warp --------------------------------------------------------------------------------------

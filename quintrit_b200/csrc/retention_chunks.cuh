@@ -4,8 +4,8 @@
 //   y_t = a^(t + 1) q_t S + sum over s <= t of a^(t - s) (q_t . k_s) v_s        t, s: places in the chunk
 //
 // so the chunks need not follow one another: U of every chunk at once, then S at every chunk's start (one multiply-add per element and chunk), then
-// every chunk's outputs at once. 64 tokens a chunk, products on the warp tensor cores; queries, keys, states and decayed weights go in as two bf16
-// terms, values as one. The last kernel also divides each head's output by its root mean square and multiplies it by silu(g).
+// every chunk's outputs at once. 64 tokens a chunk, products on the warp tensor cores; queries, keys, states and decayed weights or values go in as
+// two bf16 terms. The last kernel also divides each head's output by its root mean square and multiplies it by silu(g).
 #pragma once
 #include "gated_scan.cuh"
 #include "mma_bf16.cuh"
@@ -13,7 +13,9 @@
 namespace qtb {
 
 constexpr int kRetT = 64;      // tokens of a chunk
-constexpr int kRetV = 64;      // value columns per block of the first kernel, and per turn of the last
+constexpr int kRetV = 64;      // value columns per block of the state kernel
+constexpr int kRetPart = 32;   // value columns per turn of the output kernel
+constexpr int kRetPrep = 16;   // tokens per block of the preparing kernel
 
 // Compiled sizes: rows of the state and value columns, 0 if a head is too large.
 inline int retention_rows(int dim) { return dim <= 32 ? 32 : dim <= 64 ? 64 : dim <= 128 ? 128 : dim <= 256 ? 256 : 0; }
@@ -21,15 +23,18 @@ inline int retention_cols(int vdim) { return vdim <= 64 ? 64 : vdim <= 128 ? 128
 inline int retention_chunks(int tokens) { return (tokens + kRetT - 1) / kRetT; }
 
 struct RetentionWork {
+    bf16 *q_hi, *q_lo, *k_hi, *k_lo;  // rotated (keys also scaled), [head][token][rows], zero beyond dim and beyond the last token
+    bf16* v;               // [head][token][v_pad]
     float* u;              // [head][chunk][v_pad][rows]
     bf16 *s_hi, *s_lo;     // the state before each chunk, same order
-    int rows, v_pad;
+    int rows, v_pad, tokens;  // tokens: rounded up to whole chunks
 };
 inline size_t retention_work(char* base, int heads, int dim, int vdim, int tokens, RetentionWork* w) {
-    w->rows = retention_rows(dim), w->v_pad = retention_cols(vdim);
-    const size_t n = size_t(heads) * retention_chunks(tokens) * w->v_pad * w->rows;
-    w->u = reinterpret_cast<float*>(base), w->s_hi = reinterpret_cast<bf16*>(base + n * 4), w->s_lo = w->s_hi + n;
-    return n * 8;
+    w->rows = retention_rows(dim), w->v_pad = retention_cols(vdim), w->tokens = retention_chunks(tokens) * kRetT;
+    const size_t n = size_t(heads) * retention_chunks(tokens) * w->v_pad * w->rows, qk = size_t(heads) * w->tokens * w->rows, v = size_t(heads) * w->tokens * w->v_pad;
+    w->u = reinterpret_cast<float*>(base), w->s_hi = reinterpret_cast<bf16*>(w->u + n), w->s_lo = w->s_hi + n;
+    w->q_hi = w->s_lo + n, w->q_lo = w->q_hi + qk, w->k_hi = w->q_lo + qk, w->k_lo = w->k_hi + qk, w->v = w->k_lo + qk;
+    return n * 8 + qk * 8 + v * 2;
 }
 
 struct RetentionArgs {
@@ -44,12 +49,75 @@ struct RetentionArgs {
 __device__ __forceinline__ void decay_powers(float decay, float* pw) {
     for (int i = threadIdx.x; i <= kRetT; i += blockDim.x) pw[i] = i == 0 ? 1.0f : decay > 0.0f ? exp2f(static_cast<float>(i) * log2f(decay)) : 0.0f;
 }
-__device__ __forceinline__ void put_split(bf16* hi, bf16* lo, int at, float v) {
-    const bf16 h = __float2bfloat16_rn(v);
-    hi[at] = h, lo[at] = __float2bfloat16_rn(v - __bfloat162float(h));
+// Queries, keys and values of every token as the products take them. PAIRS: two neighbouring elements at a time (even sizes and columns).
+// grid: (heads, padded tokens / 16), 128 threads
+template <bool PAIRS>
+__global__ void __launch_bounds__(128) retention_prepare_kernel(const __grid_constant__ RetentionArgs r) {
+    const ScanArgs& a = r.scan;
+    const RetentionWork& w = r.work;
+    constexpr int S = PAIRS ? 2 : 1;
+    const int head = blockIdx.x, t0 = blockIdx.y * kRetPrep, tid = threadIdx.x, n = a.n, half = a.rot_dims / 2;
+    const uint32_t pos0 = seq_position(a.seq, a.pos, 0);
+    const float scale = 1.0f / sqrtf(static_cast<float>(n));
+    auto put = [&](bf16* hi, bf16* lo, size_t at, const float (&v)[S]) {
+        if constexpr (PAIRS) {
+            uint32_t h, l;
+            split_bf16(v[0], v[1], &h, &l);
+            *reinterpret_cast<uint32_t*>(hi + at) = h, *reinterpret_cast<uint32_t*>(lo + at) = l;
+        } else {
+            const bf16 h = __float2bfloat16_rn(v[0]);
+            hi[at] = h, lo[at] = __float2bfloat16_rn(v[0] - __bfloat162float(h));
+        }
+    };
+    auto get = [&](const float* p, bool there, float (&v)[S]) {
+        if constexpr (PAIRS) {
+            const float2 f = there ? *reinterpret_cast<const float2*>(p) : make_float2(0.0f, 0.0f);
+            v[0] = f.x, v[1] = f.y;
+        } else {
+            v[0] = there ? *p : 0.0f;
+        }
+    };
+    const int items = (w.rows - half) / S;  // an item is a pair to rotate (two neighbouring ones), or elements that stay as they are
+#pragma unroll 2
+    for (int i = tid; i < kRetPrep * items; i += 128) {
+        const int t = t0 + i / items, j = i % items * S;
+        const bool there = t < a.tokens;
+        const float* p = a.p + size_t(min(t, a.tokens - 1)) * a.ld + head * n;
+        const float* pk = p + a.heads * n;
+        const size_t at = (size_t(head) * w.tokens + t) * w.rows;
+        float q[S], k[S];
+        if (j < half) {
+            float q2[S], k2[S];
+            get(p + j, there, q), get(p + j + half, there, q2), get(pk + j, there, k), get(pk + j + half, there, k2);
+#pragma unroll
+            for (int e = 0; e < S; ++e) {
+                const float2 cs = rotation(a.turns[j + e], pos0 + t);
+                const float2 rq = rotate_pair(q[e], q2[e], cs), rk = rotate_pair(k[e], k2[e], cs);
+                q[e] = rq.x, q2[e] = rq.y, k[e] = rk.x * scale, k2[e] = rk.y * scale;
+            }
+            put(w.q_hi, w.q_lo, at + j, q), put(w.q_hi, w.q_lo, at + j + half, q2);
+            put(w.k_hi, w.k_lo, at + j, k), put(w.k_hi, w.k_lo, at + j + half, k2);
+        } else {
+            const bool in = there && j + half < n;
+            get(p + j + half, in, q), get(pk + j + half, in, k);
+#pragma unroll
+            for (int e = 0; e < S; ++e) k[e] *= scale;
+            put(w.q_hi, w.q_lo, at + j + half, q), put(w.k_hi, w.k_lo, at + j + half, k);
+        }
+    }
+    const int cols = w.v_pad / S;
+#pragma unroll 4
+    for (int i = tid; i < kRetPrep * cols; i += 128) {
+        const int t = t0 + i / cols, c = i % cols * S;
+        float v[S];
+        get(a.p + size_t(min(t, a.tokens - 1)) * a.ld + 2 * a.heads * n + head * a.vdim + c, t < a.tokens && c < a.vdim, v);
+        bf16* out = w.v + (size_t(head) * w.tokens + t) * w.v_pad + c;
+        if constexpr (PAIRS) *reinterpret_cast<uint32_t*>(out) = pack_bf16(v[0], v[1]);
+        else *out = __float2bfloat16_rn(v[0]);
+    }
 }
 
-// U of every chunk. grid: (heads, chunks, ceil(vdim / 64)), 128 threads; a warp owns 16 value columns
+// U of every chunk. grid: (heads, chunks, v_pad / 64), 128 threads; a warp owns 16 value columns
 template <int N> __host__ __device__ constexpr size_t retention_state_smem() { return size_t(2 * kRetT) * (N + 8) * 2 + size_t(kRetT) * (kRetV + 8) * 2; }
 template <int N>
 __global__ void __launch_bounds__(128) retention_state_kernel(const __grid_constant__ RetentionArgs r) {
@@ -59,26 +127,20 @@ __global__ void __launch_bounds__(128) retention_state_kernel(const __grid_const
     constexpr int kPitch = N + 8, kVPitch = kRetV + 8;
     bf16 *kh = reinterpret_cast<bf16*>(rt_sm), *kl = kh + kRetT * kPitch, *vs = kl + kRetT * kPitch;
     const int head = blockIdx.x, chunk = blockIdx.y, chunks = gridDim.y, v0 = blockIdx.z * kRetV, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, c = lane & 3;
-    const int t0 = chunk * kRetT, len = min(kRetT, a.tokens - t0), n = a.n, half = a.rot_dims / 2, items = N - half;
-    const uint32_t pos0 = seq_position(a.seq, a.pos, 0) + t0;
+    const int t0 = chunk * kRetT, len = min(kRetT, a.tokens - t0);
+    const size_t row0 = size_t(head) * r.work.tokens + t0;
+    for (int i = tid; i < kRetT * (N / 8); i += 128) {
+        const int t = i / (N / 8), p = i % (N / 8);
+        cp_async16(kh + t * kPitch + p * 8, r.work.k_hi + (row0 + t) * N + p * 8, true);
+        cp_async16(kl + t * kPitch + p * 8, r.work.k_lo + (row0 + t) * N + p * 8, true);
+    }
+    for (int i = tid; i < kRetT * (kRetV / 8); i += 128) {
+        const int t = i / (kRetV / 8), p = i % (kRetV / 8);
+        cp_async16(vs + t * kVPitch + p * 8, r.work.v + (row0 + t) * r.work.v_pad + v0 + p * 8, true);
+    }
+    cp_async_commit_group();
     decay_powers(a.decay[head], pw);
-    __syncthreads();
-    const float scale = 1.0f / sqrtf(static_cast<float>(n));
-    for (int i = tid; i < kRetT * items; i += 128) {
-        const int t = i / items, j = i % items;
-        const float* p = a.p + size_t(t0 + min(t, len - 1)) * a.ld + a.heads * n + head * n;
-        const float f = t < len ? scale * pw[len - 1 - t] : 0.0f;
-        if (j < half) {
-            const float2 k = rotate_pair(p[j], p[j + half], rotation(a.turns[j], pos0 + t));
-            put_split(kh, kl, t * kPitch + j, k.x * f), put_split(kh, kl, t * kPitch + j + half, k.y * f);
-        } else {
-            put_split(kh, kl, t * kPitch + j + half, j + half < n ? p[j + half] * f : 0.0f);
-        }
-    }
-    for (int i = tid; i < kRetT * kRetV; i += 128) {
-        const int t = i / kRetV, v = i % kRetV;
-        vs[t * kVPitch + v] = __float2bfloat16_rn(t < len && v0 + v < a.vdim ? a.p[size_t(t0 + t) * a.ld + 2 * a.heads * n + head * a.vdim + v0 + v] : 0.0f);
-    }
+    cp_async_wait_group<0>();
     __syncthreads();
     float u[N / 8][4];
 #pragma unroll
@@ -87,16 +149,22 @@ __global__ void __launch_bounds__(128) retention_state_kernel(const __grid_const
         for (int e = 0; e < 4; ++e) u[j][e] = 0.0f;
 #pragma unroll
     for (int s = 0; s < kRetT / 16; ++s) {
-        uint32_t xv[4];
+        uint32_t xv[4], xh[4], xl[4];
         load_frag_b(xv, vs + s * 16 * kVPitch + warp * 16, kVPitch);
-        const uint32_t xt[4] = {xv[0], xv[2], xv[1], xv[3]};  // transposed: an A operand, value columns as rows
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {  // transposed an A operand, value columns as rows; its tokens: s * 16 + 2 c, + 1 (e < 2), + 8, + 9
+            const uint32_t x = xv[((e & 1) << 1) | (e >> 1)];
+            const int t = s * 16 + 2 * c + (e >> 1) * 8;  // (tokens beyond len: keys and values are zero)
+            split_bf16(__uint_as_float(x << 16) * pw[max(len - 1 - t, 0)], __uint_as_float(x & 0xffff0000u) * pw[max(len - 2 - t, 0)], &xh[e], &xl[e]);
+        }
 #pragma unroll
         for (int j = 0; j < N / 8; j += 2) {
             uint32_t h[4], l[4];
             load_frag_b(h, kh + s * 16 * kPitch + j * 8, kPitch);
             load_frag_b(l, kl + s * 16 * kPitch + j * 8, kPitch);
-            mma_16816(u[j], xt, h[0], h[1]), mma_16816(u[j + 1], xt, h[2], h[3]);
-            mma_16816(u[j], xt, l[0], l[1]), mma_16816(u[j + 1], xt, l[2], l[3]);
+            mma_16816(u[j], xh, h[0], h[1]), mma_16816(u[j + 1], xh, h[2], h[3]);
+            mma_16816(u[j], xl, h[0], h[1]), mma_16816(u[j + 1], xl, h[2], h[3]);
+            mma_16816(u[j], xh, l[0], l[1]), mma_16816(u[j + 1], xh, l[2], l[3]);
         }
     }
     float* out = r.work.u + ((size_t(head) * chunks + chunk) * r.work.v_pad + v0 + warp * 16) * N;
@@ -143,36 +211,33 @@ __global__ void __launch_bounds__(128) retention_carry_kernel(const __grid_const
         if (v < a.vdim && d + e < a.n) state[d + e] = s[e];
 }
 
-// Outputs of a chunk. grid: (heads, chunks), 128 threads; a warp owns 16 tokens and all value columns
-template <int N> __host__ __device__ constexpr size_t retention_out_smem() { return size_t(4 * kRetT) * (N + 8) * 2 + size_t(kRetT) * (kRetV + 8) * 2; }
+// Outputs of a chunk. grid: (heads, chunks), 128 threads; a warp owns 16 tokens and all value columns, 32 of them at a time: the next 32 columns of
+// the state and the values are on their way while the products of these are made.
+template <int N> __host__ __device__ constexpr size_t retention_out_stage() { return size_t(2 * kRetPart) * (N + 8) * 2 + size_t(kRetT) * (kRetPart + 8) * 2; }
+template <int N> __host__ __device__ constexpr size_t retention_out_smem() {
+    const size_t keys = size_t(2 * kRetT) * (N + 8) * 2;  // (in the stages' place until the scores are made)
+    return keys + (2 * retention_out_stage<N>() > keys ? 2 * retention_out_stage<N>() : keys);
+}
 template <int N, int V>
 __global__ void __launch_bounds__(128) retention_out_kernel(const __grid_constant__ RetentionArgs r) {
     extern __shared__ __align__(16) unsigned char rt_sm[];
     __shared__ float pw[kRetT + 1];
     const ScanArgs& a = r.scan;
-    constexpr int kPitch = N + 8, kVPitch = kRetV + 8;
-    bf16 *qh = reinterpret_cast<bf16*>(rt_sm), *ql = qh + kRetT * kPitch, *kh = ql + kRetT * kPitch, *kl = kh + kRetT * kPitch, *vs = kl + kRetT * kPitch;
+    constexpr int kPitch = N + 8, kVPitch = kRetPart + 8, kParts = V / kRetPart, kCols = kRetPart / 8;
+    bf16 *qh = reinterpret_cast<bf16*>(rt_sm), *ql = qh + kRetT * kPitch, *kh = ql + kRetT * kPitch, *kl = kh + kRetT * kPitch;
+    unsigned char* stages = reinterpret_cast<unsigned char*>(kh);
     const int head = blockIdx.x, chunk = blockIdx.y, chunks = gridDim.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, c = lane & 3;
-    const int t0 = chunk * kRetT, len = min(kRetT, a.tokens - t0), n = a.n, half = a.rot_dims / 2, items = N - half;
-    const uint32_t pos0 = seq_position(a.seq, a.pos, 0) + t0;
-    decay_powers(a.decay[head], pw);
-    const float scale = 1.0f / sqrtf(static_cast<float>(n));
-    for (int i = tid; i < kRetT * items; i += 128) {
-        const int t = i / items, j = i % items;
-        const float* p = a.p + size_t(t0 + min(t, len - 1)) * a.ld + head * n;
-        const float* pk = p + a.heads * n;
-        const bool there = t < len;
-        if (j < half) {
-            const float2 cs = rotation(a.turns[j], pos0 + t);
-            const float2 q = rotate_pair(p[j], p[j + half], cs), k = rotate_pair(pk[j], pk[j + half], cs);
-            put_split(qh, ql, t * kPitch + j, there ? q.x : 0.0f), put_split(qh, ql, t * kPitch + j + half, there ? q.y : 0.0f);
-            put_split(kh, kl, t * kPitch + j, there ? k.x * scale : 0.0f), put_split(kh, kl, t * kPitch + j + half, there ? k.y * scale : 0.0f);
-        } else {
-            const bool in = there && j + half < n;
-            put_split(qh, ql, t * kPitch + j + half, in ? p[j + half] : 0.0f);
-            put_split(kh, kl, t * kPitch + j + half, in ? pk[j + half] * scale : 0.0f);
-        }
+    const int t0 = chunk * kRetT, len = min(kRetT, a.tokens - t0), n = a.n;
+    const size_t row0 = size_t(head) * r.work.tokens + t0;
+    for (int i = tid; i < kRetT * (N / 8); i += 128) {
+        const int t = i / (N / 8), p = i % (N / 8), at = t * kPitch + p * 8;
+        const size_t from = (row0 + t) * N + p * 8;
+        cp_async16(qh + at, r.work.q_hi + from, true), cp_async16(ql + at, r.work.q_lo + from, true);
+        cp_async16(kh + at, r.work.k_hi + from, true), cp_async16(kl + at, r.work.k_lo + from, true);
     }
+    cp_async_commit_group();
+    decay_powers(a.decay[head], pw);
+    cp_async_wait_group<0>();
     __syncthreads();
     // decayed scores of the chunk's tokens, as A operands of the product with the values
     uint32_t ph[kRetT / 16][4], pl[kRetT / 16][4];
@@ -188,6 +253,7 @@ __global__ void __launch_bounds__(128) retention_out_kernel(const __grid_constan
             load_frag_a(h, qh + warp * 16 * kPitch + k * 16, kPitch), load_frag_a(l, ql + warp * 16 * kPitch + k * 16, kPitch);
 #pragma unroll
             for (int j = 0; j < kRetT / 8; j += 2) {
+                if (j / 2 > warp) continue;  // (all of these keys come later)
                 uint32_t bh[4], bl[4];
                 load_frag_bt(bh, kh + j * 8 * kPitch + k * 16, kPitch), load_frag_bt(bl, kl + j * 8 * kPitch + k * 16, kPitch);
                 mma_16816(s[j], h, bh[0], bh[1]), mma_16816(s[j + 1], h, bh[2], bh[3]);
@@ -209,26 +275,33 @@ __global__ void __launch_bounds__(128) retention_out_kernel(const __grid_constan
         }
     }
     const float from_state[2] = {pw[warp * 16 + g + 1], pw[warp * 16 + g + 9]};
-    bf16 *sh = kh, *sl = kl;  // the keys' place, 64 rows of the state at a time
-    float o[V / 8][4], ss[2] = {0.0f, 0.0f};
-#pragma unroll
-    for (int part = 0; part < V / kRetV; ++part) {
-        const int v0 = part * kRetV;
-        __syncthreads();
-        const size_t at = ((size_t(head) * chunks + chunk) * r.work.v_pad + v0) * N;
-        for (int i = tid; i < kRetV * (N / 8); i += 128) {
+    auto fetch = [&](int part) {
+        bf16 *sh = reinterpret_cast<bf16*>(stages + (part & 1) * retention_out_stage<N>()), *sl = sh + kRetPart * kPitch, *vs = sl + kRetPart * kPitch;
+        const size_t at = ((size_t(head) * chunks + chunk) * r.work.v_pad + part * kRetPart) * N;
+        for (int i = tid; i < kRetPart * (N / 8); i += 128) {
             const int v = i / (N / 8), p = i % (N / 8);
             cp_async16(sh + v * kPitch + p * 8, r.work.s_hi + at + size_t(v) * N + p * 8, true);
             cp_async16(sl + v * kPitch + p * 8, r.work.s_lo + at + size_t(v) * N + p * 8, true);
         }
-        cp_async_commit_group();
-        for (int i = tid; i < kRetT * kRetV; i += 128) {
-            const int t = i / kRetV, v = i % kRetV;
-            vs[t * kVPitch + v] = __float2bfloat16_rn(t < len && v0 + v < a.vdim ? a.p[size_t(t0 + t) * a.ld + 2 * a.heads * n + head * a.vdim + v0 + v] : 0.0f);
+        for (int i = tid; i < kRetT * (kRetPart / 8); i += 128) {
+            const int t = i / (kRetPart / 8), p = i % (kRetPart / 8);
+            cp_async16(vs + t * kVPitch + p * 8, r.work.v + (row0 + t) * r.work.v_pad + part * kRetPart + p * 8, true);
         }
-        cp_async_wait_group<0>();
+        cp_async_commit_group();
+    };
+    __syncthreads();  // every warp is done with the keys
+    fetch(0);
+    float o[V / 8][4], ss[2] = {0.0f, 0.0f};
+#pragma unroll
+    for (int part = 0; part < kParts; ++part) {
+        if (part + 1 < kParts) {
+            fetch(part + 1);
+            cp_async_wait_group<1>();
+        } else {
+            cp_async_wait_group<0>();
+        }
         __syncthreads();
-        constexpr int kCols = kRetV / 8;
+        const bf16 *sh = reinterpret_cast<const bf16*>(stages + (part & 1) * retention_out_stage<N>()), *sl = sh + kRetPart * kPitch, *vs = sl + kRetPart * kPitch;
         float (*po)[4] = o + part * kCols;
 #pragma unroll
         for (int j = 0; j < kCols; ++j)
@@ -252,7 +325,8 @@ __global__ void __launch_bounds__(128) retention_out_kernel(const __grid_constan
 #pragma unroll
             for (int e = 0; e < 4; ++e) po[j][e] *= from_state[e >> 1];
 #pragma unroll
-        for (int k = 0; k < kRetT / 16; ++k)
+        for (int k = 0; k < kRetT / 16; ++k) {
+            if (k > warp) continue;  // (their weights are zero)
 #pragma unroll
             for (int j = 0; j < kCols; j += 2) {
                 uint32_t b[4];
@@ -260,10 +334,12 @@ __global__ void __launch_bounds__(128) retention_out_kernel(const __grid_constan
                 mma_16816(po[j], ph[k], b[0], b[1]), mma_16816(po[j + 1], ph[k], b[2], b[3]);
                 mma_16816(po[j], pl[k], b[0], b[1]), mma_16816(po[j + 1], pl[k], b[2], b[3]);
             }
+        }
 #pragma unroll
         for (int j = 0; j < kCols; ++j)
 #pragma unroll
             for (int e = 0; e < 4; ++e) ss[e >> 1] = fmaf(po[j][e], po[j][e], ss[e >> 1]);  // (columns beyond vdim are zero)
+        __syncthreads();  // the stage may be filled again
     }
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
