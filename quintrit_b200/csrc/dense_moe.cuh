@@ -16,61 +16,53 @@ struct RouterArgs {
     float scale;
 };
 
-// One warp: the chosen experts of a token, best first, and their weights, from its logits. score: `experts` floats of shared memory (this warp's).
-// Equal scores: the lower index first.
-__device__ __forceinline__ void choose_experts(const RouterArgs& r, const float* logits, float* score, int* chosen, float* weight) {
-    const int lane = threadIdx.x & 31;
+// One warp: the chosen experts of a token, best first, and their weights, from its logits; equal scores by the lower index. key: 2 * `experts`
+// words of shared memory (this warp's). A key is the score's bits plus one (scores are not negative, so their order is that of the bits); 0 stands for
+// an expert that cannot be chosen (any more).
+__device__ __forceinline__ void choose_experts(const RouterArgs& r, const float* logits, uint32_t* key, int* chosen, float* weight) {
+    const int lane = threadIdx.x & 31, size = r.experts / r.groups;
+    uint32_t* group = key + r.experts;
     float mx = -INFINITY, sum = 0.0f;
     for (int i = lane; i < r.experts; i += 32) mx = fmaxf(mx, logits[i]);
     for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
     for (int i = lane; i < r.experts; i += 32) {
         const float e = expf(logits[i] - mx);
-        score[i] = e, sum += e;
+        key[i] = __float_as_uint(e) + 1u, sum += e;
     }
     sum = warp_sum(sum);
     __syncwarp();
-    const int size = r.experts / r.groups;
-    auto best_of = [&](float v, int i) {  // the warp's largest value, the lower index of equal ones
-        for (int o = 16; o > 0; o >>= 1) {
-            const float v2 = __shfl_xor_sync(0xffffffffu, v, o);
-            const int i2 = __shfl_xor_sync(0xffffffffu, i, o);
-            if (v2 > v || (v2 == v && i2 < i)) v = v2, i = i2;
+    if (r.keep < r.groups) {  // a group counts by its largest score, and is dropped when `keep` others are better
+        for (int g = lane; g < r.groups; g += 32) {
+            uint32_t m = 0;
+            for (int i = 0; i < size; ++i) m = max(m, key[g * size + i]);
+            group[g] = m;
         }
-        return make_float2(v, __int_as_float(i));
-    };
-    if (r.keep < r.groups) {
-        // a group is dropped when `keep` others are better; its scores then no longer count (exponentials are not negative)
-        for (int g0 = 0; g0 < r.groups; g0 += 32) {
-            const int g = g0 + lane;
-            float mine = -1.0f;
+        __syncwarp();
+        for (int g = lane; g < r.groups; g += 32) {
+            const uint32_t mine = group[g];
             int better = 0;
-            if (g < r.groups)
-                for (int i = 0; i < size; ++i) mine = fmaxf(mine, score[g * size + i]);
-            for (int o = 0; o < r.groups; ++o) {
-                float other = -1.0f;
-                if (r.groups <= 32) {
-                    other = __shfl_sync(0xffffffffu, mine, o);
-                } else {
-                    for (int i = 0; i < size; ++i) other = fmaxf(other, fabsf(score[o * size + i]));
-                }
-                better += (other > mine || (other == mine && o < g)) ? 1 : 0;
-            }
-            __syncwarp();
-            // (a dropped score changes its sign, so that a group looked at later still sees its size; -0.0 stands for a dropped zero)
-            if (g < r.groups && better >= r.keep)
-                for (int i = 0; i < size; ++i) score[g * size + i] = -score[g * size + i] - 1e-30f;
-            __syncwarp();
+            for (int o = 0; o < r.groups; ++o) better += group[o] > mine || (group[o] == mine && o < g) ? 1 : 0;
+            if (better >= r.keep)
+                for (int i = 0; i < size; ++i) key[g * size + i] = 0u;
         }
+        __syncwarp();
     }
-    for (int k = 0; k < r.top; ++k) {
-        float v = -INFINITY;
-        int at = r.experts;
+    uint32_t best = 0;  // this lane's best expert left
+    int at = r.experts;
+    auto look = [&]() {
+        best = 0, at = r.experts;
         for (int i = lane; i < r.experts; i += 32)
-            if (score[i] > v) v = score[i], at = i;
-        const float2 b = best_of(v, at);
-        at = min(__float_as_int(b.y), r.experts - 1);  // (stays in range whatever the logits are)
-        if (lane == 0) chosen[k] = at, weight[k] = b.x / sum * r.scale;
-        if (lane == (at & 31)) score[at] = -INFINITY;
+            if (key[i] > best) best = key[i], at = i;
+    };
+    look();
+    for (int k = 0; k < r.top; ++k) {
+        const uint32_t top = __reduce_max_sync(0xffffffffu, best);
+        const int e = min(static_cast<int>(__reduce_min_sync(0xffffffffu, best == top ? static_cast<uint32_t>(at) : 0xffffffffu)), r.experts - 1);  // (in range whatever the logits are)
+        if (lane == 0) chosen[k] = e, weight[k] = __uint_as_float(top - 1u) / sum * r.scale;
+        if (lane == (e & 31)) {
+            key[e] = 0u;
+            look();
+        }
         __syncwarp();
     }
 }
@@ -90,14 +82,14 @@ struct MoeUpStepArgs {
 
 template <typename T>
 __global__ void __launch_bounds__(kProjectThreads, 4) moe_up_step_kernel(const __grid_constant__ MoeUpStepArgs a) {
-    extern __shared__ float act_smem[];  // the input, then the router's scores
+    extern __shared__ float act_smem[];  // the input, then the router's keys
     __shared__ int chosen[32];
     __shared__ float weight[32];
     const int tid = threadIdx.x, warps = gridDim.x * (kProjectThreads / 32), units = a.router.top * a.ff;
     pdl_trigger();
     pdl_wait();
     if (tid < 32) {
-        choose_experts(a.router, a.logits, act_smem + a.pitch, chosen, weight);
+        choose_experts(a.router, a.logits, reinterpret_cast<uint32_t*>(act_smem + a.pitch), chosen, weight);
         if (blockIdx.x == 0 && tid < a.router.top) a.chosen[tid] = chosen[tid], a.weight[tid] = weight[tid];
     }
     else {
@@ -138,7 +130,7 @@ constexpr int kMoeDownRows = kProjectThreads / 32;  // at most: a warp ends a ro
 
 // A block takes a few rows of the result; its warps share the products of these rows with the activations of every chosen expert.
 template <typename T>
-__global__ void __launch_bounds__(kProjectThreads) moe_down_step_kernel(const __grid_constant__ MoeDownStepArgs a) {
+__global__ void __launch_bounds__(kProjectThreads, 4) moe_down_step_kernel(const __grid_constant__ MoeDownStepArgs a) {
     extern __shared__ float act_smem[];  // activations of the experts, of the shared expert
     __shared__ float part[kMoeDownRows * 33];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, row0 = blockIdx.x * a.rows, rows = min(a.rows, a.width - row0), per = a.top + 1, units = rows * per;
@@ -160,7 +152,7 @@ __global__ void __launch_bounds__(kProjectThreads) moe_down_step_kernel(const __
         for (int j = lane; j < a.depth.n - 1; j += 32) past = fmaf(a.depth.w[j], a.depth.x[j * a.depth.stride + end_row], past);
     }
     constexpr int kPer = 16 / sizeof(T), kWarps = kProjectThreads / 32;
-    // a warp takes two (row, expert) products at a time, the next two on their way
+    // a warp takes two (row, expert) products at a time
     struct Two { uint4 v[2][4]; };
     auto load = [&](int unit, int p0, Two& b) {
 #pragma unroll
@@ -172,7 +164,7 @@ __global__ void __launch_bounds__(kProjectThreads) moe_down_step_kernel(const __
             for (int i = 0; i < 4; ++i) b.v[k][i] = p0 + 32 * i < pieces ? load_stream(row + size_t(p0 + 32 * i) * kPer) : make_uint4(0, 0, 0, 0);
         }
     };
-    Two now, next;
+    Two now;
     load(warp, lane, now);
     for (int i = tid; i < a.top * (a.pitch / kPer); i += kProjectThreads) {
         const int k = i / (a.pitch / kPer), p = i % (a.pitch / kPer);
@@ -184,8 +176,7 @@ __global__ void __launch_bounds__(kProjectThreads) moe_down_step_kernel(const __
     for (int unit = warp; unit < units; unit += 2 * kWarps) {
         float sum[2] = {0.0f, 0.0f};
         for (int p0 = lane; p0 - lane < longest; p0 += 128) {
-            if (p0 != lane) load(unit, p0, now);
-            if (p0 == lane && unit + 2 * kWarps < units) load(unit + 2 * kWarps, lane, next);
+            if (p0 != lane || unit != warp) load(unit, p0, now);
 #pragma unroll
             for (int k = 0; k < 2; ++k) {
                 const int u = unit + k * kWarps;
@@ -203,7 +194,6 @@ __global__ void __launch_bounds__(kProjectThreads) moe_down_step_kernel(const __
             sum[k] = warp_sum(sum[k]);
             if (lane == 0 && u < units) part[u / per * 33 + u % per] = sum[k];
         }
-        now = next;
     }
     __syncthreads();
     if (warp < rows) {
@@ -233,14 +223,14 @@ struct MoeRouteArgs {
     int up_rows, down_rows, tile;  // weight rows of an expert in the two stacks; activation rows of a run
 };
 
-// A warp per token. dynamic shared memory: 4 * experts floats
+// A warp per token. dynamic shared memory: 8 * experts words
 __global__ void __launch_bounds__(128) moe_route_kernel(const __grid_constant__ MoeRouteArgs a) {
-    extern __shared__ float route_sm[];
+    extern __shared__ uint32_t route_sm[];
     __shared__ int chosen[4][32];
     __shared__ float weight[4][32];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, t = blockIdx.x * 4 + warp, top = a.router.top;
     if (t >= a.tokens) return;
-    choose_experts(a.router, a.logits + size_t(t) * a.router.experts, route_sm + warp * a.router.experts, chosen[warp], weight[warp]);
+    choose_experts(a.router, a.logits + size_t(t) * a.router.experts, route_sm + warp * 2 * a.router.experts, chosen[warp], weight[warp]);
     __syncwarp();
     if (lane < top) {
         const int e = chosen[warp][lane];

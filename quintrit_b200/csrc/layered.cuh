@@ -23,6 +23,7 @@
 #include "gated_scan.cuh"
 #include "layered_spec.hpp"
 #include "logistic_attention.cuh"
+#include "logistic_attention_tc.cuh"
 #include "pooled_attention.cuh"
 #include "pooled_attention_mma.cuh"
 #include "retention_chunks.cuh"
@@ -102,6 +103,7 @@ struct LayeredStore {
         float *state = nullptr, *conv = nullptr;
         size_t state_stride = 0, conv_stride = 0;  // floats per slot
         PooledCache cache{};
+        CUtensorMap kmap{}, vmap{};                // logistic attention: the cached keys and values, [slot][position][kv heads x padded dim]
     };
     std::vector<Mixer> mixers;
 };
@@ -114,7 +116,7 @@ struct LayeredDecoder {
     float *x = nullptr, *p1 = nullptr, *g1 = nullptr, *g2 = nullptr, *y[2] = {nullptr, nullptr}, *many_logits = nullptr;  // g1, g2: gates, or the results of two mixers
     void *h1 = nullptr, *h2 = nullptr, *y_t[2] = {nullptr, nullptr}, *m = nullptr, *h_head = nullptr;
     CUtensorMap map_h1{}, map_h2{}, map_head{};
-    std::vector<CUtensorMap> map_y, map_m;  // per mixer, per layer: the pitches differ
+    std::vector<CUtensorMap> map_y, map_q, map_m;  // per mixer, per mixer, per layer: the pitches differ
     float *x_mid = nullptr, *past = nullptr;  // residual stream between mixer and feed-forward; vectors of the depth averages, [vector][token][width]
     void* q = nullptr;                      // normed queries
     struct Experts {                        // mixture of experts: router, chosen pairs and their activations and results
@@ -390,6 +392,9 @@ int layered_store_create(const LayeredModel& m, int slots, int ctx, Alloc alloc,
             const size_t dp = round_up(l.dim, 8), vp = round_up(l.vdim, 8), rows = size_t(slots) * c.ring * l.kv_heads, pools = size_t(slots) * c.blocks * l.kv_heads;
             if ((rc = alloc(&c.k, rows * dp * m.elem())) || (rc = alloc(&c.v, rows * vp * m.elem())) || (rc = alloc(&c.pk, pools * dp * m.elem())) || (rc = alloc(&c.pv, pools * vp * m.elem())))
                 return rc;
+            if (l.kind == MixerKind::kLogistic && !m.f32 && logistic_tc_fits(l.dim, l.vdim) &&
+                ((rc = tensor_map_3d_bf16(&s.kmap, c.k, l.kv_heads * dp, c.ring, slots, 64, kLtKeys)) || (rc = tensor_map_3d_bf16(&s.vmap, c.v, l.kv_heads * vp, c.ring, slots, 64, kLtKeys))))
+                return rc;
         }
     return QUINTRIT_OK;
 }
@@ -411,17 +416,11 @@ inline void layered_store_view(const LayeredModel& m, const LayeredStore& st, si
 inline int attention_splits(const MixerSpec& l, int ctx, int n, int sm_count) {
     if (l.kind == MixerKind::kLogistic) {
         const int gqa = l.heads / l.kv_heads, per = logistic_heads(gqa), groups = l.kv_heads * ((gqa + per - 1) / per) * n;
-        return std::max(1, std::min({(ctx + kLaKeys - 1) / kLaKeys, 4 * sm_count / groups, 64}));
+        return std::max(1, std::min({(ctx + kLaKeys - 1) / kLaKeys, (sm_count + groups - 1) / groups, 64}));
     }
     const int groups = l.kv_heads * ((l.heads / l.kv_heads + kPaHeads - 1) / kPaHeads) * n;
     const int keys = std::min(ctx, l.window) + (l.pool > 0 ? ctx / l.pool : 0);
     return std::max(1, std::min({(keys + kPaTile - 1) / kPaTile, 4 * sm_count / groups, 64}));
-}
-inline int logistic_dims_slot(int dims) { return dims == 32 ? 0 : dims == 64 ? 1 : dims == 96 ? 2 : dims == 128 ? 3 : dims == 192 ? 4 : 5; }
-typedef void (*LogisticKernel)(LogisticArgs);
-inline LogisticKernel logistic_kernel_for(int dims) {
-    static const LogisticKernel k[] = {logistic_mma_kernel<32>, logistic_mma_kernel<64>, logistic_mma_kernel<96>, logistic_mma_kernel<128>, logistic_mma_kernel<192>, logistic_mma_kernel<256>};
-    return k[logistic_dims_slot(dims)];
 }
 typedef void (*LogisticStep)(LogisticArgs, int, int);
 template <typename T, bool OWN> LogisticStep logistic_step_for(int heads) {
@@ -473,7 +472,7 @@ inline int layered_decoder_setup(quintrit_b200_decoder* d, const std::shared_ptr
                     work = std::max(work, chunk_work(nullptr, l.kind == MixerKind::kMamba2, l.heads, l.vdim, l.key_dim(), l.groups, kLayeredChunk, &cw));
                 continue;
             }
-            if (l.kind == MixerKind::kLogistic) queries = std::max(queries, size_t(l.heads) * round_up(l.dim, 8));
+            if (l.kind == MixerKind::kLogistic) queries = std::max(queries, size_t(l.heads) * round_up(l.dim, 64));
             const int per = l.kind == MixerKind::kLogistic ? logistic_heads(l.heads / l.kv_heads) : kPaHeads;
             groups = std::max<size_t>(groups, size_t(l.kv_heads) * ((l.heads / l.kv_heads + per - 1) / per));
             for (int n = 1; n <= kLayeredMaxBatch; ++n) {
@@ -500,11 +499,14 @@ inline int layered_decoder_setup(quintrit_b200_decoder* d, const std::shared_ptr
             (rc = tensor_map_2d_bf16(&y->map_head, y->h_head, m.embed.pitch, kDenseBox, kDenseK, kDenseBox)))
             return rc;
         if (top > 0 && (rc = tensor_map_2d_bf16(&x.map_h, x.h, m.embed.pitch, C * top, kDenseK, kDenseBox))) return rc;
-        y->map_y.resize(m.mixers), y->map_m.resize(m.layers.size()), x.map_m.resize(m.layers.size());
+        y->map_y.resize(m.mixers), y->map_q.resize(m.mixers), y->map_m.resize(m.layers.size()), x.map_m.resize(m.layers.size());
         for (size_t i = 0; i < m.layers.size(); ++i) {
             const LayeredLayer& ly = m.layers[i];
-            for (size_t k = 0; k < ly.mix.size(); ++k)
+            for (size_t k = 0; k < ly.mix.size(); ++k) {
+                const MixerSpec& l = ly.mix[k].spec;
                 if ((rc = tensor_map_2d_bf16(&y->map_y[ly.mixer0 + k], y->y_t[k], ly.mix[k].o.pitch, C, kDenseK, kDenseBox))) return rc;
+                if (l.kind == MixerKind::kLogistic && (rc = tensor_map_2d_bf16(&y->map_q[ly.mixer0 + k], y->q, size_t(l.heads) * round_up(l.dim, 64), C, 64, kLtRows))) return rc;
+            }
             y->map_m[i] = y->map_y[ly.mixer0];
             if (ly.spec.ff_kind != FfKind::kNone && (rc = tensor_map_2d_bf16(&y->map_m[i], y->m, ly.down.pitch, C, kDenseK, kDenseBox))) return rc;
             if (ly.spec.ff_kind == FfKind::kExperts && (rc = tensor_map_2d_bf16(&x.map_m[i], x.m, ly.experts_down.pitch, C * ly.spec.top, kDenseK, kDenseBox))) return rc;
@@ -541,7 +543,7 @@ inline int layered_decoder_setup(quintrit_b200_decoder* d, const std::shared_ptr
                              reinterpret_cast<const void*>(pooled_attention_mma_kernel<128>)};
     for (int heads : {1, 4, 8})
         for (LogisticStep k : {logistic_step_for<bf16, true>(heads), logistic_step_for<float, true>(heads), logistic_step_for<float, false>(heads)}) kernels.push_back(reinterpret_cast<const void*>(k));
-    for (int dims : {32, 64, 96, 128, 192, 256}) kernels.push_back(reinterpret_cast<const void*>(logistic_kernel_for(dims)));
+    kernels.push_back(reinterpret_cast<const void*>(logistic_mma_kernel<kLogisticMmaDims>)), kernels.push_back(reinterpret_cast<const void*>(logistic_tc_kernel));
     for (int rows : {32, 64, 128, 256}) {
         kernels.push_back(reinterpret_cast<const void*>(retention_kernels(rows, 64).state));
         for (int cols : {64, 128, 256}) kernels.push_back(reinterpret_cast<const void*>(retention_kernels(rows, cols).out));
@@ -553,7 +555,7 @@ inline int layered_decoder_setup(quintrit_b200_decoder* d, const std::shared_ptr
     for (const LayeredLayer& ly : m.layers) {
         size_t need = std::max<size_t>({3 * wp * 4, (size_t(ly.mix[0].o.pitch) + (ly.mix.size() > 1 ? ly.mix[1].o.pitch : ly.down.pitch)) * 4});
         if (!ly.spec.parallel) need = std::max(need, (size_t(ly.mix[0].o.pitch) + 2 * (ly.mix.size() > 1 ? ly.mix[1].o.pitch : ly.mix[0].o.pitch)) * 4);
-        if (ly.spec.ff_kind == FfKind::kExperts) need = std::max({need, (size_t(ly.spec.top) * ly.experts_down.pitch + ly.down.pitch) * 4, (wp + 4 * ly.spec.experts) * 4});
+        if (ly.spec.ff_kind == FfKind::kExperts) need = std::max({need, (size_t(ly.spec.top) * ly.experts_down.pitch + ly.down.pitch) * 4, (wp + 8 * size_t(ly.spec.experts)) * 4});
         for (const LayeredMixer& x : ly.mix) {
             const MixerSpec& l = x.spec;
             need = std::max(need, size_t(l.inner()) * 4);
@@ -608,9 +610,9 @@ inline int layered_retention_chunks(quintrit_b200_decoder* d, const MixerSpec& l
     retention_work(d->lay->work, l.heads, l.dim, l.vdim, a.tokens, &r.work);
     const RetentionKernels f = retention_kernels(r.work.rows, r.work.v_pad);
     const int chunks = retention_chunks(a.tokens);
-    const bool even = l.dim % 2 == 0 && l.vdim % 2 == 0 && l.rot_dims % 4 == 0 && a.ld % 2 == 0 && (a.p - d->lay->p1) % 2 == 0;
-    const dim3 grid(l.heads, r.work.tokens / kRetPrep);
-    even ? retention_prepare_kernel<true><<<grid, 128, 0, d->stream>>>(r) : retention_prepare_kernel<false><<<grid, 128, 0, d->stream>>>(r);
+    r.pairs = l.dim % 2 == 0 && l.vdim % 2 == 0 && l.rot_dims % 4 == 0 && a.ld % 2 == 0 && (a.p - d->lay->p1) % 2 == 0;
+    const dim3 grid((l.heads + 3) / 4, r.work.tokens / kRetPrep);
+    r.pairs ? retention_prepare_kernel<true><<<grid, 128, 0, d->stream>>>(r) : retention_prepare_kernel<false><<<grid, 128, 0, d->stream>>>(r);
     QTB_LAUNCH_CHECK();
     f.state<<<dim3(l.heads, chunks, r.work.v_pad / kRetV), 128, f.state_smem, d->stream>>>(r);
     QTB_LAUNCH_CHECK();
@@ -654,6 +656,8 @@ inline int layered_chunk_scan(quintrit_b200_decoder* d, const MixerSpec& l, cons
     QTB_LAUNCH_CHECK();
     return QUINTRIT_OK;
 }
+
+constexpr unsigned int kDenseSpinLimit = 1u << 16;  // polls of up to 20 us each: about a second before a wait gives up
 
 // Mixer k of a layer over the projections in y.p1. *ready: its output is in y.y_t[k], normed, gated and in the storage type, not in y.y[k].
 template <typename T>
@@ -704,7 +708,7 @@ int layered_mixer(quintrit_b200_decoder* d, size_t li, int k, int n, const Layer
         a.tokens = tokens, a.pos = tg.pos, a.seq = tg.seq, a.p = p, a.ld = ld;
         a.heads = l.heads, a.kv_heads = l.kv_heads, a.dim = l.dim, a.vdim = l.vdim, a.dim_pad = round_up(l.dim, 8), a.vdim_pad = round_up(l.vdim, 8);
         a.scale = l.scale, a.eps = d->eps, a.q_norm = w.q_norm, a.k_norm = w.k_norm, a.temp_coef = l.temp_coef, a.temp_every = l.temp_every, a.value_norm = l.value_norm;
-        a.slope = w.slope, a.bias = w.logit_bias, a.q = y.q, a.k = st.cache.k, a.v = st.cache.v, a.capacity = st.cache.ring;
+        a.slope = w.slope, a.bias = w.logit_bias, a.q = y.q, a.q_pad = round_up(l.dim, 64), a.k = st.cache.k, a.v = st.cache.v, a.capacity = st.cache.ring;
         a.out = y.y_t[k], a.out_pitch = w.o.pitch, a.y = y.y[k], a.part = y.part_acc, a.done = y.done;
         const int gqa = l.heads / l.kv_heads, per = logistic_heads(gqa), hg = l.kv_heads * ((gqa + per - 1) / per), elem = sizeof(T);
         const size_t smem = logistic_step_smem(per, a.dim_pad, a.vdim, a.vdim_pad, elem);
@@ -715,11 +719,16 @@ int layered_mixer(quintrit_b200_decoder* d, size_t li, int k, int n, const Layer
             QTB_LAUNCH_CHECK();
             return QUINTRIT_OK;
         }
-        logistic_prepare_kernel<T><<<n, 256, 0, s>>>(a);
+        logistic_prepare_kernel<T><<<n + (sizeof(T) == 2 ? kLtKeys - 1 : 0), 256, 0, s>>>(a);
         QTB_LAUNCH_CHECK();
         if constexpr (sizeof(T) == 2) {
-            const int dims = logistic_mma_dims(l.dim, l.vdim);
-            logistic_kernel_for(dims)<<<dim3((tokens + kPmRows - 1) / kPmRows, l.heads), kPmThreads, pooled_mma_smem(dims), s>>>(a);
+            if (logistic_tc_fits(l.dim, l.vdim)) {
+                LogisticTcArgs t{};
+                t.a = a, t.k_slices = logistic_tc_slices(l.dim), t.v_slices = logistic_tc_slices(l.vdim), t.slot = tg.slot, t.status = d->d_counters + 2, t.spin_limit = kDenseSpinLimit;
+                logistic_tc_kernel<<<dim3((tokens + kLtRows - 1) / kLtRows, l.heads), kLtThreads, logistic_tc_smem(l.dim, l.vdim), s>>>(y.map_q[ly.mixer0 + k], st.kmap, st.vmap, t);
+            } else {
+                logistic_mma_kernel<kLogisticMmaDims><<<dim3((tokens + kPmRows - 1) / kPmRows, l.heads), kPmThreads, pooled_mma_smem(kLogisticMmaDims), s>>>(a);
+            }
             *ready = true;
         } else {
             a.splits = 1;
@@ -759,8 +768,6 @@ int layered_mixer(quintrit_b200_decoder* d, size_t li, int k, int n, const Layer
     QTB_LAUNCH_CHECK();
     return QUINTRIT_OK;
 }
-
-constexpr unsigned int kDenseSpinLimit = 1u << 16;  // polls of up to 20 us each: about a second before a wait gives up
 
 // Product of `n_stack` stacks over the activations h (bf16: through their tensor maps), tokens = n.
 template <typename T>
@@ -913,7 +920,7 @@ int layered_sequential_step(quintrit_b200_decoder* d, size_t li, const LayeredTa
     MoeUpStepArgs u{};
     u.router = layered_router(l.spec), u.logits = y.ex.logits, u.h = y.h2, u.w = l.experts_in.w, u.pitch = l.experts_in.pitch, u.rows_pad = l.expert_rows(), u.ff = l.spec.ff;
     u.m = y.ex.m, u.m_pitch = l.experts_down.pitch, u.chosen = y.ex.chosen, u.weight = y.ex.weight;
-    launch_dependent(moe_up_step_kernel<T>, dim3(std::min((l.spec.top * l.spec.ff + warps - 1) / warps, 4 * m.sm_count)), kProjectThreads, (size_t(u.pitch) + l.spec.experts) * sizeof(float), s, u);
+    launch_dependent(moe_up_step_kernel<T>, dim3(std::min((l.spec.top * l.spec.ff + warps - 1) / warps, 4 * m.sm_count)), kProjectThreads, (size_t(u.pitch) + 2 * l.spec.experts) * sizeof(float), s, u);
     QTB_LAUNCH_CHECK();
     MoeDownStepArgs f{};
     f.x = sets > 1 ? y.x_mid : y.x, f.x_out = y.x, f.width = W, f.top = l.spec.top, f.m = y.ex.m, f.w = l.experts_down.w, f.pitch = l.experts_down.pitch, f.rows_pad = l.expert_down_rows();
@@ -935,7 +942,7 @@ int layered_experts(quintrit_b200_decoder* d, size_t li, int n) {
     MoeRouteArgs r{};
     r.router = layered_router(sp), r.tokens = n, r.logits = x.logits, r.chosen = x.chosen, r.weight = x.weight, r.count = x.count, r.rank = x.rank, r.first = x.first, r.row = x.row;
     r.up_runs = x.up_runs, r.down_runs = x.down_runs, r.n_runs = x.n_runs, r.up_rows = l.expert_rows(), r.down_rows = l.expert_down_rows(), r.tile = sizeof(T) != 2 ? kF32Tile : n * sp.top >= 160 * sp.experts ? 256 : 128;  // (the wider tile where an expert's share fills most of it)
-    moe_route_kernel<<<(n + 3) / 4, 128, size_t(4) * sp.experts * sizeof(float), s>>>(r);
+    moe_route_kernel<<<(n + 3) / 4, 128, size_t(8) * sp.experts * sizeof(uint32_t), s>>>(r);
     QTB_LAUNCH_CHECK();
     moe_plan_kernel<<<1, 1024, 0, s>>>(r);
     QTB_LAUNCH_CHECK();

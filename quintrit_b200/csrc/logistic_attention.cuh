@@ -25,7 +25,8 @@ struct LogisticArgs {
     float temp_coef, temp_every;    // q times 1 + coef ln(floor((pos + 1) / every) + 1)
     bool value_norm;
     const float *slope, *bias;      // per head
-    void* q;                  // [token][heads][dim_pad], storage type: what logistic_prepare_kernel makes of the queries
+    void* q;                  // [token][heads][q_pad], storage type: what logistic_prepare_kernel makes of the queries, zero beyond dim
+    int q_pad;
     void *k, *v;              // cache: [slot][capacity][kv_heads][dim_pad], [..][vdim_pad]
     int capacity;
     void* out;                // [token][out_pitch], storage type (many tokens) ...
@@ -36,12 +37,20 @@ struct LogisticArgs {
     unsigned int* done;       // step, splits > 1: [token][head groups], zero between launches
 };
 
-// Norms of one token's queries, keys and values; the queries' temperature; keys and values go to the cache. One block per token.
+// Norms of one token's queries, keys and values; the queries' temperature; keys and values go to the cache. One block per token; blocks beyond
+// the last token clear the rows of the cache that follow it, so that kernels may multiply whole tiles of it by weights of zero.
 template <typename T>
 __global__ void __launch_bounds__(256) logistic_prepare_kernel(const __grid_constant__ LogisticArgs a) {
     __shared__ float red[8];
     const int z = blockIdx.x;
     const uint32_t slot = a.seq.pos_stride != 0 ? seq_of(a.seq, z) : 0, pos = seq_position(a.seq, a.pos, z);
+    if (z >= a.tokens) {  // (of a prompt: its position is pos)
+        if (pos >= static_cast<uint32_t>(a.capacity)) return;
+        const size_t row = size_t(slot) * a.capacity + pos;
+        for (int i = threadIdx.x; i < a.kv_heads * a.dim_pad; i += blockDim.x) static_cast<T*>(a.k)[row * a.kv_heads * a.dim_pad + i] = to_storage<T>(0.0f);
+        for (int i = threadIdx.x; i < a.kv_heads * a.vdim_pad; i += blockDim.x) static_cast<T*>(a.v)[row * a.kv_heads * a.vdim_pad + i] = to_storage<T>(0.0f);
+        return;
+    }
     const float *q = a.p + size_t(z) * a.ld, *k = q + a.heads * a.dim, *v = k + a.kv_heads * a.dim;
     const int tid = threadIdx.x, nt = blockDim.x, nq = a.heads * a.dim, nk = a.kv_heads * a.dim;
     float iq = 1.0f, ik = 1.0f;
@@ -58,9 +67,9 @@ __global__ void __launch_bounds__(256) logistic_prepare_kernel(const __grid_cons
         ik = 1.0f / sqrtf(block_sum(s, red) / static_cast<float>(nk) + a.eps);
     }
     const float temp = a.temp_coef != 0.0f ? 1.0f + a.temp_coef * logf(floorf(static_cast<float>(pos + 1) / a.temp_every) + 1.0f) : 1.0f;
-    T* qo = static_cast<T*>(a.q) + size_t(z) * a.heads * a.dim_pad;
-    for (int i = tid; i < a.heads * a.dim_pad; i += nt) {
-        const int h = i / a.dim_pad, e = i % a.dim_pad, at = h * a.dim + e;
+    T* qo = static_cast<T*>(a.q) + size_t(z) * a.heads * a.q_pad;
+    for (int i = tid; i < a.heads * a.q_pad; i += nt) {
+        const int h = i / a.q_pad, e = i % a.q_pad, at = h * a.dim + e;
         qo[i] = to_storage<T>(e < a.dim ? q[at] * iq * (a.q_norm != nullptr ? a.q_norm[at] : 1.0f) * temp : 0.0f);
     }
     const size_t row = size_t(slot) * a.capacity + pos;
@@ -190,7 +199,7 @@ __global__ void __launch_bounds__(kLaThreads, H > 4 ? 1 : 2) logistic_step_kerne
             }
         }
     } else {
-        for (int i = tid; i < nh * a.dim_pad; i += kLaThreads) qs[i] = from_storage(static_cast<const T*>(a.q)[(size_t(z) * a.heads + h0) * a.dim_pad + i]);
+        for (int i = tid; i < nh * a.dim_pad; i += kLaThreads) qs[i] = from_storage(static_cast<const T*>(a.q)[(size_t(z) * a.heads + h0 + i / a.dim_pad) * a.q_pad + i % a.dim_pad]);
     }
     float acc[H][P];
 #pragma unroll
@@ -286,45 +295,53 @@ __global__ void __launch_bounds__(kLaThreads, H > 4 ? 1 : 2) logistic_step_kerne
     if (!last_block) return;
     if (tid == 0) *counter = 0;
     __threadfence();
-    // the shares that had keys, their sums by parts of the block: as many threads per result as there are for it
-    const int live = per > 0 ? max(1, (total + per - 1) / per) : 1, results = nh * a.vdim, teams = max(1, min(kLaThreads / max(results, 1), 8));
-    if (teams == 1) {
+    // the shares that had keys; as many threads per four results as there are for them
+    const int live = per > 0 ? max(1, (total + per - 1) / per) : 1, results = nh * a.vdim;
+    const float* part0 = a.part + (size_t(z) * a.heads + h0) * a.splits * a.vdim;
+    float* y0 = a.y + (size_t(z) * a.heads + h0) * a.vdim;
+    if (a.vdim % 4 != 0) {
         for (int i = tid; i < results; i += kLaThreads) {
-            const int h = i / a.vdim, c = i % a.vdim;
-            const float* part = a.part + ((size_t(z) * a.heads + h0 + h) * a.splits) * a.vdim + c;
+            const float* part = part0 + size_t(i / a.vdim) * a.splits * a.vdim + i % a.vdim;
             float s = 0.0f;
 #pragma unroll 16
             for (int k = 0; k < live; ++k) s += __ldcg(part + size_t(k) * a.vdim);
-            a.y[(size_t(z) * a.heads + h0 + h) * a.vdim + c] = s;
+            y0[i] = s;
         }
         return;
     }
-    const int team = tid / results, i = tid % results, h = i / a.vdim, c = i % a.vdim;
-    float s = 0.0f;
-    if (team < teams) {
-        const float* part = a.part + ((size_t(z) * a.heads + h0 + h) * a.splits) * a.vdim + c;
-#pragma unroll 16
-        for (int k = team; k < live; k += teams) s += __ldcg(part + size_t(k) * a.vdim);
-        red[tid] = s;
-    }
+    const int quads = results / 4, per_head = a.vdim / 4, teams = max(1, min(kLaThreads / quads, 8)), team = tid / quads;
+    float4* team_sum = reinterpret_cast<float4*>(la_sm);  // [teams][quads]: at most kLaThreads
+    if (teams == 1 || team < teams)
+        for (int i = teams == 1 ? tid : tid % quads; i < quads; i += teams == 1 ? kLaThreads : quads) {
+            const float4* part = reinterpret_cast<const float4*>(part0 + size_t(i / per_head) * a.splits * a.vdim) + i % per_head;
+            float4 s = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll 8
+            for (int k = teams == 1 ? 0 : team; k < live; k += teams) {
+                const float4 f = __ldcg(part + size_t(k) * per_head);
+                s.x += f.x, s.y += f.y, s.z += f.z, s.w += f.w;
+            }
+            if (teams == 1) reinterpret_cast<float4*>(y0)[i] = s;
+            else team_sum[tid] = s;
+        }
+    if (teams == 1) return;
     __syncthreads();
     if (team != 0) return;
-    for (int t = 1; t < teams; ++t) s += red[t * results + i];
-    a.y[(size_t(z) * a.heads + h0 + h) * a.vdim + c] = s;
+    float4 s = team_sum[tid];
+    for (int t = 1; t < teams; ++t) {
+        const float4 f = team_sum[t * quads + tid];
+        s.x += f.x, s.y += f.y, s.z += f.z, s.w += f.w;
+    }
+    reinterpret_cast<float4*>(y0)[tid] = s;
 }
 
 // ---- many query positions on the tensor cores of a warp --------------------------------------------------------------------------------------
-// 64 query positions of one head per block, keys in tiles of 64, fetched two tiles deep. A weight depends on its own score alone, so nothing is
+// For heads of more than 128 dimensions (logistic_attention_tc.cuh takes the others). 64 query positions of one head per block, keys in tiles of 64, fetched two tiles deep. A weight depends on its own score alone, so nothing is
 // rescaled. Weights enter the second product as two bf16 terms. grid: (query tiles, heads)
-inline int logistic_mma_dims(int dim, int vdim) {
-    const int d = dim > vdim ? dim : vdim;
-    return d <= 32 ? 32 : d <= 64 ? 64 : d <= 96 ? 96 : d <= 128 ? 128 : d <= 192 ? 192 : 256;
-}
+constexpr int kLogisticMmaDims = 256;
 template <int D>
 __global__ void __launch_bounds__(kPmThreads) logistic_mma_kernel(const __grid_constant__ LogisticArgs a) {
     extern __shared__ __align__(16) unsigned char pm_sm[];
     constexpr int kPitch = D + 8;
-    constexpr bool kKeepQ = D <= 128;           // query operands stay in registers
     bf16* qs = reinterpret_cast<bf16*>(pm_sm);  // [64][kPitch]
     bf16* kv = qs + kPmRows * kPitch;           // two stages of keys and values, [64][kPitch] each
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, c = lane & 3;
@@ -333,11 +350,11 @@ __global__ void __launch_bounds__(kPmThreads) logistic_mma_kernel(const __grid_c
     const int first = pos0 + q0, last = pos0 + min(q0 + kPmRows, a.tokens) - 1;
     const int dp = a.dim_pad, vp = a.vdim_pad;
     const bf16 *key0 = static_cast<const bf16*>(a.k) + size_t(kvh) * dp, *value0 = static_cast<const bf16*>(a.v) + size_t(kvh) * vp;
-    const bf16* query0 = static_cast<const bf16*>(a.q) + size_t(head) * dp;
+    const bf16* query0 = static_cast<const bf16*>(a.q) + size_t(head) * a.q_pad;
     for (int i = tid; i < kPmRows * (D / 8); i += kPmThreads) {
         const int r = i / (D / 8), p = i % (D / 8);
         const bool valid = q0 + r < a.tokens && p * 8 < dp;
-        cp_async16(qs + r * kPitch + p * 8, query0 + (valid ? size_t(q0 + r) * a.heads * dp + p * 8 : 0), valid);
+        cp_async16(qs + r * kPitch + p * 8, query0 + (valid ? size_t(q0 + r) * a.heads * a.q_pad + p * 8 : 0), valid);
     }
     const int tiles = last / kPmKeys + 1;
     auto fetch = [&](int tile, int stage) {
@@ -351,7 +368,6 @@ __global__ void __launch_bounds__(kPmThreads) logistic_mma_kernel(const __grid_c
         cp_async_commit_group();
     };
     fetch(0, 0);
-    uint32_t q[kKeepQ ? D / 16 : 1][4];
     float o[D / 8][4];
 #pragma unroll
     for (int j = 0; j < D / 8; ++j)
@@ -369,11 +385,6 @@ __global__ void __launch_bounds__(kPmThreads) logistic_mma_kernel(const __grid_c
             cp_async_wait_group<0>();
         }
         __syncthreads();
-        if constexpr (kKeepQ) {
-            if (tile == 0)
-#pragma unroll
-                for (int k = 0; k < D / 16; ++k) load_frag_a(q[k], qs + warp * 16 * kPitch + k * 16, kPitch);
-        }
         const bf16 *ks = kv + (tile & 1) * 2 * kPmKeys * kPitch, *vs = ks + kPmKeys * kPitch;
         float s[kPmKeys / 8][4];
 #pragma unroll
@@ -382,13 +393,14 @@ __global__ void __launch_bounds__(kPmThreads) logistic_mma_kernel(const __grid_c
             for (int e = 0; e < 4; ++e) s[j][e] = 0.0f;
 #pragma unroll
         for (int k = 0; k < D / 16; ++k) {
-            if constexpr (!kKeepQ) load_frag_a(q[0], qs + warp * 16 * kPitch + k * 16, kPitch);
+            uint32_t q[4];  // (too many to stay in registers)
+            load_frag_a(q, qs + warp * 16 * kPitch + k * 16, kPitch);
 #pragma unroll
             for (int j = 0; j < kPmKeys / 8; j += 2) {
                 uint32_t b[4];
                 load_frag_bt(b, ks + j * 8 * kPitch + k * 16, kPitch);
-                mma_16816(s[j], q[kKeepQ ? k : 0], b[0], b[1]);
-                mma_16816(s[j + 1], q[kKeepQ ? k : 0], b[2], b[3]);
+                mma_16816(s[j], q, b[0], b[1]);
+                mma_16816(s[j + 1], q, b[2], b[3]);
             }
         }
         const int k0 = tile * kPmKeys;

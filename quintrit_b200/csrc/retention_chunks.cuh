@@ -43,6 +43,7 @@ struct RetentionArgs {
     float eps;             // of the heads' norm
     void* out;             // [token][out_pitch], bf16
     int out_pitch;
+    bool pairs;            // sizes and columns are even: two neighbouring elements at a time
 };
 
 // powers a^0 .. a^T of a head's decay
@@ -50,15 +51,18 @@ __device__ __forceinline__ void decay_powers(float decay, float* pw) {
     for (int i = threadIdx.x; i <= kRetT; i += blockDim.x) pw[i] = i == 0 ? 1.0f : decay > 0.0f ? exp2f(static_cast<float>(i) * log2f(decay)) : 0.0f;
 }
 // Queries, keys and values of every token as the products take them. PAIRS: two neighbouring elements at a time (even sizes and columns).
-// grid: (heads, padded tokens / 16), 128 threads
+// Four heads a block: they share the angles. grid: (ceil(heads / 4), padded tokens / 16), 128 threads
 template <bool PAIRS>
 __global__ void __launch_bounds__(128) retention_prepare_kernel(const __grid_constant__ RetentionArgs r) {
+    __shared__ float2 angle[kRetPrep][128];  // (a head has at most 256 rotated dimensions)
     const ScanArgs& a = r.scan;
     const RetentionWork& w = r.work;
     constexpr int S = PAIRS ? 2 : 1;
-    const int head = blockIdx.x, t0 = blockIdx.y * kRetPrep, tid = threadIdx.x, n = a.n, half = a.rot_dims / 2;
+    const int t0 = blockIdx.y * kRetPrep, tid = threadIdx.x, n = a.n, half = a.rot_dims / 2;
     const uint32_t pos0 = seq_position(a.seq, a.pos, 0);
     const float scale = 1.0f / sqrtf(static_cast<float>(n));
+    for (int i = tid; i < kRetPrep * half; i += 128) angle[i / half][i % half] = rotation(a.turns[i % half], pos0 + t0 + i / half);
+    __syncthreads();
     auto put = [&](bf16* hi, bf16* lo, size_t at, const float (&v)[S]) {
         if constexpr (PAIRS) {
             uint32_t h, l;
@@ -77,43 +81,44 @@ __global__ void __launch_bounds__(128) retention_prepare_kernel(const __grid_con
             v[0] = there ? *p : 0.0f;
         }
     };
-    const int items = (w.rows - half) / S;  // an item is a pair to rotate (two neighbouring ones), or elements that stay as they are
-#pragma unroll 2
-    for (int i = tid; i < kRetPrep * items; i += 128) {
-        const int t = t0 + i / items, j = i % items * S;
-        const bool there = t < a.tokens;
-        const float* p = a.p + size_t(min(t, a.tokens - 1)) * a.ld + head * n;
-        const float* pk = p + a.heads * n;
-        const size_t at = (size_t(head) * w.tokens + t) * w.rows;
-        float q[S], k[S];
-        if (j < half) {
-            float q2[S], k2[S];
-            get(p + j, there, q), get(p + j + half, there, q2), get(pk + j, there, k), get(pk + j + half, there, k2);
-#pragma unroll
-            for (int e = 0; e < S; ++e) {
-                const float2 cs = rotation(a.turns[j + e], pos0 + t);
-                const float2 rq = rotate_pair(q[e], q2[e], cs), rk = rotate_pair(k[e], k2[e], cs);
-                q[e] = rq.x, q2[e] = rq.y, k[e] = rk.x * scale, k2[e] = rk.y * scale;
-            }
-            put(w.q_hi, w.q_lo, at + j, q), put(w.q_hi, w.q_lo, at + j + half, q2);
-            put(w.k_hi, w.k_lo, at + j, k), put(w.k_hi, w.k_lo, at + j + half, k2);
-        } else {
-            const bool in = there && j + half < n;
-            get(p + j + half, in, q), get(pk + j + half, in, k);
-#pragma unroll
-            for (int e = 0; e < S; ++e) k[e] *= scale;
-            put(w.q_hi, w.q_lo, at + j + half, q), put(w.k_hi, w.k_lo, at + j + half, k);
-        }
-    }
-    const int cols = w.v_pad / S;
+    const int items = (w.rows - half) / S, cols = w.v_pad / S;  // an item is a pair to rotate (two neighbouring ones), or elements that stay as they are
+    for (int head = blockIdx.x * 4; head < min(a.heads, static_cast<int>(blockIdx.x) * 4 + 4); ++head) {
 #pragma unroll 4
-    for (int i = tid; i < kRetPrep * cols; i += 128) {
-        const int t = t0 + i / cols, c = i % cols * S;
-        float v[S];
-        get(a.p + size_t(min(t, a.tokens - 1)) * a.ld + 2 * a.heads * n + head * a.vdim + c, t < a.tokens && c < a.vdim, v);
-        bf16* out = w.v + (size_t(head) * w.tokens + t) * w.v_pad + c;
-        if constexpr (PAIRS) *reinterpret_cast<uint32_t*>(out) = pack_bf16(v[0], v[1]);
-        else *out = __float2bfloat16_rn(v[0]);
+        for (int i = tid; i < kRetPrep * items; i += 128) {
+            const int t = t0 + i / items, j = i % items * S;
+            const bool there = t < a.tokens;
+            const float* p = a.p + size_t(min(t, a.tokens - 1)) * a.ld + head * n;
+            const float* pk = p + a.heads * n;
+            const size_t at = (size_t(head) * w.tokens + t) * w.rows;
+            float q[S], k[S];
+            if (j < half) {
+                float q2[S], k2[S];
+                get(p + j, there, q), get(p + j + half, there, q2), get(pk + j, there, k), get(pk + j + half, there, k2);
+#pragma unroll
+                for (int e = 0; e < S; ++e) {
+                    const float2 cs = angle[t - t0][j + e];
+                    const float2 rq = rotate_pair(q[e], q2[e], cs), rk = rotate_pair(k[e], k2[e], cs);
+                    q[e] = rq.x, q2[e] = rq.y, k[e] = rk.x * scale, k2[e] = rk.y * scale;
+                }
+                put(w.q_hi, w.q_lo, at + j, q), put(w.q_hi, w.q_lo, at + j + half, q2);
+                put(w.k_hi, w.k_lo, at + j, k), put(w.k_hi, w.k_lo, at + j + half, k2);
+            } else {
+                const bool in = there && j + half < n;
+                get(p + j + half, in, q), get(pk + j + half, in, k);
+#pragma unroll
+                for (int e = 0; e < S; ++e) k[e] *= scale;
+                put(w.q_hi, w.q_lo, at + j + half, q), put(w.k_hi, w.k_lo, at + j + half, k);
+            }
+        }
+#pragma unroll 4
+        for (int i = tid; i < kRetPrep * cols; i += 128) {
+            const int t = t0 + i / cols, c = i % cols * S;
+            float v[S];
+            get(a.p + size_t(min(t, a.tokens - 1)) * a.ld + 2 * a.heads * n + head * a.vdim + c, t < a.tokens && c < a.vdim, v);
+            bf16* out = w.v + (size_t(head) * w.tokens + t) * w.v_pad + c;
+            if constexpr (PAIRS) *reinterpret_cast<uint32_t*>(out) = pack_bf16(v[0], v[1]);
+            else *out = __float2bfloat16_rn(v[0]);
+        }
     }
 }
 
@@ -350,12 +355,23 @@ __global__ void __launch_bounds__(128) retention_out_kernel(const __grid_constan
         const float inv = 1.0f / sqrtf(ss[h] / static_cast<float>(a.vdim) + r.eps);
         const float* gate = a.p + size_t(t0 + t) * a.ld + 2 * a.heads * n + a.heads * a.vdim + head * a.vdim;
         bf16* out = static_cast<bf16*>(r.out) + size_t(t0 + t) * r.out_pitch + head * a.vdim;
+        const auto gated = [&](float v, float z) { return v * inv * __fdividef(z, 1.0f + __expf(-z)); };
+        if (r.pairs) {
+#pragma unroll
+            for (int j = 0; j < V / 8; ++j) {
+                const int v = j * 8 + 2 * c;
+                if (v >= a.vdim) continue;
+                const float2 z = *reinterpret_cast<const float2*>(gate + v);
+                *reinterpret_cast<uint32_t*>(out + v) = pack_bf16(gated(o[j][2 * h], z.x), gated(o[j][2 * h + 1], z.y));
+            }
+            continue;
+        }
 #pragma unroll
         for (int j = 0; j < V / 8; ++j)
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
                 const int v = j * 8 + 2 * c + e;
-                if (v < a.vdim) out[v] = __float2bfloat16_rn(o[j][2 * h + e] * inv * silu_f(gate[v]));
+                if (v < a.vdim) out[v] = __float2bfloat16_rn(gated(o[j][2 * h + e], gate[v]));
             }
     }
 }
