@@ -82,7 +82,9 @@ struct NormParams {
     const float* b;      // not nullptr: the tanh form
     float alpha;
 };
-__device__ __forceinline__ float norm_value(const NormParams& n, float x, float inv, int i) { return n.b != nullptr ? tanhf(n.alpha * x) * n.w[i] + n.b[i] : x * inv * n.w[i]; }
+__device__ __forceinline__ float norm_value(const NormParams& n, float x, float inv, int i) {
+    return n.b != nullptr ? tanhf(n.alpha * x) * __ldg(n.w + i) + __ldg(n.b + i) : x * inv * __ldg(n.w + i);
+}
 
 // Two vectors whose RMS norms, each with its weight, are averaged and added to the residual stream.
 struct PairSum {

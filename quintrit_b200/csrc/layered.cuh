@@ -612,7 +612,7 @@ inline int layered_retention_chunks(quintrit_b200_decoder* d, const MixerSpec& l
     const int chunks = retention_chunks(a.tokens);
     r.pairs = l.dim % 2 == 0 && l.vdim % 2 == 0 && l.rot_dims % 4 == 0 && a.ld % 2 == 0 && (a.p - d->lay->p1) % 2 == 0;
     const dim3 grid((l.heads + 3) / 4, r.work.tokens / kRetPrep);
-    r.pairs ? retention_prepare_kernel<true><<<grid, 128, 0, d->stream>>>(r) : retention_prepare_kernel<false><<<grid, 128, 0, d->stream>>>(r);
+    r.pairs ? retention_prepare_kernel<true><<<grid, 256, 0, d->stream>>>(r) : retention_prepare_kernel<false><<<grid, 256, 0, d->stream>>>(r);
     QTB_LAUNCH_CHECK();
     f.state<<<dim3(l.heads, chunks, r.work.v_pad / kRetV), 128, f.state_smem, d->stream>>>(r);
     QTB_LAUNCH_CHECK();

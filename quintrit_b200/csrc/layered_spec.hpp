@@ -119,6 +119,11 @@ struct ConfigReader {
         }
         return p;
     }
+    // An object that may be left out (or null).
+    const JsonValue* optional(const JsonValue& v, const std::string& where, const char* key) {
+        const JsonValue* p = v.get(key);
+        return p == nullptr || p->is(JsonValue::kNull) ? nullptr : object(v, where, key);
+    }
     int size(const JsonValue& v, const std::string& where, const char* key) {
         const JsonValue* p = v.get(key);
         uint64_t u = 0;
@@ -213,8 +218,7 @@ inline MixerSpec read_retention(ConfigReader& r, const JsonValue& v, const std::
     MixerSpec x;
     x.kind = MixerKind::kRetention;
     x.heads = r.size(v, where, "heads"), x.dim = r.size(v, where, "dim"), x.vdim = r.size(v, where, "vdim");
-    const JsonValue& rot = *r.object(v, where, "rot");
-    x.rot_dims = r.size(rot, where + "rot.", "dims"), x.rot_base = r.real(rot, where + "rot.", "base");
+    if (const JsonValue* rot = r.optional(v, where, "rot")) x.rot_dims = r.size(*rot, where + "rot.", "dims"), x.rot_base = r.real(*rot, where + "rot.", "base");
     const JsonValue* decay = v.get("decay");
     if (decay == nullptr || !decay->is(JsonValue::kArray) || decay->items.size() != static_cast<size_t>(x.heads)) {
         r.fail_key(where, "decay", "is not a list of one number per head");
@@ -233,8 +237,7 @@ inline MixerSpec read_logistic(ConfigReader& r, const JsonValue& v, const std::s
     x.kind = MixerKind::kLogistic;
     x.heads = r.size(v, where, "heads"), x.kv_heads = r.size(v, where, "kv_heads"), x.dim = r.size(v, where, "dim"), x.vdim = r.size(v, where, "vdim");
     x.scale = r.number(v, where, "scale");
-    const JsonValue& temp = *r.object(v, where, "q_temp");
-    x.temp_coef = r.number(temp, where + "q_temp.", "coef"), x.temp_every = r.number(temp, where + "q_temp.", "every");
+    if (const JsonValue* temp = r.optional(v, where, "q_temp")) x.temp_coef = r.number(*temp, where + "q_temp.", "coef"), x.temp_every = r.number(*temp, where + "q_temp.", "every");
     if (!(x.temp_every > 0.0f)) r.fail_key(where + "q_temp.", "every", "is not positive");
     x.value_norm = true, x.distance_bias = true;
     x.in = {m + "q", m + "k", m + "v"}, x.out = m + "o";
@@ -274,13 +277,13 @@ inline std::string read_tosevik(const JsonValue& cfg, LayeredSpec* out) {
             const std::string kind = r.text(*mlp, where + "mlp.", "kind"), f = p + "mlp.";
             if (kind != "moe") return "config.json: " + where + "mlp.kind '" + kind + "' is unknown";
             const JsonValue& router = *r.object(*mlp, where + "mlp.", "router");
-            const JsonValue& groups = *r.object(router, where + "mlp.router.", "groups");
             l.ff_kind = FfKind::kExperts, l.norm2 = p + "norm2";
             l.ff = r.size(*r.object(*mlp, where + "mlp.", "expert"), where + "mlp.expert.", "ff");
             l.shared_ff = r.size(*r.object(*mlp, where + "mlp.", "shared"), where + "mlp.shared.", "ff");
             l.experts = r.size(router, where + "mlp.router.", "experts"), l.top = r.size(router, where + "mlp.router.", "top");
             l.router_scale = r.number(router, where + "mlp.router.", "scale");
-            l.expert_groups = r.size(groups, where + "mlp.router.groups.", "count"), l.keep_groups = r.size(groups, where + "mlp.router.groups.", "keep");
+            if (const JsonValue* g = r.optional(router, where + "mlp.router.", "groups"))
+                l.expert_groups = r.size(*g, where + "mlp.router.groups.", "count"), l.keep_groups = r.size(*g, where + "mlp.router.groups.", "keep");
             l.expert_prefix = f + "e", l.router = f + "router";
             l.shared_gate = f + "shared.gate", l.shared_up = f + "shared.up", l.shared_down = f + "shared.down", l.shared_scale = f + "shared.sg";
         }

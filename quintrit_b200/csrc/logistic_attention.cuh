@@ -68,15 +68,16 @@ __global__ void __launch_bounds__(256) logistic_prepare_kernel(const __grid_cons
     }
     const float temp = a.temp_coef != 0.0f ? 1.0f + a.temp_coef * logf(floorf(static_cast<float>(pos + 1) / a.temp_every) + 1.0f) : 1.0f;
     T* qo = static_cast<T*>(a.q) + size_t(z) * a.heads * a.q_pad;
+#pragma unroll 4
     for (int i = tid; i < a.heads * a.q_pad; i += nt) {
         const int h = i / a.q_pad, e = i % a.q_pad, at = h * a.dim + e;
-        qo[i] = to_storage<T>(e < a.dim ? q[at] * iq * (a.q_norm != nullptr ? a.q_norm[at] : 1.0f) * temp : 0.0f);
+        qo[i] = to_storage<T>(e < a.dim ? __ldg(q + at) * iq * (a.q_norm != nullptr ? __ldg(a.q_norm + at) : 1.0f) * temp : 0.0f);
     }
     const size_t row = size_t(slot) * a.capacity + pos;
     T* ko = static_cast<T*>(a.k) + row * a.kv_heads * a.dim_pad;
     for (int i = tid; i < a.kv_heads * a.dim_pad; i += nt) {
         const int h = i / a.dim_pad, e = i % a.dim_pad, at = h * a.dim + e;
-        ko[i] = to_storage<T>(e < a.dim ? k[at] * ik * (a.k_norm != nullptr ? a.k_norm[at] : 1.0f) : 0.0f);
+        ko[i] = to_storage<T>(e < a.dim ? __ldg(k + at) * ik * (a.k_norm != nullptr ? __ldg(a.k_norm + at) : 1.0f) : 0.0f);
     }
     T* vo = static_cast<T*>(a.v) + row * a.kv_heads * a.vdim_pad;
     const int warps = nt >> 5, lane = tid & 31;
@@ -201,7 +202,9 @@ __global__ void __launch_bounds__(kLaThreads, H > 4 ? 1 : 2) logistic_step_kerne
     } else {
         for (int i = tid; i < nh * a.dim_pad; i += kLaThreads) qs[i] = from_storage(static_cast<const T*>(a.q)[(size_t(z) * a.heads + h0 + i / a.dim_pad) * a.q_pad + i % a.dim_pad]);
     }
-    float acc[H][P];
+    float acc[H][P], slope[H], bias[H];
+#pragma unroll
+    for (int h = 0; h < H; ++h) slope[h] = a.slope[h0 + min(h, nh - 1)], bias[h] = a.bias[h0 + min(h, nh - 1)];
 #pragma unroll
     for (int h = 0; h < H; ++h)
 #pragma unroll
@@ -234,17 +237,22 @@ __global__ void __launch_bounds__(kLaThreads, H > 4 ? 1 : 2) logistic_step_kerne
                             for (int u = 0; u < 4; ++u) s[u][h] = fmaf(q[e], kf[u][e], s[u][h]);
                     }
             }
+            for (int o = key_lanes >> 1; o > 0; o >>= 1)
 #pragma unroll
-            for (int h = 0; h < H; ++h)
-                if (h < nh) {
+                for (int h = 0; h < H; ++h)
 #pragma unroll
-                    for (int u = 0; u < 4; ++u) {
-                        float v = s[u][h];
-                        for (int o = key_lanes >> 1; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-                        const int r = r0 + u * kgroups;
-                        if (kl == 0 && r < nt) ws[h * kLaKeys + r] = sigmoid_f(v * a.scale - a.slope[h0 + h] * static_cast<float>(pos - t0 - r) + a.bias[h0 + h]);
+                    for (int u = 0; u < 4; ++u) s[u][h] += __shfl_xor_sync(0xffffffffu, s[u][h], o);
+            if (kl == 0) {
+#pragma unroll
+                for (int h = 0; h < H; ++h)
+                    if (h < nh) {
+#pragma unroll
+                        for (int u = 0; u < 4; ++u) {
+                            const int r = r0 + u * kgroups;
+                            if (r < nt) ws[h * kLaKeys + r] = sigmoid_f(s[u][h] * a.scale - slope[h] * static_cast<float>(pos - t0 - r) + bias[h]);
+                        }
                     }
-                }
+            }
         }
         __syncthreads();
         for (int r0 = vg; r0 < nt; r0 += 8 * vgroups) {
@@ -267,17 +275,18 @@ __global__ void __launch_bounds__(kLaThreads, H > 4 ? 1 : 2) logistic_step_kerne
     }
     // sums of the key groups: those of a warp by shuffles, then through shared memory
     const int rows = value_lanes < 32 ? kLaThreads / 32 : vgroups, mine = value_lanes < 32 ? warp : vg;
+    for (int o = 16; o >= value_lanes; o >>= 1)
 #pragma unroll
-    for (int h = 0; h < H; ++h)
-        if (h < nh) {
+        for (int h = 0; h < H; ++h)
 #pragma unroll
-            for (int e = 0; e < P; ++e) {
-                float v = acc[h][e];
-                for (int o = 16; o >= value_lanes; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-                const int c = vl * P + e;
-                if ((value_lanes >= 32 || lane < value_lanes) && c < a.vdim) red[(mine * H + h) * a.vdim + c] = v;
-            }
-        }
+            for (int e = 0; e < P; ++e) acc[h][e] += __shfl_xor_sync(0xffffffffu, acc[h][e], o);
+    if (value_lanes >= 32 || lane < value_lanes) {
+#pragma unroll
+        for (int h = 0; h < H; ++h)
+#pragma unroll
+            for (int e = 0; e < P; ++e)
+                if (h < nh && vl * P + e < a.vdim) red[(mine * H + h) * a.vdim + vl * P + e] = acc[h][e];
+    }
     __syncthreads();
     for (int i = tid; i < nh * a.vdim; i += kLaThreads) {
         const int h = i / a.vdim, c = i % a.vdim;

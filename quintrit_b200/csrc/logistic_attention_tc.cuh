@@ -4,7 +4,7 @@
 //   * one thread fetches the queries once and then keys and values of tile after tile with TMA (64-column slices, 128-byte swizzle) into three stages;
 //   * one thread issues S = Q K^T (both operands from shared memory) into one of two score areas of tensor memory and, a tile behind,
 //     O += P V with P from tensor memory and V as it lies in the cache - rows are keys, so it is the operand whose N runs fastest;
-//   * eight warps make the weights: a query row per lane (a warp reaches the 32 lanes that its index modulo 4 selects, two warps share them by
+//   * sixteen warps make the weights: a query row per lane (a warp reaches the 32 lanes that its index modulo 4 selects, four warps share them by
 //     columns), read with tcgen05.ld, written back as bf16 pairs over the scores they came from with tcgen05.st. A weight depends on its own score
 //     alone: nothing is rescaled, O stays in tensor memory until the end.
 //
@@ -18,7 +18,7 @@
 namespace qtb {
 
 constexpr int kLtRows = 128, kLtKeys = 128, kLtStages = 3;
-constexpr int kLtWeightWarps = 8, kLtThreads = 64 + 32 * kLtWeightWarps;  // TMA warp, MMA warp, weight warps
+constexpr int kLtWeightWarps = 16, kLtThreads = 64 + 32 * kLtWeightWarps;  // TMA warp, MMA warp, weight warps
 constexpr int kLtSlice = kLtKeys * 64 * 2;                                // bytes of a 64-column slice of 128 rows
 
 inline int logistic_tc_slices(int dim) { return (dim + 63) / 64; }
@@ -35,6 +35,12 @@ struct LogisticTcArgs {
     unsigned int* status;
     unsigned int spin_limit;
 };
+
+__device__ __forceinline__ float fast_reciprocal(float x) {
+    float y;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
 
 namespace dense_detail {
 __device__ __forceinline__ void mma_bf16_ts(uint32_t tmem_d, uint32_t tmem_a, uint64_t desc_b, uint32_t idesc, uint32_t accumulate) {
@@ -142,17 +148,17 @@ __global__ void __launch_bounds__(kLtThreads, 1) logistic_tc_kernel(const __grid
                 const int s = tile % kLtStages;
                 if (!(okay = mbar_wait(p_full(tile & 1), (tile >> 1) & 1, abort_flag, t.spin_limit) && mbar_wait(v_loaded(s), (tile / kLtStages) & 1, abort_flag, t.spin_limit))) break;
                 asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-                // slices of 64 columns of V lie kLtSlice apart, groups of eight keys 1024 bytes; the weights of keys 64 .. 127 begin at column 64 of the area
+                // slices of 64 columns of V lie kLtSlice apart, groups of eight keys 1024 bytes; the weights of 32 keys begin where their scores did
                 const uint64_t dv = smem_desc(stage0 + s * stage_bytes + ks * kLtSlice, kLtSlice, 1024, 2);
 #pragma unroll
                 for (int k = 0; k < kLtKeys / 16; ++k)
-                    mma_bf16_ts(o_acc, tmem + (tile & 1) * kLtKeys + (k >> 2) * 64 + (k & 3) * 8, dv + k * (2048 >> 4), out_desc, tile == 0 && k == 0 ? 0u : 1u);
+                    mma_bf16_ts(o_acc, tmem + (tile & 1) * kLtKeys + (k >> 1) * 32 + (k & 1) * 8, dv + k * (2048 >> 4), out_desc, tile == 0 && k == 0 ? 0u : 1u);
                 mma_commit(v_empty(s));
             }
             mma_commit(o_full);  // (also on the way out after a failed wait)
         }
     } else {
-        const int r = (warp & 3) * 32 + lane, half = (warp - 2) >> 2, row = first + r;
+        const int r = (warp & 3) * 32 + lane, part = (warp - 2) >> 2, row = first + r;
         const uint32_t mine = tmem + (uint32_t((warp & 3) * 32) << 16);
         // exp(-score) = exp2(-log2(e) score): the sign and log2(e) go into the factors
         constexpr float kLog2e = 1.4426950408889634f;
@@ -163,28 +169,27 @@ __global__ void __launch_bounds__(kLtThreads, 1) logistic_tc_kernel(const __grid
             okay = __shfl_sync(0xffffffffu, okay ? 1 : 0, 0) != 0;
             if (!okay) break;
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-            const uint32_t area = mine + (tile & 1) * kLtKeys + half * 64;
-            const int k0 = tile * kLtKeys + half * 64;
+            const uint32_t area = mine + (tile & 1) * kLtKeys + part * 32;
+            const int k0 = tile * kLtKeys + part * 32;
             const float base = fmaf(slope, static_cast<float>(row - k0), bias);
-            const bool open = k0 + 63 <= first;  // every row sees these keys
-#pragma unroll
-            for (int part = 0; part < 2; ++part) {
-                uint32_t v[2][16], p[16];
-                tmem_load16(area + part * 32, v[0]), tmem_load16(area + part * 32 + 16, v[1]);
-                asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+            uint32_t v[2][16], p[16];
+            tmem_load16(area, v[0]), tmem_load16(area + 16, v[1]);
+            asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+            auto weights = [&](bool open) {
 #pragma unroll
                 for (int i = 0; i < 16; ++i) {
-                    const int j = part * 32 + 2 * i;
-                    const float x0 = fmaf(__uint_as_float(v[i >> 3][(2 * i) & 15]), scale, fmaf(-slope, static_cast<float>(j), base));
-                    const float x1 = fmaf(__uint_as_float(v[i >> 3][(2 * i + 1) & 15]), scale, fmaf(-slope, static_cast<float>(j + 1), base));
-                    const float d0 = 1.0f + fast_exp2(fminf(x0, 62.0f)), d1 = 1.0f + fast_exp2(fminf(x1, 62.0f)), both = __fdividef(1.0f, d0 * d1);
+                    const int j = 2 * i;
+                    const float x0 = fmaf(__uint_as_float(v[i >> 3][j & 15]), scale, fmaf(-slope, static_cast<float>(j), base));
+                    const float x1 = fmaf(__uint_as_float(v[i >> 3][(j + 1) & 15]), scale, fmaf(-slope, static_cast<float>(j + 1), base));
+                    const float d0 = 1.0f + fast_exp2(fminf(x0, 62.0f)), d1 = 1.0f + fast_exp2(fminf(x1, 62.0f)), both = fast_reciprocal(d0 * d1);
                     float w0 = both * d1, w1 = both * d0;
                     if (!open) w0 = k0 + j <= row ? w0 : 0.0f, w1 = k0 + j + 1 <= row ? w1 : 0.0f;
                     p[i] = pack_bf16(w0, w1);
                 }
-                // over the first quarter of this warp's scores, then the second: all of the first part has been read when it is written
-                tmem_store16(area + part * 16, p);
-            }
+            };
+            if (k0 + 31 <= first) weights(true);  // every row sees these keys
+            else weights(false);
+            tmem_store16(area, p);  // over the first half of the scores they came from
             asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
             asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
             __syncwarp();
@@ -196,7 +201,7 @@ __global__ void __launch_bounds__(kLtThreads, 1) logistic_tc_kernel(const __grid
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
             bf16* out = static_cast<bf16*>(a.out) + size_t(q0 + r) * a.out_pitch + size_t(head) * a.vdim;
             const bool there = q0 + r < a.tokens, wide = a.vdim % 8 == 0;  // (pitches are multiples of 64: rows of eight start at 16 bytes)
-            for (int c = half * 16; c < a.vdim; c += 32) {
+            for (int c = part * 16; c < a.vdim; c += 64) {
                 uint32_t v[16];
                 tmem_load16(mine + 2 * kLtKeys + c, v);
                 asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");

@@ -15,7 +15,8 @@ namespace qtb {
 constexpr int kRetT = 64;      // tokens of a chunk
 constexpr int kRetV = 64;      // value columns per block of the state kernel
 constexpr int kRetPart = 32;   // value columns per turn of the output kernel
-constexpr int kRetPrep = 16;   // tokens per block of the preparing kernel
+constexpr int kRetPrep = 8;    // tokens per block of the preparing kernel
+constexpr int kRetStages = 3;
 
 // Compiled sizes: rows of the state and value columns, 0 if a head is too large.
 inline int retention_rows(int dim) { return dim <= 32 ? 32 : dim <= 64 ? 64 : dim <= 128 ? 128 : dim <= 256 ? 256 : 0; }
@@ -51,17 +52,17 @@ __device__ __forceinline__ void decay_powers(float decay, float* pw) {
     for (int i = threadIdx.x; i <= kRetT; i += blockDim.x) pw[i] = i == 0 ? 1.0f : decay > 0.0f ? exp2f(static_cast<float>(i) * log2f(decay)) : 0.0f;
 }
 // Queries, keys and values of every token as the products take them. PAIRS: two neighbouring elements at a time (even sizes and columns).
-// Four heads a block: they share the angles. grid: (ceil(heads / 4), padded tokens / 16), 128 threads
+// Four heads a block: they share the angles. grid: (ceil(heads / 4), padded tokens / 8), 256 threads
 template <bool PAIRS>
-__global__ void __launch_bounds__(128) retention_prepare_kernel(const __grid_constant__ RetentionArgs r) {
+__global__ void __launch_bounds__(256) retention_prepare_kernel(const __grid_constant__ RetentionArgs r) {
     __shared__ float2 angle[kRetPrep][128];  // (a head has at most 256 rotated dimensions)
     const ScanArgs& a = r.scan;
     const RetentionWork& w = r.work;
     constexpr int S = PAIRS ? 2 : 1;
-    const int t0 = blockIdx.y * kRetPrep, tid = threadIdx.x, n = a.n, half = a.rot_dims / 2;
+    const int t0 = blockIdx.y * kRetPrep, tid = threadIdx.x, n = a.n, half = a.rot_dims / 2, head0 = blockIdx.x * 4, heads = min(4, a.heads - head0);
     const uint32_t pos0 = seq_position(a.seq, a.pos, 0);
     const float scale = 1.0f / sqrtf(static_cast<float>(n));
-    for (int i = tid; i < kRetPrep * half; i += 128) angle[i / half][i % half] = rotation(a.turns[i % half], pos0 + t0 + i / half);
+    for (int i = tid; i < kRetPrep * half; i += 256) angle[i / half][i % half] = rotation(a.turns[i % half], pos0 + t0 + i / half);
     __syncthreads();
     auto put = [&](bf16* hi, bf16* lo, size_t at, const float (&v)[S]) {
         if constexpr (PAIRS) {
@@ -75,50 +76,43 @@ __global__ void __launch_bounds__(128) retention_prepare_kernel(const __grid_con
     };
     auto get = [&](const float* p, bool there, float (&v)[S]) {
         if constexpr (PAIRS) {
-            const float2 f = there ? *reinterpret_cast<const float2*>(p) : make_float2(0.0f, 0.0f);
+            const float2 f = there ? __ldg(reinterpret_cast<const float2*>(p)) : make_float2(0.0f, 0.0f);
             v[0] = f.x, v[1] = f.y;
         } else {
-            v[0] = there ? *p : 0.0f;
+            v[0] = there ? __ldg(p) : 0.0f;
         }
     };
     const int items = (w.rows - half) / S, cols = w.v_pad / S;  // an item is a pair to rotate (two neighbouring ones), or elements that stay as they are
-    for (int head = blockIdx.x * 4; head < min(a.heads, static_cast<int>(blockIdx.x) * 4 + 4); ++head) {
 #pragma unroll 4
-        for (int i = tid; i < kRetPrep * items; i += 128) {
-            const int t = t0 + i / items, j = i % items * S;
-            const bool there = t < a.tokens;
-            const float* p = a.p + size_t(min(t, a.tokens - 1)) * a.ld + head * n;
-            const float* pk = p + a.heads * n;
-            const size_t at = (size_t(head) * w.tokens + t) * w.rows;
-            float q[S], k[S];
-            if (j < half) {
-                float q2[S], k2[S];
-                get(p + j, there, q), get(p + j + half, there, q2), get(pk + j, there, k), get(pk + j + half, there, k2);
+    for (int i = tid; i < heads * kRetPrep * items; i += 256) {
+        const int row = i / items, j = i % items * S, head = head0 + row / kRetPrep, t = t0 + row % kRetPrep;
+        const bool there = t < a.tokens;
+        const float* p = a.p + size_t(min(t, a.tokens - 1)) * a.ld + head * n;
+        const float* pk = p + a.heads * n;
+        const size_t at = (size_t(head) * w.tokens + t) * w.rows;
+        const bool turns = j < half, in = there && j + half < n;  // (a rotated pair's second element is below n)
+        float q[S], k[S], q2[S], k2[S];
+        get(p + j, there && turns, q), get(p + j + half, in, q2), get(pk + j, there && turns, k), get(pk + j + half, in, k2);
 #pragma unroll
-                for (int e = 0; e < S; ++e) {
-                    const float2 cs = angle[t - t0][j + e];
-                    const float2 rq = rotate_pair(q[e], q2[e], cs), rk = rotate_pair(k[e], k2[e], cs);
-                    q[e] = rq.x, q2[e] = rq.y, k[e] = rk.x * scale, k2[e] = rk.y * scale;
-                }
-                put(w.q_hi, w.q_lo, at + j, q), put(w.q_hi, w.q_lo, at + j + half, q2);
-                put(w.k_hi, w.k_lo, at + j, k), put(w.k_hi, w.k_lo, at + j + half, k2);
-            } else {
-                const bool in = there && j + half < n;
-                get(p + j + half, in, q), get(pk + j + half, in, k);
-#pragma unroll
-                for (int e = 0; e < S; ++e) k[e] *= scale;
-                put(w.q_hi, w.q_lo, at + j + half, q), put(w.k_hi, w.k_lo, at + j + half, k);
+        for (int e = 0; e < S; ++e) {
+            if (turns) {
+                const float2 cs = angle[t - t0][j + e];
+                const float2 rq = rotate_pair(q[e], q2[e], cs), rk = rotate_pair(k[e], k2[e], cs);
+                q[e] = rq.x, q2[e] = rq.y, k[e] = rk.x, k2[e] = rk.y;
             }
+            k[e] *= scale, k2[e] *= scale;
         }
+        if (turns) put(w.q_hi, w.q_lo, at + j, q), put(w.k_hi, w.k_lo, at + j, k);
+        put(w.q_hi, w.q_lo, at + j + half, q2), put(w.k_hi, w.k_lo, at + j + half, k2);
+    }
 #pragma unroll 4
-        for (int i = tid; i < kRetPrep * cols; i += 128) {
-            const int t = t0 + i / cols, c = i % cols * S;
-            float v[S];
-            get(a.p + size_t(min(t, a.tokens - 1)) * a.ld + 2 * a.heads * n + head * a.vdim + c, t < a.tokens && c < a.vdim, v);
-            bf16* out = w.v + (size_t(head) * w.tokens + t) * w.v_pad + c;
-            if constexpr (PAIRS) *reinterpret_cast<uint32_t*>(out) = pack_bf16(v[0], v[1]);
-            else *out = __float2bfloat16_rn(v[0]);
-        }
+    for (int i = tid; i < heads * kRetPrep * cols; i += 256) {
+        const int row = i / cols, c = i % cols * S, head = head0 + row / kRetPrep, t = t0 + row % kRetPrep;
+        float v[S];
+        get(a.p + size_t(min(t, a.tokens - 1)) * a.ld + 2 * a.heads * n + head * a.vdim + c, t < a.tokens && c < a.vdim, v);
+        bf16* out = w.v + (size_t(head) * w.tokens + t) * w.v_pad + c;
+        if constexpr (PAIRS) *reinterpret_cast<uint32_t*>(out) = pack_bf16(v[0], v[1]);
+        else *out = __float2bfloat16_rn(v[0]);
     }
 }
 
@@ -216,21 +210,21 @@ __global__ void __launch_bounds__(128) retention_carry_kernel(const __grid_const
         if (v < a.vdim && d + e < a.n) state[d + e] = s[e];
 }
 
-// Outputs of a chunk. grid: (heads, chunks), 128 threads; a warp owns 16 tokens and all value columns, 32 of them at a time: the next 32 columns of
+// Outputs of a chunk. grid: (heads, chunks), 128 threads; a warp owns 16 tokens and all value columns, 32 of them at a time: the next 64 columns of
 // the state and the values are on their way while the products of these are made.
 template <int N> __host__ __device__ constexpr size_t retention_out_stage() { return size_t(2 * kRetPart) * (N + 8) * 2 + size_t(kRetT) * (kRetPart + 8) * 2; }
-template <int N> __host__ __device__ constexpr size_t retention_out_smem() {
-    const size_t keys = size_t(2 * kRetT) * (N + 8) * 2;  // (in the stages' place until the scores are made)
-    return keys + (2 * retention_out_stage<N>() > keys ? 2 * retention_out_stage<N>() : keys);
-}
+template <int N> __host__ __device__ constexpr size_t retention_out_smem() { return size_t(2 * kRetT) * (N + 8) * 2 + kRetStages * retention_out_stage<N>(); }
 template <int N, int V>
 __global__ void __launch_bounds__(128) retention_out_kernel(const __grid_constant__ RetentionArgs r) {
     extern __shared__ __align__(16) unsigned char rt_sm[];
     __shared__ float pw[kRetT + 1];
     const ScanArgs& a = r.scan;
     constexpr int kPitch = N + 8, kVPitch = kRetPart + 8, kParts = V / kRetPart, kCols = kRetPart / 8;
-    bf16 *qh = reinterpret_cast<bf16*>(rt_sm), *ql = qh + kRetT * kPitch, *kh = ql + kRetT * kPitch, *kl = kh + kRetT * kPitch;
-    unsigned char* stages = reinterpret_cast<unsigned char*>(kh);
+    constexpr size_t kStage = retention_out_stage<N>();
+    static_assert((kRetStages - 1) * kStage >= size_t(2 * kRetT) * kPitch * 2, "the keys fit the stages behind the first until the scores are made");
+    bf16 *qh = reinterpret_cast<bf16*>(rt_sm), *ql = qh + kRetT * kPitch;
+    unsigned char* stages = reinterpret_cast<unsigned char*>(ql + kRetT * kPitch);
+    bf16 *kh = reinterpret_cast<bf16*>(stages + kStage), *kl = kh + kRetT * kPitch;
     const int head = blockIdx.x, chunk = blockIdx.y, chunks = gridDim.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, c = lane & 3;
     const int t0 = chunk * kRetT, len = min(kRetT, a.tokens - t0), n = a.n;
     const size_t row0 = size_t(head) * r.work.tokens + t0;
@@ -241,8 +235,27 @@ __global__ void __launch_bounds__(128) retention_out_kernel(const __grid_constan
         cp_async16(kh + at, r.work.k_hi + from, true), cp_async16(kl + at, r.work.k_lo + from, true);
     }
     cp_async_commit_group();
+    auto fetch = [&](int part) {
+        if (part >= kParts) {
+            cp_async_commit_group();  // (an empty group keeps the count of groups in step with the parts)
+            return;
+        }
+        bf16 *sh = reinterpret_cast<bf16*>(stages + (part % kRetStages) * kStage), *sl = sh + kRetPart * kPitch, *vs = sl + kRetPart * kPitch;
+        const size_t at = ((size_t(head) * chunks + chunk) * r.work.v_pad + part * kRetPart) * N;
+        for (int i = tid; i < kRetPart * (N / 8); i += 128) {
+            const int v = i / (N / 8), p = i % (N / 8);
+            cp_async16(sh + v * kPitch + p * 8, r.work.s_hi + at + size_t(v) * N + p * 8, true);
+            cp_async16(sl + v * kPitch + p * 8, r.work.s_lo + at + size_t(v) * N + p * 8, true);
+        }
+        for (int i = tid; i < kRetT * (kRetPart / 8); i += 128) {
+            const int t = i / (kRetPart / 8), p = i % (kRetPart / 8);
+            cp_async16(vs + t * kVPitch + p * 8, r.work.v + (row0 + t) * r.work.v_pad + part * kRetPart + p * 8, true);
+        }
+        cp_async_commit_group();
+    };
+    fetch(0);
     decay_powers(a.decay[head], pw);
-    cp_async_wait_group<0>();
+    cp_async_wait_group<1>();
     __syncthreads();
     // decayed scores of the chunk's tokens, as A operands of the product with the values
     uint32_t ph[kRetT / 16][4], pl[kRetT / 16][4];
@@ -280,33 +293,15 @@ __global__ void __launch_bounds__(128) retention_out_kernel(const __grid_constan
         }
     }
     const float from_state[2] = {pw[warp * 16 + g + 1], pw[warp * 16 + g + 9]};
-    auto fetch = [&](int part) {
-        bf16 *sh = reinterpret_cast<bf16*>(stages + (part & 1) * retention_out_stage<N>()), *sl = sh + kRetPart * kPitch, *vs = sl + kRetPart * kPitch;
-        const size_t at = ((size_t(head) * chunks + chunk) * r.work.v_pad + part * kRetPart) * N;
-        for (int i = tid; i < kRetPart * (N / 8); i += 128) {
-            const int v = i / (N / 8), p = i % (N / 8);
-            cp_async16(sh + v * kPitch + p * 8, r.work.s_hi + at + size_t(v) * N + p * 8, true);
-            cp_async16(sl + v * kPitch + p * 8, r.work.s_lo + at + size_t(v) * N + p * 8, true);
-        }
-        for (int i = tid; i < kRetT * (kRetPart / 8); i += 128) {
-            const int t = i / (kRetPart / 8), p = i % (kRetPart / 8);
-            cp_async16(vs + t * kVPitch + p * 8, r.work.v + (row0 + t) * r.work.v_pad + part * kRetPart + p * 8, true);
-        }
-        cp_async_commit_group();
-    };
     __syncthreads();  // every warp is done with the keys
-    fetch(0);
+    fetch(1);
     float o[V / 8][4], ss[2] = {0.0f, 0.0f};
 #pragma unroll
     for (int part = 0; part < kParts; ++part) {
-        if (part + 1 < kParts) {
-            fetch(part + 1);
-            cp_async_wait_group<1>();
-        } else {
-            cp_async_wait_group<0>();
-        }
+        cp_async_wait_group<1>();
         __syncthreads();
-        const bf16 *sh = reinterpret_cast<const bf16*>(stages + (part & 1) * retention_out_stage<N>()), *sl = sh + kRetPart * kPitch, *vs = sl + kRetPart * kPitch;
+        fetch(part + 2);  // into the stage of the part before this one, which every warp has left
+        const bf16 *sh = reinterpret_cast<const bf16*>(stages + (part % kRetStages) * kStage), *sl = sh + kRetPart * kPitch, *vs = sl + kRetPart * kPitch;
         float (*po)[4] = o + part * kCols;
 #pragma unroll
         for (int j = 0; j < kCols; ++j)
@@ -344,7 +339,6 @@ __global__ void __launch_bounds__(128) retention_out_kernel(const __grid_constan
         for (int j = 0; j < kCols; ++j)
 #pragma unroll
             for (int e = 0; e < 4; ++e) ss[e >> 1] = fmaf(po[j][e], po[j][e], ss[e >> 1]);  // (columns beyond vdim are zero)
-        __syncthreads();  // the stage may be filled again
     }
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
@@ -358,11 +352,18 @@ __global__ void __launch_bounds__(128) retention_out_kernel(const __grid_constan
         const auto gated = [&](float v, float z) { return v * inv * __fdividef(z, 1.0f + __expf(-z)); };
         if (r.pairs) {
 #pragma unroll
-            for (int j = 0; j < V / 8; ++j) {
-                const int v = j * 8 + 2 * c;
-                if (v >= a.vdim) continue;
-                const float2 z = *reinterpret_cast<const float2*>(gate + v);
-                *reinterpret_cast<uint32_t*>(out + v) = pack_bf16(gated(o[j][2 * h], z.x), gated(o[j][2 * h + 1], z.y));
+            for (int j0 = 0; j0 < V / 8; j0 += 8) {
+                float2 z[8];  // eight loads in flight
+#pragma unroll
+                for (int j = 0; j < 8; ++j) {
+                    const int v = (j0 + j) * 8 + 2 * c;
+                    z[j] = v < a.vdim ? __ldg(reinterpret_cast<const float2*>(gate + v)) : make_float2(0.0f, 0.0f);
+                }
+#pragma unroll
+                for (int j = 0; j < 8; ++j) {
+                    const int v = (j0 + j) * 8 + 2 * c;
+                    if (v < a.vdim) *reinterpret_cast<uint32_t*>(out + v) = pack_bf16(gated(o[j0 + j][2 * h], z[j].x), gated(o[j0 + j][2 * h + 1], z[j].y));
+                }
             }
             continue;
         }
@@ -371,7 +372,7 @@ __global__ void __launch_bounds__(128) retention_out_kernel(const __grid_constan
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
                 const int v = j * 8 + 2 * c + e;
-                if (v < a.vdim) out[v] = __float2bfloat16_rn(gated(o[j][2 * h + e], gate[v]));
+                if (v < a.vdim) out[v] = __float2bfloat16_rn(gated(o[j][2 * h + e], __ldg(gate + v)));
             }
     }
 }

@@ -37,6 +37,15 @@ def test_describe_reads_every_size_and_constant(tmp_path):
     assert {t["name"]: t["shape"] for t in d["tensors"]} == {k: tuple(v) for k, v in mf.tosevik_shapes(config()).items()}
 
 
+def test_parts_that_may_be_left_out(tmp_path):
+    cfg = config([mf.retention_layer(mf.retention(2, 8, 8), mf.experts(4, 2, 8, 8)), mf.parallel_layer(mf.logistic(2, 1, 8, 8), mf.retention(2, 8, 8))])
+    tensors = mf.random_tosevik(cfg, 1)
+    del cfg["layers"][0]["mixer"]["rot"], cfg["layers"][0]["mlp"]["router"]["groups"]
+    cfg["layers"][1]["mixer"]["left"]["q_temp"] = None
+    d = q.gguf_describe(folder(tmp_path, cfg, tensors))
+    assert "rot=0/" in d["layer_0"] and "groups=1/1" in d["layer_0"] and "q_temp=0/1 " in d["layer_1"]
+
+
 def refused(path, code, text=""):
     with pytest.raises(q.QuintritError) as e:
         q.gguf_describe(path)
