@@ -97,6 +97,16 @@ __device__ __forceinline__ float warp_sum(float v) {
     for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
     return v;
 }
+__device__ __forceinline__ float2 block_sum2(float2 v, float2* sh) {  // two sums at once; sh: one float2 per warp
+    v = make_float2(warp_sum(v.x), warp_sum(v.y));
+    const int w = threadIdx.x >> 5, nw = blockDim.x >> 5;
+    __syncthreads();
+    if ((threadIdx.x & 31) == 0) sh[w] = v;
+    __syncthreads();
+    float2 t = make_float2(0.0f, 0.0f);
+    for (int i = 0; i < nw; ++i) t.x += sh[i].x, t.y += sh[i].y;
+    return t;
+}
 __device__ __forceinline__ float block_sum(float v, float* sh) {  // sh: one float per warp
     v = warp_sum(v);
     const int w = threadIdx.x >> 5, nw = blockDim.x >> 5;
@@ -201,6 +211,7 @@ template <typename T>
 __global__ void __launch_bounds__(kProjectThreads, 4) norm_project_kernel(NormProjectArgs a) {
     extern __shared__ float act_smem[];
     __shared__ float red[kProjectThreads / 32];
+    __shared__ float2 red2[kProjectThreads / 32];
     const int tid = threadIdx.x, token = blockIdx.y, pitch = a.stack[0].pitch;
     const float* x = a.x + size_t(token) * a.width;
     const int warps = gridDim.x * (kProjectThreads / 32);
@@ -224,7 +235,8 @@ __global__ void __launch_bounds__(kProjectThreads, 4) norm_project_kernel(NormPr
         float sl = 0.0f, sr = 0.0f;
 #pragma unroll 4
         for (int i = tid; i < a.width; i += kProjectThreads) sl += l[i] * l[i], sr += r[i] * r[i];
-        sl = block_sum(sl, red), sr = block_sum(sr, red);
+        const float2 both = block_sum2(make_float2(sl, sr), red2);
+        sl = both.x, sr = both.y;
         const float il = 0.5f / sqrtf(sl / static_cast<float>(a.width) + a.eps), ir = 0.5f / sqrtf(sr / static_cast<float>(a.width) + a.eps);
 #pragma unroll 4
         for (int i = tid; i < a.width; i += kProjectThreads) {
@@ -536,6 +548,7 @@ template <typename T>
 __global__ void __launch_bounds__(256) rows_kernel(const __grid_constant__ RowsArgs a) {
     extern __shared__ float act_smem[];
     __shared__ float red[8];
+    __shared__ float2 red2[8];
     const size_t t = blockIdx.x, row = t * a.width;
     const int tid = threadIdx.x;
     float il = 0.0f, ir = 0.0f;
@@ -547,7 +560,8 @@ __global__ void __launch_bounds__(256) rows_kernel(const __grid_constant__ RowsA
             const float l = a.pair.r[0][row + i], r = a.pair.r[1][row + i];
             sl += l * l, sr += r * r;
         }
-        sl = block_sum(sl, red), sr = block_sum(sr, red);
+        const float2 both = block_sum2(make_float2(sl, sr), red2);
+        sl = both.x, sr = both.y;
         il = 0.5f / sqrtf(sl / static_cast<float>(a.width) + a.eps), ir = 0.5f / sqrtf(sr / static_cast<float>(a.width) + a.eps);
     }
     float ss = 0.0f;

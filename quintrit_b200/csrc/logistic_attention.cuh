@@ -202,9 +202,7 @@ __global__ void __launch_bounds__(kLaThreads, H > 4 ? 1 : 2) logistic_step_kerne
     } else {
         for (int i = tid; i < nh * a.dim_pad; i += kLaThreads) qs[i] = from_storage(static_cast<const T*>(a.q)[(size_t(z) * a.heads + h0 + i / a.dim_pad) * a.q_pad + i % a.dim_pad]);
     }
-    float acc[H][P], slope[H], bias[H];
-#pragma unroll
-    for (int h = 0; h < H; ++h) slope[h] = a.slope[h0 + min(h, nh - 1)], bias[h] = a.bias[h0 + min(h, nh - 1)];
+    float acc[H][P];
 #pragma unroll
     for (int h = 0; h < H; ++h)
 #pragma unroll
@@ -245,14 +243,17 @@ __global__ void __launch_bounds__(kLaThreads, H > 4 ? 1 : 2) logistic_step_kerne
             if (kl == 0) {
 #pragma unroll
                 for (int h = 0; h < H; ++h)
-                    if (h < nh) {
 #pragma unroll
-                        for (int u = 0; u < 4; ++u) {
-                            const int r = r0 + u * kgroups;
-                            if (r < nt) ws[h * kLaKeys + r] = sigmoid_f(s[u][h] * a.scale - slope[h] * static_cast<float>(pos - t0 - r) + bias[h]);
-                        }
+                    for (int u = 0; u < 4; ++u) {
+                        const int r = r0 + u * kgroups;
+                        if (h < nh && r < nt) ws[h * kLaKeys + r] = s[u][h];
                     }
             }
+        }
+        __syncthreads();
+        for (int i = tid; i < nh * kLaKeys; i += kLaThreads) {  // (entries beyond nt are not used)
+            const int h = i / kLaKeys, r = i % kLaKeys;
+            if (r < nt) ws[i] = sigmoid_f(ws[i] * a.scale - a.slope[h0 + h] * static_cast<float>(pos - t0 - r) + a.bias[h0 + h]);
         }
         __syncthreads();
         for (int r0 = vg; r0 < nt; r0 += 8 * vgroups) {
