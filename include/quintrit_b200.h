@@ -292,10 +292,11 @@ typedef struct quintrit_gpu_options {
  * query/key-norm models QUINTRIT_ERR_UNSUPPORTED (a file whose projections are all Q2_0 runs through the block-scaled kernels). On failure *out_decoder is NULL. The decoder owns the weights.
  */
 /* `path` may also be a model folder (config.json + model.safetensors): config.json's "architecture" names the design, and its sizes, constants
- * and layers describe the model (Lasosun: mamba2, hgrn2 and windowed attention layers). Such a model serves in bfloat16, or in 32-bit
+ * and layers describe the model (Lasosun: mamba2, hgrn2 and windowed attention layers; Tosevik: retention, logistic attention beside retention,
+ * mixtures of experts). Such a model serves in bfloat16, or in 32-bit
  * arithmetic throughout with the flag QUINTRIT_B200_OPEN_FLOAT32 in options.flags (also of quintrit_model_open_gpu). Its layers keep recurrent
- * states and windows instead of a cache of every token, so a sequence continues from its end or starts again from position 0
- * (QUINTRIT_ERR_UNSUPPORTED for a position between), and its context may have any length up to the model's number of positions. */
+ * states, so a sequence continues from its end or starts again from position 0 (QUINTRIT_ERR_UNSUPPORTED for a position between). The context
+ * may have any length up to the model's number of positions; a model without such a bound takes options.context_length, 8192 if that is 0. */
 #define QUINTRIT_B200_OPEN_FLOAT32 0x100u
 int quintrit_b200_decoder_open_gguf(const char* path, const quintrit_gpu_options_t* options, quintrit_b200_decoder_t** out_decoder);
 

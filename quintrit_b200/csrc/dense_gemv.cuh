@@ -207,7 +207,10 @@ struct NormProjectArgs {
 
 constexpr int kProjectThreads = 256;
 
-template <typename T>
+// FORM: what stands before the projections is known when the kernel is compiled, which keeps it short. kProjectRms: RMS norms; kProjectTanh: the tanh
+// norm; kProjectAny: either, of a pair sum (both of the latter also write h_out).
+enum ProjectForm : int { kProjectRms = 0, kProjectTanh = 1, kProjectAny = 2 };
+template <typename T, int FORM>
 __global__ void __launch_bounds__(kProjectThreads, 4) norm_project_kernel(NormProjectArgs a) {
     extern __shared__ float act_smem[];
     __shared__ float red[kProjectThreads / 32];
@@ -228,8 +231,14 @@ __global__ void __launch_bounds__(kProjectThreads, 4) norm_project_kernel(NormPr
             }
     }
     bool first = true;
+    if (FORM != kProjectRms && blockIdx.x == 0 && tid == 0 && a.width >= 4) {  // vectors that every block reads after the wait
+        const uint32_t bytes = a.width * 4 & ~15;
+        l2_prefetch(a.norm[0].w, bytes);
+        if (a.norm[0].b != nullptr) l2_prefetch(a.norm[0].b, bytes);
+        if (a.pair.r[0] != nullptr) l2_prefetch(a.pair.w[0], bytes), l2_prefetch(a.pair.w[1], bytes);
+    }
     pdl_wait();
-    if (a.pair.r[0] != nullptr) {
+    if (FORM == kProjectAny && a.pair.r[0] != nullptr) {
         float* sum = act_smem + a.n_stack * pitch;
         const float *l = a.pair.r[0] + size_t(token) * a.width, *r = a.pair.r[1] + size_t(token) * a.width;
         float sl = 0.0f, sr = 0.0f;
@@ -247,7 +256,7 @@ __global__ void __launch_bounds__(kProjectThreads, 4) norm_project_kernel(NormPr
         x = sum;  // (each thread reads back what it wrote)
     }
     float inv = 1.0f;
-    if (a.norm[0].b == nullptr) {
+    if (FORM == kProjectRms || (FORM == kProjectAny && a.norm[0].b == nullptr)) {
         float ss = 0.0f;
 #pragma unroll 4
         for (int i = tid; i < a.width; i += kProjectThreads) ss += x[i] * x[i];
@@ -256,9 +265,12 @@ __global__ void __launch_bounds__(kProjectThreads, 4) norm_project_kernel(NormPr
     for (int s = 0; s < a.n_stack; ++s)
 #pragma unroll 4
         for (int i = tid; i < pitch; i += kProjectThreads) {
-            const float v = i < a.width ? round_to<T>(norm_value(a.norm[s], x[i], inv, i)) : 0.0f;
+            const float v = i < a.width ? round_to<T>(FORM == kProjectRms    ? x[i] * inv * a.norm[s].w[i]
+                                                        : FORM == kProjectTanh ? tanhf(a.norm[s].alpha * x[i]) * a.norm[s].w[i] + a.norm[s].b[i]
+                                                                               : norm_value(a.norm[s], x[i], inv, i))
+                                          : 0.0f;
             act_smem[s * pitch + act_index<T>(i, pitch)] = v;
-            if (a.h_out != nullptr && s == 0 && blockIdx.x == 0) static_cast<T*>(a.h_out)[size_t(token) * pitch + i] = to_storage<T>(v);
+            if (FORM != kProjectRms && a.h_out != nullptr && s == 0 && blockIdx.x == 0) static_cast<T*>(a.h_out)[size_t(token) * pitch + i] = to_storage<T>(v);
         }
     __syncthreads();
     for (int s = 0; s < a.n_stack; ++s)
@@ -285,13 +297,13 @@ __global__ void __launch_bounds__(kProjectThreads, 4) norm_project_kernel(NormPr
 }
 
 // ---- output norm of a mixer -----------------------------------------------------------------------------------------------------------
-// y of one token in `parts` equal parts, each divided by its own root mean square, times w[i % w_len] (w may be nullptr) and times
-// silu(gate[i]) (gate may be nullptr); in place in shared memory, in the order act_index<T>. red: one float per warp.
-template <typename T>
+// y of one token in `parts` equal parts, each divided by its own root mean square, times w[i % w_len], or with GATED times silu(gate[i]) instead
+// (gate may be nullptr); in place in shared memory, in the order act_index<T>. red: one float per warp.
+template <typename T, bool GATED>
 __device__ __forceinline__ void parts_norm(float* y, int n, int pitch, int parts, float eps, const float* w, int w_len, const float* gate, float* red) {
     const auto ending = [&](float v, int e) {
-        if (w != nullptr) v *= w[e % w_len];
-        return round_to<T>(gate != nullptr ? v * silu_f(gate[e]) : v);
+        if constexpr (GATED) return round_to<T>(gate != nullptr ? v * silu_f(gate[e]) : v);
+        else return round_to<T>(v * w[e % w_len]);
     };
     const int len = n / parts, warps = blockDim.x >> 5, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     if (parts >= warps) {  // a warp per part
@@ -381,7 +393,7 @@ __global__ void __launch_bounds__(kProjectThreads, 4) finish_project_kernel(Fini
         for (int i = tid; i < a.down_pitch / kPer; i += kProjectThreads) act_put_storage(m, i, a.down_pitch, static_cast<const T*>(a.m) + size_t(token) * a.down_pitch);
     }
     __syncthreads();
-    if (norm) parts_norm<T>(y, a.inner, a.o_pitch, a.norm_parts, a.eps, a.norm_w, a.norm_len, nullptr, red);
+    if (norm) parts_norm<T, false>(y, a.inner, a.o_pitch, a.norm_parts, a.eps, a.norm_w, a.norm_len, nullptr, red);
     for (int row = blockIdx.x * (kProjectThreads / 32) + (tid >> 5); row < a.width; row += warps) {
         float so[1], sd[1] = {0.0f};
         const T *o_row = static_cast<const T*>(a.o) + size_t(row) * a.o_pitch, *d_row = static_cast<const T*>(a.down) + size_t(row) * a.down_pitch;
@@ -447,7 +459,7 @@ __global__ void __launch_bounds__(kProjectThreads, 4) out_project_kernel(const _
             if (gate != nullptr && i < m.inner) gates[i] = z;
         }
         __syncthreads();
-        if (m.parts > 0) parts_norm<T>(y, m.inner, m.pitch, m.parts, a.eps, nullptr, 1, gate != nullptr ? gates : nullptr, red);
+        if (m.parts > 0) parts_norm<T, true>(y, m.inner, m.pitch, m.parts, a.eps, nullptr, 1, gate != nullptr ? gates : nullptr, red);
         else __syncthreads();
     }
     for (int unit = unit0; unit < units; unit += warps) {
@@ -628,7 +640,7 @@ __global__ void __launch_bounds__(256) rows_kernel(const __grid_constant__ RowsA
 }
 
 // The mixer's output norm of many tokens (parts_norm), into the storage type; without a norm a plain conversion. gate (may be nullptr):
-// y is first multiplied by silu(gate[token * gate_ld + i]); gate_after: the normed y is.
+// y is first multiplied by silu(gate[token * gate_ld + i]); gate_after: the normed y is (w is then nullptr).
 template <typename T>
 __global__ void __launch_bounds__(256) finish_rows_kernel(const float* y, const float* gate, const float* gate_after, int gate_ld, int inner, int parts, float eps, const float* w, int w_len, T* out,
                                                           int pitch) {
@@ -640,7 +652,8 @@ __global__ void __launch_bounds__(256) finish_rows_kernel(const float* y, const 
         act_smem[i] = gate != nullptr ? v * silu_f(gate[size_t(t) * gate_ld + i]) : v;
     }
     __syncthreads();
-    if (parts > 0) parts_norm<float>(act_smem, inner, inner, parts, eps, w, w_len, gate_after != nullptr ? gate_after + size_t(t) * gate_ld : nullptr, red);
+    if (parts > 0 && w != nullptr) parts_norm<float, false>(act_smem, inner, inner, parts, eps, w, w_len, nullptr, red);
+    else if (parts > 0) parts_norm<float, true>(act_smem, inner, inner, parts, eps, nullptr, 1, gate_after != nullptr ? gate_after + size_t(t) * gate_ld : nullptr, red);
     for (int i = threadIdx.x; i < inner; i += blockDim.x) out[size_t(t) * pitch + i] = to_storage<T>(act_smem[i]);
 }
 

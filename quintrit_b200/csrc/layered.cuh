@@ -521,7 +521,9 @@ inline int layered_decoder_setup(quintrit_b200_decoder* d, const std::shared_ptr
         QTB_CUDA(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, optin - static_cast<int>(fa.sharedSizeBytes)));
         return QUINTRIT_OK;
     };
-    std::vector<const void*> kernels = {reinterpret_cast<const void*>(norm_project_kernel<bf16>), reinterpret_cast<const void*>(norm_project_kernel<float>),
+    std::vector<const void*> kernels = {reinterpret_cast<const void*>(norm_project_kernel<bf16, kProjectRms>), reinterpret_cast<const void*>(norm_project_kernel<float, kProjectRms>),
+                             reinterpret_cast<const void*>(norm_project_kernel<bf16, kProjectTanh>), reinterpret_cast<const void*>(norm_project_kernel<float, kProjectTanh>),
+                             reinterpret_cast<const void*>(norm_project_kernel<bf16, kProjectAny>), reinterpret_cast<const void*>(norm_project_kernel<float, kProjectAny>),
                              reinterpret_cast<const void*>(finish_project_kernel<bf16>), reinterpret_cast<const void*>(finish_project_kernel<float>),
                              reinterpret_cast<const void*>(finish_rows_kernel<bf16>), reinterpret_cast<const void*>(finish_rows_kernel<float>),
                              reinterpret_cast<const void*>(out_project_kernel<bf16>), reinterpret_cast<const void*>(out_project_kernel<float>),
@@ -579,6 +581,11 @@ inline DenseStack layered_stack(const LayeredMatrix& w) {
     DenseStack s{};
     s.w = w.w, s.pitch = w.pitch, s.cols = w.cols;
     return s;
+}
+
+template <typename T> void (*layered_project_kernel(const NormProjectArgs& a))(NormProjectArgs) {
+    if (a.pair.r[0] != nullptr || (a.norm[0].b == nullptr && a.h_out != nullptr)) return norm_project_kernel<T, kProjectAny>;
+    return a.norm[0].b != nullptr ? norm_project_kernel<T, kProjectTanh> : norm_project_kernel<T, kProjectRms>;
 }
 
 // The two stacks of a layer's projections with their endings; returns how many there are.
@@ -830,7 +837,7 @@ int layered_parallel_layer(quintrit_b200_decoder* d, size_t li, int n, const Lay
             for (int k = 0; k < st[i].n_seg; ++k) units += (st[i].seg[k].rows + 1) / 2;
         }
         const int warps = kProjectThreads / 32;
-        launch_dependent(norm_project_kernel<T>, dim3(std::min((units + warps - 1) / warps, 4 * m.sm_count)), kProjectThreads, size_t(n_stack) * wp * sizeof(float), s, a);
+        launch_dependent(layered_project_kernel<T>(a), dim3(std::min((units + warps - 1) / warps, 4 * m.sm_count)), kProjectThreads, size_t(n_stack) * wp * sizeof(float), s, a);
         QTB_LAUNCH_CHECK();
         if ((rc = layered_mixer<T>(d, li, 0, n, tg, &ready)) != QUINTRIT_OK) return rc;
         FinishProjectArgs f{};
@@ -882,7 +889,7 @@ int layered_sequential_step(quintrit_b200_decoder* d, size_t li, const LayeredTa
         int units = 0;
         for (int k = 0; k < a.stack[0].n_seg; ++k) units += (a.stack[0].seg[k].rows + 1) / 2;
         a.eps = m.spec.eps, a.width = W, a.n_stack = 1;
-        launch_dependent(norm_project_kernel<T>, dim3(std::min((units + warps - 1) / warps, 4 * m.sm_count)), kProjectThreads, size_t(a.pair.r[0] != nullptr ? 2 : 1) * wp * sizeof(float), s, a);
+        launch_dependent(layered_project_kernel<T>(a), dim3(std::min((units + warps - 1) / warps, 4 * m.sm_count)), kProjectThreads, size_t(a.pair.r[0] != nullptr ? 2 : 1) * wp * sizeof(float), s, a);
         QTB_LAUNCH_CHECK();
         return QUINTRIT_OK;
     };
@@ -1075,7 +1082,7 @@ int layered_head(quintrit_b200_decoder* d, int row, float* logits) {
     a.stack[0] = layered_stack(m.head);
     a.stack[0].n_seg = 1, a.stack[0].seg[0] = DenseSeg{0, m.spec.vocab, kSegPlain, m.spec.vocab, logits, nullptr, nullptr};
     const int warps = kProjectThreads / 32;
-    launch_dependent(norm_project_kernel<T>, dim3(std::min((m.spec.vocab / 2 + warps) / warps, 4 * m.sm_count)), kProjectThreads, size_t(m.head.pitch) * sizeof(float), d->stream, a);
+    launch_dependent(layered_project_kernel<T>(a), dim3(std::min((m.spec.vocab / 2 + warps) / warps, 4 * m.sm_count)), kProjectThreads, size_t(m.head.pitch) * sizeof(float), d->stream, a);
     QTB_LAUNCH_CHECK();
     return QUINTRIT_OK;
 }
